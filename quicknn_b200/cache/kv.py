@@ -48,6 +48,7 @@ class LineView:
     writes: bool = True
     has_values: bool = True         # False: ``v`` is ``k`` (a line that keeps one row per position)
     index: int = -1                 # which cache line this is (a key for what layers hand each other within a step)
+    block_state: Optional[torch.Tensor] = None   # [slots, *shape]: fixed-size state of the block around the mixer, or None
     has_readers: bool = False       # another scheduled layer reads this line after its writer (set by the model)
 
 
@@ -80,7 +81,9 @@ class CacheGroup:
 
 class KVCache:
     def __init__(self, needs: Sequence[Optional[CacheNeed]], states: Sequence[Optional[StateNeed]],
-                 max_tokens: int, max_slots: int, max_seq: int, dtype: torch.dtype, device):
+                 max_tokens: int, max_slots: int, max_seq: int, dtype: torch.dtype, device,
+                 block_states: Sequence[Optional[StateNeed]] = ()):
+        """``needs``, ``states``: what the mixer of every line keeps; ``block_states``: the state of the block around it."""
         if max_tokens < 1 or max_slots < 1 or max_seq < 1:
             raise ValueError("max_tokens, max_slots and max_seq must be positive")
         self.dtype, self.device = dtype, device
@@ -110,11 +113,19 @@ class KVCache:
         self.longest_host = np.zeros(max_slots, dtype=np.int32)    # the longest that a slot's sequence has been: what its rings have overwritten
         self.lengths_dev = torch.zeros(max_slots, dtype=torch.int32, device=device)
         self._lengths_dirty = False
-        self.state: Dict[int, torch.Tensor] = {}
-        for line, st in enumerate(states):
-            if st is not None:
-                sd = dtype if st.dtype == "compute" else getattr(torch, st.dtype)
-                self.state[line] = torch.zeros((max_slots,) + tuple(st.shape), dtype=sd, device=device)
+        def regions(needed) -> Dict[int, torch.Tensor]:
+            out: Dict[int, torch.Tensor] = {}
+            for line, st in enumerate(needed):
+                if st is not None:
+                    sd = dtype if st.dtype == "compute" else getattr(torch, st.dtype)
+                    out[line] = torch.zeros((max_slots,) + tuple(st.shape), dtype=sd, device=device)
+            return out
+
+        self.state = regions(states)
+        self.block_state = regions(block_states)
+
+    def _all_states(self) -> List[torch.Tensor]:
+        return list(self.state.values()) + list(self.block_state.values())
 
     # ---- slots ------------------------------------------------------------------------
     def allocate(self) -> int:
@@ -122,7 +133,7 @@ class KVCache:
         self.lengths_host[slot] = 0
         self.longest_host[slot] = 0
         self._lengths_dirty = True
-        for t in self.state.values():
+        for t in self._all_states():
             t[slot].zero_()
         return slot
 
@@ -203,7 +214,7 @@ class KVCache:
         back to ``L - (ring - window + 1)`` at most; fixed-size state describes the whole sequence and cannot go back at all
         (the reference rebuilds recurrent state on a changed prefix, src/models/QuickNN.Models.LLM.pas:725-733)."""
         length, longest = int(self.lengths_host[slot]), int(self.longest_host[slot])
-        if self.state:
+        if self.state or self.block_state:
             return length
         limit = 0
         for g in self.groups:
@@ -228,17 +239,18 @@ class KVCache:
 
     # ---- views ------------------------------------------------------------------------
     def line(self, line: int, writes: bool = True) -> Optional[LineView]:
-        st = self.state.get(line)
+        st, bst = self.state.get(line), self.block_state.get(line)
         if line not in self._line_group:
-            if st is None:
+            if st is None and bst is None:
                 return None
-            return LineView(None, None, None, 0, PAGE, self.lengths_dev, st, writes, index=line)
+            return LineView(None, None, None, 0, PAGE, self.lengths_dev, st, writes, index=line, block_state=bst)
         gi, li = self._line_group[line]
         g = self.groups[gi]
-        return LineView(g.k[li], g.v[li], g.table_dev, g.ring, PAGE, self.lengths_dev, st, writes, g.need.values, index=line)
+        return LineView(g.k[li], g.v[li], g.table_dev, g.ring, PAGE, self.lengths_dev, st, writes, g.need.values, index=line,
+                        block_state=bst)
 
     def bytes(self) -> int:
-        return sum(g.bytes() for g in self.groups) + sum(t.numel() * t.element_size() for t in self.state.values())
+        return sum(g.bytes() for g in self.groups) + sum(t.numel() * t.element_size() for t in self._all_states())
 
     def bytes_read_per_step(self, slots: Sequence[int]) -> int:
         """Bytes of keys and values that one decode step of these sequences has to read."""

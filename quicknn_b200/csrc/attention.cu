@@ -345,13 +345,14 @@ attn_decode_tiled_kernel(const T* __restrict__ q, size_t q_stride, const T* __re
                                  n_splits, part_o, part_ml);
 }
 
-// out[b, h, :] = sum_s e^{m_s - M} O_s / sum_s e^{m_s - M} l_s.  The block is cut into G groups of hd/4
+// out[b, h, :] = sum_s e^{m_s - M} O_s / (sum_s e^{m_s - M} l_s + e^{sink_h - M}), the last term with sinks only.  The block is cut into G groups of hd/4
 // threads; group g adds up splits g, g + G, g + 2G, ... (four head elements per thread, 16-byte loads that
 // do not wait for one another), and the G partial sums are added in ascending order of g: an order that
 // depends on the number of splits and the head size only.
 template <typename T>
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    T* __restrict__ out, size_t out_stride, int nq, int hd, int n_splits) {
+                                    T* __restrict__ out, size_t out_stride, int nq, int hd, int n_splits,
+                                    const float* __restrict__ sinks) {
     pdl_wait();
     extern __shared__ __align__(16) float comb[];  // [G][hd] partial sums, then [n_splits] weights and 1/sum
     const int lpg = hd / 4, G = max(1, min((int)blockDim.x / lpg, n_splits));
@@ -403,7 +404,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
         if (threadIdx.x == 0) {
             float ll = 0.f;
             for (int s = 0; s < n_splits; ++s) ll += wl[s];   // ascending order
-            coef[n_splits] = ll > 0.f ? 1.f / ll : 0.f;
+            coef[n_splits] = softmax_inverse(mm, ll, sinks != nullptr ? sinks + h : nullptr);
         }
     }
     __syncthreads();
@@ -447,7 +448,7 @@ extern "C" int qnn_attn_decode_mma_split(const void* q, long long q_stride, cons
                                          const int* slots, const int* slot_len, int B, int nq, int nkv, int hd,
                                          float scale, float cap, int window, float* part_o, float* part_ml,
                                          int n_splits, void* out, long long out_stride, int* combined,
-                                         const float* slopes, cudaStream_t st);
+                                         const float* slopes, const float* sinks, cudaStream_t st);
 
 // threads of the combine kernel's block: a group of hd/4 threads for every key range, up to 1024; and the
 // groups that such a block has (see attn_combine_kernel)
@@ -470,7 +471,7 @@ static int decode_launch(const void* q, long long q_stride, const void* k_pool, 
                          const int* page_table, int max_pages, int page_size, int ring, const int* slots,
                          const int* slot_len, int B, int nq, int nkv, int hd, float scale, float cap, int window,
                          float* part_o, float* part_ml, int n_splits, void* out, long long out_stride,
-                         const float* slopes, cudaStream_t st) {
+                         const float* slopes, const float* sinks, cudaStream_t st) {
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     const Geometry geo = geometry<T>(hd, nq / nkv);
     if (!geo.ok) return QNN_ERR_UNSUPPORTED;
@@ -489,7 +490,7 @@ static int decode_launch(const void* q, long long q_stride, const void* k_pool, 
         int combined = 0;
         const int rc = qnn_attn_decode_mma_split(q, q_stride, k_pool, v_pool, page_table, max_pages, page_size, ring,
                                                  slots, slot_len, B, nq, nkv, hd, scale, cap, window, part_o, part_ml,
-                                                 n_splits, out, out_stride, &combined, slopes, st);
+                                                 n_splits, out, out_stride, &combined, slopes, sinks, st);
         if (rc == 0 && combined) return 0;            // merged inside the kernel's clusters
         if (rc == 0) launched = true;
         else if (rc != QNN_ERR_UNSUPPORTED) return rc;
@@ -523,7 +524,7 @@ static int decode_launch(const void* q, long long q_stride, const void* k_pool, 
     if (e != cudaSuccess) return (int)e;
     size_t comb_floats = (size_t)combine_groups(hd, n_splits) * hd;
     if (comb_floats < (size_t)n_splits) comb_floats = (size_t)n_splits;      // the weighted sums pass through it first
-    qnn::launch_pdl(attn_combine_kernel<T>, dim3(B * nq), dim3(combine_threads(hd, n_splits)), (comb_floats + n_splits + 1) * sizeof(float), st, part_o, part_ml, (T*)out, (size_t)out_stride, nq, hd, n_splits);
+    qnn::launch_pdl(attn_combine_kernel<T>, dim3(B * nq), dim3(combine_threads(hd, n_splits)), (comb_floats + n_splits + 1) * sizeof(float), st, part_o, part_ml, (T*)out, (size_t)out_stride, nq, hd, n_splits, sinks);
     QNN_LAUNCH_CHECK();
 }
 
@@ -547,12 +548,12 @@ QNN_API int qnn_attn_decode(const void* q, long long q_stride, int dtype, const 
                             const int* page_table, int max_pages, int page_size, int ring, const int* slots,
                             const int* slot_len, int B, int nq, int nkv, int hd, float scale, float cap, int window,
                             float* part_o, float* part_ml, int n_splits, void* out, long long out_stride,
-                            const float* slopes, cudaStream_t st) {
+                            const float* slopes, const float* sinks, cudaStream_t st) {
     if (B <= 0) return 0;
     if (n_splits < 1 || n_splits > 65535 || B > 65535) return QNN_ERR_ARGUMENT;
     if (dtype == QNN_DT_BF16)
         return decode_launch<bf16>(q, q_stride, k_pool, v_pool, page_table, max_pages, page_size, ring, slots, slot_len,
-                                   B, nq, nkv, hd, scale, cap, window, part_o, part_ml, n_splits, out, out_stride, slopes, st);
+                                   B, nq, nkv, hd, scale, cap, window, part_o, part_ml, n_splits, out, out_stride, slopes, sinks, st);
     return decode_launch<float>(q, q_stride, k_pool, v_pool, page_table, max_pages, page_size, ring, slots, slot_len, B,
-                                nq, nkv, hd, scale, cap, window, part_o, part_ml, n_splits, out, out_stride, slopes, st);
+                                nq, nkv, hd, scale, cap, window, part_o, part_ml, n_splits, out, out_stride, slopes, sinks, st);
 }

@@ -78,13 +78,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&h);
 }
 
-// out[h, d] = sum_r e^{m_r - M} O_r[d] / sum_r e^{m_r - M} l_r over the ranks of the cluster in
+// out[h, d] = sum_r e^{m_r - M} O_r[d] / (sum_r e^{m_r - M} l_r + e^{sink_h - M}), the last term with sinks only, over the ranks of the cluster in
 // ascending order: the sums that the combine kernel forms from the scratch.  `cs` is this CTA's
 // [head][HD + 2] (O, max, sum) in shared memory, at the same address in every CTA of the cluster;
 // every CTA merges a share of the (head, d) pairs.  Kept out of line so that the main loop of the
 // kernel compiles as it does without it.
 template <int HD>
-__device__ __noinline__ void cluster_merge(const float* cs, int S, int heads, bf16* __restrict__ out) {
+__device__ __noinline__ void cluster_merge(const float* cs, int S, int heads, bf16* __restrict__ out,
+                                           const float* __restrict__ sinks) {
     constexpr int ROW = HD + 2;
     cluster_barrier();
     const unsigned rank = cluster_rank();
@@ -110,7 +111,7 @@ __device__ __noinline__ void cluster_merge(const float* cs, int S, int heads, bf
             ll += c * lr[r];
             acc += c * orr[r];
         }
-        const float inv = ll > 0.f ? 1.f / ll : 0.f;
+        const float inv = softmax_inverse(mm, ll, sinks != nullptr ? sinks + hh : nullptr);
         out[(size_t)hh * HD + d] = __float2bfloat16(acc * inv);
     }
     cluster_barrier();                            // nobody leaves while its memory is still read
@@ -123,7 +124,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16* 
                        int page_size, int ring, const int* __restrict__ slots, const int* __restrict__ slot_len,
                        int nq, int nkv, float scale, float cap, int window, float* __restrict__ part_o,
                        float* __restrict__ part_ml, int n_splits, bf16* __restrict__ out, size_t out_stride,
-                       const float* __restrict__ slopes) {
+                       const float* __restrict__ slopes, const float* __restrict__ sinks) {
     const bool CLUSTER = out != nullptr;         // launched as clusters of n_splits CTAs that merge their ranges
     constexpr int KSTEPS = HD / 16;              // k16 steps of S^T, and 16-row tiles of O^T
     constexpr int CH = HD / 8;                   // 16-byte chunks per row
@@ -354,7 +355,8 @@ attn_decode_mma_kernel(const bf16* __restrict__ q, size_t q_stride, const bf16* 
         }
     }
     if (CLUSTER)
-        cluster_merge<HD>(cs, n_splits, min(8, G - h0), out + (size_t)b * out_stride + (size_t)(kh * G + h0) * HD);
+        cluster_merge<HD>(cs, n_splits, min(8, G - h0), out + (size_t)b * out_stride + (size_t)(kh * G + h0) * HD,
+                          sinks != nullptr ? sinks + kh * G + h0 : nullptr);
 }
 
 // Largest cluster that merges in the kernel.  Clusters of 8 CTAs with 98 KB of shared memory each
@@ -442,7 +444,7 @@ template <int HD, int MMA_WARPS>
 int launch(const void* q, long long q_stride, const void* k_pool, const void* v_pool, const int* page_table,
            int max_pages, int page_size, int ring, const int* slots, const int* slot_len, int B, int nq, int nkv,
            float scale, float cap, int window, float* part_o, float* part_ml, int n_splits, void* out,
-           long long out_stride, int* combined, const float* slopes, cudaStream_t st) {
+           long long out_stride, int* combined, const float* slopes, const float* sinks, cudaStream_t st) {
     const size_t smem = smem_bytes<HD, MMA_WARPS, false>(max_pages);
     const size_t smem_c = smem_bytes<HD, MMA_WARPS, true>(max_pages);
     if (smem > 220 * 1024 || smem_c > 220 * 1024) return QNN_ERR_UNSUPPORTED;
@@ -479,14 +481,14 @@ int launch(const void* q, long long q_stride, const void* k_pool, const void* v_
         cudaError_t e = cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<HD, MMA_WARPS, STC>, (const bf16*)q,
                                            (size_t)q_stride, (const bf16*)k_pool, (const bf16*)v_pool, page_table,
                                            max_pages, page_size, ring, slots, slot_len, nq, nkv, scale, cap, window,
-                                           part_o, part_ml, n_splits, (bf16*)out, (size_t)out_stride, slopes);
+                                           part_o, part_ml, n_splits, (bf16*)out, (size_t)out_stride, slopes, sinks);
         if (e != cudaSuccess) return (int)e;
         *combined = 1;
         return (int)cudaGetLastError();
     }
     qnn::launch_pdl(attn_decode_mma_kernel<HD, MMA_WARPS, ST>, dim3(grid), dim3(MMA_WARPS * 32), smem, st, (const bf16*)q, (size_t)q_stride, (const bf16*)k_pool, (const bf16*)v_pool,
                                              page_table, max_pages, page_size, ring, slots, slot_len, nq, nkv, scale,
-                                             cap, window, part_o, part_ml, n_splits, (bf16*)nullptr, (size_t)0, slopes);
+                                             cap, window, part_o, part_ml, n_splits, (bf16*)nullptr, (size_t)0, slopes, sinks);
     return (int)cudaGetLastError();
 }
 
@@ -504,13 +506,13 @@ extern "C" int qnn_attn_decode_mma_split(const void* q, long long q_stride, cons
                                          const int* slots, const int* slot_len, int B, int nq, int nkv, int hd,
                                          float scale, float cap, int window, float* part_o, float* part_ml,
                                          int n_splits, void* out, long long out_stride, int* combined,
-                                         const float* slopes, cudaStream_t st) {
+                                         const float* slopes, const float* sinks, cudaStream_t st) {
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     if (page_size < TILE || (page_size & (page_size - 1))) return QNN_ERR_UNSUPPORTED;
     if (ring > 0 && (ring % page_size)) return QNN_ERR_UNSUPPORTED;
     if ((q_stride * 2) % 4 || ((uintptr_t)q & 3)) return QNN_ERR_UNSUPPORTED;
 #define QNN_MMA_ARGS q, q_stride, k_pool, v_pool, page_table, max_pages, page_size, ring, slots, slot_len, B, nq, nkv, \
-                     scale, cap, window, part_o, part_ml, n_splits, out, out_stride, combined, slopes, st
+                     scale, cap, window, part_o, part_ml, n_splits, out, out_stride, combined, slopes, sinks, st
     static int warps = 0;
     if (warps == 0) {
         const char* e = getenv("QNN_MMA_WARPS");

@@ -57,7 +57,7 @@ __global__ void __launch_bounds__(PF_WARPS * 32, (BM + 4 * BN) * HD * 2 <= 112 *
 attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v,
                         size_t row_stride, bf16* __restrict__ out, size_t out_stride,
                         const int* __restrict__ seq_row0, const int* __restrict__ seq_len, int nq, int nkv, float scale,
-                        float cap, int window, const float* __restrict__ slopes) {
+                        float cap, int window, const float* __restrict__ slopes, const float* __restrict__ sinks) {
     pdl_wait();
     constexpr int KSTEPS = HD / 16, CH = HD / 8, ROWB = HD * 2, NDT = HD / 8;
     constexpr int TILEB = BN * ROWB;
@@ -219,7 +219,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, 
     for (int r = 0; r < 2; ++r) {
         const int row = qrow_lo + r * 8;
         if (row < len) {
-            const float inv = l_[r] > 0.f ? 1.f / l_[r] : 0.f;
+            const float inv = softmax_inverse(m_[r], l_[r], sinks != nullptr ? sinks + h : nullptr);
             uint32_t* dst = reinterpret_cast<uint32_t*>(out + (size_t)(row0 + row) * out_stride + (size_t)h * HD);
 #pragma unroll
             for (int nd = 0; nd < NDT; ++nd) dst[nd * 4 + t] = pack_bf16(o[nd][2 * r] * inv, o[nd][2 * r + 1] * inv);
@@ -230,7 +230,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, 
 template <int HD, int BN>
 int launch(const void* q, const void* k, const void* v, long long row_stride, void* out, long long out_stride,
            const int* seq_row0, const int* seq_len, int B, int max_len, int nq, int nkv, float scale, float cap,
-           int window, const float* slopes, cudaStream_t st) {
+           int window, const float* slopes, const float* sinks, cudaStream_t st) {
     auto kern = attn_prefill_mma_kernel<HD, BN>;
     const size_t smem = (size_t)(BM + 4 * BN) * HD * 2;
     static bool configured = false;
@@ -242,7 +242,7 @@ int launch(const void* q, const void* k, const void* v, long long row_stride, vo
     dim3 grid(nq, B, (max_len + BM - 1) / BM);
     qnn::launch_pdl(kern, dim3(grid), dim3(PF_WARPS * 32), smem, st, (const bf16*)q, (const bf16*)k, (const bf16*)v, (size_t)row_stride,
                                             (bf16*)out, (size_t)out_stride, seq_row0, seq_len, nq, nkv, scale, cap,
-                                            window, slopes);
+                                            window, slopes, sinks);
     return (int)cudaGetLastError();
 }
 
@@ -254,7 +254,7 @@ int launch(const void* q, const void* k, const void* v, long long row_stride, vo
 QNN_API int qnn_attn_prefill_mma(const void* q, const void* k, const void* v, long long row_stride, void* out,
                                  long long out_stride, const int* seq_row0, const int* seq_len, int B, int max_len,
                                  int nq, int nkv, int hd, float scale, float cap, int window, const float* slopes,
-                                 cudaStream_t st) {
+                                 const float* sinks, cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return 0;
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     if (B > 65535 || (max_len + BM - 1) / BM > 65535) return QNN_ERR_UNSUPPORTED;
@@ -262,10 +262,10 @@ QNN_API int qnn_attn_prefill_mma(const void* q, const void* k, const void* v, lo
         (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) || ((uintptr_t)out & 3))
         return QNN_ERR_ARGUMENT;
     switch (hd) {
-        case 64: return launch<64, 64>(q, k, v, row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, st);
-        case 128: return launch<128, 64>(q, k, v, row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, st);
+        case 64: return launch<64, 64>(q, k, v, row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, sinks, st);
+        case 128: return launch<128, 64>(q, k, v, row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, sinks, st);
         case 256: return launch<256, 32>(q, k, v,      // 32-key tiles: 96 KB of shared memory, two CTAs per SM
-                                          row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, st);
+                                          row_stride, out, out_stride, seq_row0, seq_len, B, max_len, nq, nkv, scale, cap, window, slopes, sinks, st);
         default: return QNN_ERR_UNSUPPORTED;
     }
 }

@@ -127,7 +127,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             bf16* __restrict__ out, size_t out_stride, const int* __restrict__ seq_row0,
                             const int* __restrict__ seq_len, const int* __restrict__ seq_q0, int nq, int nkv,
                             float scale, float cap, int window, int* __restrict__ status, int split_levels,
-                            const float* __restrict__ slopes) {
+                            const float* __restrict__ slopes, const float* __restrict__ sinks) {
     constexpr int KS = k_stages(HD), VS = v_stages(HD);
     constexpr int Q_BYTES = BM * HD * 2;                             // HD / 64 blocks of [128 x 64]
     constexpr int KP_BYTES = 2 * BN * HD * 2;                        // a pair of key tiles: HD / 64 blocks of [128 x 64]
@@ -607,8 +607,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const float mm = fmaxf(have0 ? m_used : -CUDART_INF_F, have1 ? m_other : -CUDART_INF_F);
             const float w0 = have0 ? exp2_fast((m_used - mm) * k2) : 0.f;
             const float w1 = have1 ? exp2_fast((m_other - mm) * k2) : 0.f;
+            // a head's sink joins the denominator once, against the same reference (k2 holds log2(e))
             const float l_row = l_sum * w0 + l_other * w1;
-            const float inv = l_row > 0.f ? 1.f / l_row : 0.f;
+            const float l_all = sinks != nullptr ? l_row + exp2_fast(sinks[h] * LOG2E - mm * k2) : l_row;
+            const float inv = l_row > 0.f ? 1.f / l_all : 0.f;
             const float f0 = w0 * inv, f1 = w1 * inv;
             unsigned char* orow = sOut + rloc * (HD * 2);
             const unsigned char* prow = sK + rloc * (HD * 4);
@@ -673,7 +675,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 template <int HD, bool FIXED>
 int launch_attn(const void* qkv, long long total_rows, void* out, long long out_stride, const int* seq_row0,
                 const int* seq_len, const int* seq_q0, int B, int max_len, int nq, int nkv, float scale, float cap,
-                int window, int* status, const float* slopes, cudaStream_t st) {
+                int window, int* status, const float* slopes, const float* sinks, cudaStream_t st) {
     const long long width = (long long)(nq + 2 * nkv) * HD;
     CUtensorMap map_q, map_kv;
     int rc = make_map(&map_q, qkv, total_rows, width, BM);
@@ -746,7 +748,7 @@ int launch_attn(const void* qkv, long long total_rows, void* out, long long out_
         cfg.numAttrs = pdl ? 1 : 0;
     }
     cudaError_t e = cudaLaunchKernelEx(&cfg, kern, map_q, map_kv, (bf16*)out, (size_t)out_stride, seq_row0, seq_len, seq_q0, nq,
-                                       nkv, scale, cap, window, status, split, slopes);
+                                       nkv, scale, cap, window, status, split, slopes, sinks);
     return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
@@ -763,13 +765,13 @@ int launch_attn(const void* qkv, long long total_rows, void* out, long long out_
 QNN_API int qnn_attn_prefill_tcgen05(const void* qkv, long long total_rows, void* out, long long out_stride,
                                      const int* seq_row0, const int* seq_len, const int* seq_q0, int B, int max_len,
                                      int nq, int nkv, int hd, float scale, float cap, int window, int* status,
-                                     const float* slopes, cudaStream_t st) {
+                                     const float* slopes, const float* sinks, cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return 0;
     if (hd != 64 && hd != 128 && hd != 256) return QNN_ERR_UNSUPPORTED;
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     if (B > 65535 || nq > 32767 || (max_len + BM - 1) / BM > 65535) return QNN_ERR_UNSUPPORTED;
     if (((uintptr_t)qkv & 15) || ((uintptr_t)out & 15) || (out_stride * 2) % 16) return QNN_ERR_UNSUPPORTED;
-#define QNN_ATTN_ARGS qkv, total_rows, out, out_stride, seq_row0, seq_len, seq_q0, B, max_len, nq, nkv, scale, cap, window, status, slopes, st
+#define QNN_ATTN_ARGS qkv, total_rows, out, out_stride, seq_row0, seq_len, seq_q0, B, max_len, nq, nkv, scale, cap, window, status, slopes, sinks, st
     // With a softcap up to 70 the exponent cap * log2(e) stays below 101, so that neither exp(score) nor a row's
     // sum over a million keys leaves float32: the fixed-reference softmax with both groups of warps.  QNN_ATTN_FIXED=0
     // keeps the running maximum (for comparisons).

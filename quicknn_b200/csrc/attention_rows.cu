@@ -13,14 +13,15 @@ constexpr int PRE_WARPS = 4;
 // the head tile.
 template <typename T, int CPL, int GT>
 __device__ __forceinline__ void store_rows(T* __restrict__ out_row, int kh, int G, int gt0, int hd, int LPT, int chunks,
-                                           const float (&l)[GT], const float (&o)[GT][CPL][Vec16<T>::N]) {
+                                           const float* __restrict__ sinks, const float (&m)[GT], const float (&l)[GT],
+                                           const float (&o)[GT][CPL][Vec16<T>::N]) {
     constexpr int VEC = Vec16<T>::N;
     const int lane = threadIdx.x & 31, sl = lane % LPT, ti = lane / LPT;
     if (ti != 0) return;
 #pragma unroll
     for (int g = 0; g < GT; ++g) {
         if (gt0 + g >= G) continue;
-        const float inv = l[g] > 0.f ? 1.f / l[g] : 0.f;
+        const float inv = softmax_inverse(m[g], l[g], sinks != nullptr ? sinks + kh * G + gt0 + g : nullptr);
         T* dst = out_row + (size_t)(kh * G + gt0 + g) * hd;
 #pragma unroll
         for (int i = 0; i < CPL; ++i) {
@@ -46,7 +47,8 @@ attn_prefill_generic_kernel(const T* __restrict__ q, size_t q_stride, const T* _
                             size_t row_stride, T* __restrict__ out, size_t out_stride, const int* __restrict__ tok_pos,
                             const int* __restrict__ tok_row0, int n_tokens, int nq, int nkv, int hd, int LPT,
                             float scale, float cap, int window, const int* __restrict__ page_table, int max_pages,
-                            int page_size, int ring, const float* __restrict__ slopes) {
+                            int page_size, int ring, const float* __restrict__ slopes,
+                            const float* __restrict__ sinks) {
     pdl_wait();
     constexpr int VEC = Vec16<T>::N;
     const int warp = threadIdx.x >> 5;
@@ -84,7 +86,7 @@ attn_prefill_generic_kernel(const T* __restrict__ q, size_t q_stride, const T* _
         }
     }
     merge_groups<CPL, GT, VEC>(LPT, m, l, o);
-    store_rows<T, CPL, GT>(out + (size_t)t * out_stride, kh, G, gt0, hd, LPT, chunks, l, o);
+    store_rows<T, CPL, GT>(out + (size_t)t * out_stride, kh, G, gt0, hd, LPT, chunks, sinks, m, l, o);
 }
 
 // A step that continues sequences by several tokens (or starts some and continues others): token t
@@ -102,7 +104,7 @@ attn_extend_generic_kernel(const T* __restrict__ q, size_t q_stride, const T* __
                            const int* __restrict__ tok_row0, const int* __restrict__ tok_slot, int n_tokens, int nq,
                            int nkv, int hd, int LPT, float scale, float cap, int window,
                            const int* __restrict__ page_table, int max_pages, int page_size, int ring,
-                           const float* __restrict__ slopes) {
+                           const float* __restrict__ slopes, const float* __restrict__ sinks) {
     pdl_wait();
     constexpr int VEC = Vec16<T>::N;
     const int warp = threadIdx.x >> 5;
@@ -140,7 +142,7 @@ attn_extend_generic_kernel(const T* __restrict__ q, size_t q_stride, const T* __
         attend_range<T, CPL, GT>(qr, kv, begin > first ? begin : first, end, 0, TPW, LPT, chunks, cap, sl, p, m, l, o);
     }
     merge_groups<CPL, GT, VEC>(LPT, m, l, o);
-    store_rows<T, CPL, GT>(out + (size_t)t * out_stride, kh, G, gt0, hd, LPT, chunks, l, o);
+    store_rows<T, CPL, GT>(out + (size_t)t * out_stride, kh, G, gt0, hd, LPT, chunks, sinks, m, l, o);
 }
 
 }  // namespace
@@ -149,7 +151,8 @@ template <typename T>
 static int prefill_launch(const void* q, long long q_stride, const void* k, const void* v, long long row_stride,
                           void* out, long long out_stride, const int* tok_pos, const int* tok_row0, int n_tokens,
                           int nq, int nkv, int hd, float scale, float cap, int window, const int* page_table,
-                          int max_pages, int page_size, int ring, bool paged, const float* slopes, cudaStream_t st) {
+                          int max_pages, int page_size, int ring, bool paged, const float* slopes, const float* sinks,
+                          cudaStream_t st) {
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     const Geometry geo = geometry<T>(hd, nq / nkv);
     if (!geo.ok) return QNN_ERR_UNSUPPORTED;
@@ -163,12 +166,12 @@ static int prefill_launch(const void* q, long long q_stride, const void* k, cons
             qnn::launch_pdl(attn_prefill_generic_kernel<T, CPL, GT, true>, dim3(grid), dim3(PRE_WARPS * 32), 0, st, 
                 (const T*)q, (size_t)q_stride, (const T*)k, (const T*)v, (size_t)row_stride, (T*)out,
                 (size_t)out_stride, tok_pos, tok_row0, n_tokens, nq, nkv, hd, geo.lpt, scale, cap, window, page_table,
-                max_pages, page_size, ring, slopes);
+                max_pages, page_size, ring, slopes, sinks);
         else
             qnn::launch_pdl(attn_prefill_generic_kernel<T, CPL, GT, false>, dim3(grid), dim3(PRE_WARPS * 32), 0, st, 
                 (const T*)q, (size_t)q_stride, (const T*)k, (const T*)v, (size_t)row_stride, (T*)out,
                 (size_t)out_stride, tok_pos, tok_row0, n_tokens, nq, nkv, hd, geo.lpt, scale, cap, window, page_table,
-                max_pages, page_size, ring, slopes);
+                max_pages, page_size, ring, slopes, sinks);
     })
     QNN_LAUNCH_CHECK();
 }
@@ -178,13 +181,13 @@ static int prefill_launch(const void* q, long long q_stride, const void* k, cons
 QNN_API int qnn_attn_prefill_generic(const void* q, const void* k, const void* v, long long row_stride, int dtype,
                                      void* out, long long out_stride, const int* tok_pos, const int* tok_row0,
                                      int n_tokens, int nq, int nkv, int hd, float scale, float cap, int window,
-                                     const float* slopes, cudaStream_t st) {
+                                     const float* slopes, const float* sinks, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     if (dtype == QNN_DT_BF16)
         return prefill_launch<bf16>(q, row_stride, k, v, row_stride, out, out_stride, tok_pos, tok_row0, n_tokens, nq,
-                                    nkv, hd, scale, cap, window, nullptr, 0, 1, 0, false, slopes, st);
+                                    nkv, hd, scale, cap, window, nullptr, 0, 1, 0, false, slopes, sinks, st);
     return prefill_launch<float>(q, row_stride, k, v, row_stride, out, out_stride, tok_pos, tok_row0, n_tokens, nq, nkv,
-                                 hd, scale, cap, window, nullptr, 0, 1, 0, false, slopes, st);
+                                 hd, scale, cap, window, nullptr, 0, 1, 0, false, slopes, sinks, st);
 }
 
 // Cached keys before this step's tokens, this step's own rows from there on (see
@@ -194,7 +197,7 @@ static int extend_launch(const void* q, const void* k, const void* v, long long 
                          const void* v_pool, const int* page_table, int max_pages, int page_size, int ring, void* out,
                          long long out_stride, const int* tok_pos, const int* tok_row0, const int* tok_slot, int n_tokens,
                          int nq, int nkv, int hd, float scale, float cap, int window, const float* slopes,
-                         cudaStream_t st) {
+                         const float* sinks, cudaStream_t st) {
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     const Geometry geo = geometry<T>(hd, nq / nkv);
     if (!geo.ok) return QNN_ERR_UNSUPPORTED;
@@ -207,7 +210,7 @@ static int extend_launch(const void* q, const void* k, const void* v, long long 
         qnn::launch_pdl(attn_extend_generic_kernel<T, CPL, GT>, dim3(grid), dim3(PRE_WARPS * 32), 0, st, (const T*)q,
                         (size_t)row_stride, (const T*)k, (const T*)v, (size_t)row_stride, (const T*)k_pool,
                         (const T*)v_pool, (T*)out, (size_t)out_stride, tok_pos, tok_row0, tok_slot, n_tokens, nq, nkv, hd,
-                        geo.lpt, scale, cap, window, page_table, max_pages, page_size, ring, slopes);
+                        geo.lpt, scale, cap, window, page_table, max_pages, page_size, ring, slopes, sinks);
     })
     QNN_LAUNCH_CHECK();
 }
@@ -216,13 +219,13 @@ QNN_API int qnn_attn_extend(const void* q, const void* k, const void* v, long lo
                             const void* k_pool, const void* v_pool, const int* page_table, int max_pages, int page_size,
                             int ring, void* out, long long out_stride, const int* tok_pos, const int* tok_row0,
                             const int* tok_slot, int n_tokens, int nq, int nkv, int hd, float scale, float cap,
-                            int window, const float* slopes, cudaStream_t st) {
+                            int window, const float* slopes, const float* sinks, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     if (dtype == QNN_DT_BF16)
         return extend_launch<bf16>(q, k, v, row_stride, k_pool, v_pool, page_table, max_pages, page_size, ring, out,
-                                   out_stride, tok_pos, tok_row0, tok_slot, n_tokens, nq, nkv, hd, scale, cap, window, slopes, st);
+                                   out_stride, tok_pos, tok_row0, tok_slot, n_tokens, nq, nkv, hd, scale, cap, window, slopes, sinks, st);
     return extend_launch<float>(q, k, v, row_stride, k_pool, v_pool, page_table, max_pages, page_size, ring, out,
-                                out_stride, tok_pos, tok_row0, tok_slot, n_tokens, nq, nkv, hd, scale, cap, window, slopes, st);
+                                out_stride, tok_pos, tok_row0, tok_slot, n_tokens, nq, nkv, hd, scale, cap, window, slopes, sinks, st);
 }
 
 // Several query rows per sequence against the paged cache: token t of the sequence in slot
@@ -232,13 +235,13 @@ QNN_API int qnn_attn_prefill_paged(const void* q, long long q_stride, int dtype,
                                    const int* page_table, int max_pages, int page_size, int ring, void* out,
                                    long long out_stride, const int* tok_pos, const int* tok_slot, int n_tokens, int nq,
                                    int nkv, int hd, float scale, float cap, int window, const float* slopes,
-                                   cudaStream_t st) {
+                                   const float* sinks, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     if (dtype == QNN_DT_BF16)
         return prefill_launch<bf16>(q, q_stride, k_pool, v_pool, 0, out, out_stride, tok_pos, tok_slot, n_tokens, nq,
-                                    nkv, hd, scale, cap, window, page_table, max_pages, page_size, ring, true, slopes, st);
+                                    nkv, hd, scale, cap, window, page_table, max_pages, page_size, ring, true, slopes, sinks, st);
     return prefill_launch<float>(q, q_stride, k_pool, v_pool, 0, out, out_stride, tok_pos, tok_slot, n_tokens, nq, nkv,
-                                 hd, scale, cap, window, page_table, max_pages, page_size, ring, true, slopes, st);
+                                 hd, scale, cap, window, page_table, max_pages, page_size, ring, true, slopes, sinks, st);
 }
 
 // ---------------------------------------------------------------------------------

@@ -131,6 +131,14 @@ __device__ __forceinline__ float softcap(float x, float cap) {
     return x;
 }
 
+// What an unnormalised softmax row is multiplied by: 1 / (sum of exp(score - m)), 0 for a row without keys.  `sink`
+// (null: none) points at a learned number of the row's head that joins the denominator as exp(sink): it has no key and no
+// value and counts once.  Where it is so much larger than every score that exp(sink - m) overflows, the factor is 0.
+__device__ __forceinline__ float softmax_inverse(float m, float l, const float* sink) {
+    if (!(l > 0.f)) return 0.f;
+    return 1.f / (sink != nullptr ? l + expf(*sink - m) : l);
+}
+
 __device__ __forceinline__ float gelu_tanh(float x) {
     return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }

@@ -1,0 +1,140 @@
+// The real-gated linear recurrence (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for Efficient
+// Language Models"): one number of state per channel.
+//
+//   r = sigmoid(zr + br),  i = sigmoid(zi + bi),  log a = -decay * r,  a = exp(log a)
+//   S_t = a S_(t-1) + sqrt(1 - a^2) i u_t            out = scale * S_t * gelu(y_t + by)
+//
+// `decay` (one positive number per channel) is formed when the model is loaded.  Everything from the gates' logits to the
+// state is float32; 1 - a^2 is formed as -expm1(2 log a), which keeps its digits where a is near 1.
+//
+// A thread walks one channel of one sequence.  Sequences of more than one segment are walked in segments side by side, since
+// the recurrence is linear in S: a first kernel leaves (log a, the added term) in the place of the gates' logits and, per
+// segment, the sum of log a and the state that the segment reaches from 0 (the first segment: from the sequence's state); a
+// second kernel forms every segment's starting state from those in order and walks it again with the output.  The last
+// segment's thread leaves the state.
+#include "common.cuh"
+
+using namespace qnn;
+
+namespace {
+
+constexpr int THREADS = 128;
+
+struct Rec {
+    float* z;                   // logits [rows][ldz]: channel c of block b = c / part: columns 2 b part + (c - b part), + part for i
+    const void* rb;             // biases [C]
+    const void* ib;
+    const float* decay;         // [C]
+    const void* u;              // rows of pitch ldu
+    const void* y;              // rows of pitch ldy, may be null (no output gate): out = scale * S
+    const void* yb;             // [C] or null
+    void* out;                  // rows of pitch ldo
+    float* state;               // slot s: state + s * slot_stride, [C]
+    float* scratch;             // [sequences][segments][3][C]: sum of log a, state reached, (segment 0:) state it began with
+    const int* seq_row0;
+    const int* seq_len;
+    const int* slots;
+    long long ldz, ldu, ldy, ldo, slot_stride;
+    int b_dt, u_dt, y_dt, yb_dt, out_dt, C, part, seg, nseg;
+    float scale;
+};
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// (log a, what is added to the state) of row t, channel c
+__device__ __forceinline__ float2 gates(float zr, float zi, float br, float bi, float decay, float u) {
+    const float la = -decay * sigmoid_f(zr + br);
+    return make_float2(la, sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + bi) * u);
+}
+
+template <bool AGGREGATE>       // true: the first of the two kernels; false with nseg > 1: the second; nseg 1: the only one
+__global__ void __launch_bounds__(THREADS) recurrence_kernel(const Rec p) {
+    pdl_wait();
+    const int c = blockIdx.x * THREADS + threadIdx.x;
+    if (c >= p.C) return;
+    const int b = blockIdx.z, sg = blockIdx.y;
+    const int row0 = p.seq_row0 != nullptr ? p.seq_row0[b] : b;
+    const int n = p.seq_len != nullptr ? p.seq_len[b] : 1;
+    const int slot = p.slots[b];
+    const int r0 = sg * p.seg, r1 = min(r0 + p.seg, n);
+    if (r0 >= n) return;
+    if (slot < 0) {
+        if (!AGGREGATE)
+            for (int r = r0; r < r1; ++r) store_from_f(p.out, p.out_dt, (size_t)(row0 + r) * p.ldo + c, 0.f);
+        return;
+    }
+    const int blk = c / p.part;
+    const size_t zc = (size_t)blk * 2 * p.part + (c - blk * p.part);
+    float* state = p.state + (size_t)slot * p.slot_stride + c;
+    const float br = load_as_f(p.rb, p.b_dt, c), bi = load_as_f(p.ib, p.b_dt, c), decay = p.decay[c];
+    if (AGGREGATE) {
+        float* sc = p.scratch + ((size_t)b * p.nseg + sg) * 3 * p.C + c;
+        float S = 0.f, sum = 0.f;
+        if (sg == 0) {
+            S = *state;
+            sc[2 * (size_t)p.C] = S;
+        }
+#pragma unroll 4
+        for (int r = r0; r < r1; ++r) {
+            float* z = p.z + (size_t)(row0 + r) * p.ldz + zc;
+            const float2 ab = gates(z[0], z[p.part], br, bi, decay, load_as_f(p.u, p.u_dt, (size_t)(row0 + r) * p.ldu + c));
+            z[0] = ab.x;
+            z[p.part] = ab.y;
+            sum += ab.x;
+            S = fmaf(expf(ab.x), S, ab.y);
+        }
+        sc[0] = sum;
+        sc[p.C] = S;
+        return;
+    }
+    const bool whole = p.nseg == 1;
+    float S;
+    if (whole) {
+        S = *state;
+    } else {
+        const float* sc = p.scratch + (size_t)b * p.nseg * 3 * p.C + c;
+        S = sc[2 * (size_t)p.C];
+        for (int k = 0; k < sg; ++k, sc += 3 * (size_t)p.C)
+            S = k == 0 ? sc[p.C] : fmaf(expf(sc[0]), S, sc[p.C]);
+    }
+    const float yb = p.yb != nullptr ? load_as_f(p.yb, p.yb_dt, c) : 0.f;
+#pragma unroll 4
+    for (int r = r0; r < r1; ++r) {
+        const size_t row = (size_t)(row0 + r);
+        const float* z = p.z + row * p.ldz + zc;
+        float2 ab = make_float2(z[0], z[p.part]);
+        if (whole) ab = gates(ab.x, ab.y, br, bi, decay, load_as_f(p.u, p.u_dt, row * p.ldu + c));
+        S = fmaf(expf(ab.x), S, ab.y);
+        const float gate = p.y != nullptr ? gelu_tanh(load_as_f(p.y, p.y_dt, row * p.ldy + c) + yb) : 1.f;
+        store_from_f(p.out, p.out_dt, row * p.ldo + c, p.scale * S * gate);
+    }
+    if (r1 == n) *state = S;
+}
+
+}  // namespace
+
+// seq_row0, seq_len both null: a row per sequence.  `longest`: the most rows that one sequence brings.  With nseg > 1
+// (segments of `seg` rows) z is overwritten and scratch holds n_seqs * nseg * 3 * C floats.
+QNN_API int qnn_linear_recurrence(float* z, long long ldz, const void* rb, const void* ib, int b_dt, const float* decay,
+                                  const void* u, int u_dt, long long ldu, const void* y, int y_dt, long long ldy,
+                                  const void* yb, int yb_dt, float scale, void* out, int out_dt, long long ldo, float* state,
+                                  long long slot_stride, const int* seq_row0, const int* seq_len, const int* slots, int n_seqs,
+                                  int C, int part, int seg, int nseg, float* scratch, cudaStream_t st) {
+    if (n_seqs <= 0) return 0;
+    if (C <= 0 || part <= 0 || C % part || nseg < 1 || seg < 1 || n_seqs > 65535 || nseg > 65535 || ldz < 2LL * C ||
+        ldu < C || ldo < C || (y != nullptr && ldy < C) || slot_stride < C || (nseg > 1 && (scratch == nullptr || seq_row0 == nullptr)))
+        return QNN_ERR_ARGUMENT;
+    Rec p;
+    p.z = z; p.rb = rb; p.ib = ib; p.decay = decay; p.u = u; p.y = y; p.yb = yb; p.out = out; p.state = state;
+    p.scratch = scratch; p.seq_row0 = seq_row0; p.seq_len = seq_len; p.slots = slots; p.ldz = ldz; p.ldu = ldu; p.ldy = ldy;
+    p.ldo = ldo; p.slot_stride = slot_stride; p.b_dt = b_dt; p.u_dt = u_dt; p.y_dt = y_dt; p.yb_dt = yb_dt; p.out_dt = out_dt;
+    p.C = C; p.part = part; p.seg = seg; p.nseg = nseg; p.scale = scale;
+    const dim3 grid((C + THREADS - 1) / THREADS, nseg, n_seqs);
+    if (nseg > 1) {
+        launch_pdl(recurrence_kernel<true>, grid, dim3(THREADS), 0, st, p);
+        const cudaError_t e = cudaGetLastError();
+        if (e != cudaSuccess) return (int)e;
+    }
+    launch_pdl(recurrence_kernel<false>, grid, dim3(THREADS), 0, st, p);
+    QNN_LAUNCH_CHECK();
+}

@@ -123,17 +123,18 @@ small_linear_thread_kernel(const TX* __restrict__ x, const TW* __restrict__ w, f
     out[(size_t)(t0 + r) * N + n0 + c] = finish(d, bias, bias_dt, inv_tau, n0 + c);
 }
 
-// o[t, h, :] *= sigmoid(x[t, :] . w[h, :]): the gate per head formed (float32) and applied in one kernel; a block per
-// row, the warps share the heads.  A lane's terms and the order of their sum depend on the width only.
+// out[t, h, :] = o[t, h, :] * scale * sigmoid(x[t, :] . w[h, :]) (out may be o): the gate per head formed (float32) and
+// applied in one kernel; a block per row, the warps share the heads.  A lane's terms and the order of their sum depend on
+// the width only.
 template <typename TX, typename TW>
-__global__ void gate_heads_kernel(const TX* __restrict__ x, const TW* __restrict__ w, int W, void* __restrict__ o, int o_dt,
-                                  int H, int D) {
+__global__ void gate_heads_kernel(const TX* __restrict__ x, long long ldx, const TW* __restrict__ w, int W, const void* o, int o_dt,
+                                  void* out, long long ldo, float scale, int H, int D) {
     extern __shared__ float gate[];                       // [H]
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
-    const TX* xr = x + (size_t)blockIdx.x * W;
+    const TX* xr = x + (size_t)blockIdx.x * ldx;
     constexpr int VX = Vec16<TX>::N, VW = Vec16<TW>::N, V = VX > VW ? VX : VW;
-    const bool vec = (W % V) == 0 && ((((uintptr_t)x | (uintptr_t)w) & 15) == 0);
+    const bool vec = (W % V) == 0 && (ldx % V) == 0 && ((((uintptr_t)x | (uintptr_t)w) & 15) == 0);
     for (int h = warp; h < H; h += nwarp) {
         const TW* wr = w + (size_t)h * W;
         float d = 0.f;
@@ -151,12 +152,24 @@ __global__ void gate_heads_kernel(const TX* __restrict__ x, const TW* __restrict
             for (int i = lane; i < W; i += 32) d += to_f(xr[i]) * to_f(wr[i]);
         }
         d = warp_sum(d);
-        if (lane == 0) gate[h] = 1.f / (1.f + expf(-d));
+        if (lane == 0) gate[h] = scale * (1.f / (1.f + expf(-d)));
     }
     __syncthreads();
-    const size_t base = (size_t)blockIdx.x * H * D;
+    const size_t base = (size_t)blockIdx.x * H * D, ob = (size_t)blockIdx.x * ldo;
+    const size_t es = o_dt == QNN_DT_BF16 ? 2 : 4;
+    if (D % 8 == 0 && (ldo * es) % 16 == 0 && (((uintptr_t)o | (uintptr_t)out) & 15) == 0) {
+        for (int i = threadIdx.x * 8; i < H * D; i += blockDim.x * 8) {
+            float v[8];
+            load8_as_f(o, o_dt, base + i, v);
+            const float g = gate[i / D];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] *= g;
+            store8_from_f(out, o_dt, ob + i, v);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < H * D; i += blockDim.x)
-        store_from_f(o, o_dt, base + i, load_as_f(o, o_dt, base + i) * gate[i / D]);
+        store_from_f(out, o_dt, ob + i, load_as_f(o, o_dt, base + i) * gate[i / D]);
 }
 
 inline int row_threads(int n) { return n >= 2048 ? 512 : (n >= 512 ? 256 : 128); }
@@ -218,13 +231,14 @@ QNN_API int qnn_small_linear_f32(const void* x, int x_dt, const void* w, int w_d
     QNN_LAUNCH_CHECK();
 }
 
-QNN_API int qnn_gate_heads(const void* x, int x_dt, const void* w, int w_dt, int W, void* o, int o_dt, int T, int H, int D,
-                           cudaStream_t st) {
+// x: rows of pitch ldx; o: dense rows [T, H * D]; out: rows of pitch ldo in o's element type (o itself with ldo = H * D).
+QNN_API int qnn_gate_heads(const void* x, int x_dt, long long ldx, const void* w, int w_dt, int W, const void* o, int o_dt,
+                           void* out, long long ldo, float scale, int T, int H, int D, cudaStream_t st) {
     if (T <= 0) return 0;
-    if (W <= 0 || H <= 0 || D <= 0 || (size_t)H * sizeof(float) > 48 * 1024) return QNN_ERR_ARGUMENT;
+    if (W <= 0 || H <= 0 || D <= 0 || ldx < W || ldo < (long long)H * D || (size_t)H * sizeof(float) > 48 * 1024) return QNN_ERR_ARGUMENT;
     const dim3 grid(T), block(row_threads(H * D));
     const size_t smem = (size_t)H * sizeof(float);
-#define QNN_GH(TX, TW) launch_pdl(gate_heads_kernel<TX, TW>, grid, block, smem, st, (const TX*)x, (const TW*)w, W, o, o_dt, H, D)
+#define QNN_GH(TX, TW) launch_pdl(gate_heads_kernel<TX, TW>, grid, block, smem, st, (const TX*)x, ldx, (const TW*)w, W, o, o_dt, out, ldo, scale, H, D)
     if (x_dt == QNN_DT_BF16 && w_dt == QNN_DT_BF16) QNN_GH(bf16, bf16);
     else if (x_dt == QNN_DT_BF16) QNN_GH(bf16, float);
     else if (w_dt == QNN_DT_BF16) QNN_GH(float, bf16);

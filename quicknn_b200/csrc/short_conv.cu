@@ -1,0 +1,164 @@
+// Short causal convolutions over time, one filter per channel, with the last inputs of every sequence as state.
+//
+//   qnn_causal_conv   v_t = x_t + x_bias;  out_t = sum_j w[:, j] v_(t - taps + 1 + j) + out_bias (+ v_t with `add_input`)
+//
+// with zeros before a sequence's first position.  A sequence's state is a ring of `taps` rows of C floats: v of position p
+// lies in row p mod taps, so a step of any length leaves the rows that it does not replace where they are, and a decode
+// step writes a row that no tap of the same step reads.  Prompts, continued sequences and single tokens are one kernel: a
+// tap that falls before the step's first row comes from the ring, any other from the step's rows.  Sums are float32 in
+// the order of the taps, so they do not depend on how a sequence was cut into steps.
+//
+// A thread owns VEC channels of `rows` consecutive rows of one sequence.  The threads of a sequence's first tile read the
+// ring (tiles have at least taps - 1 rows) and, after that, write the same channels' new rows into it.
+#include "common.cuh"
+
+using namespace qnn;
+
+namespace {
+
+constexpr int THREADS = 128;
+
+template <int VEC>
+__device__ __forceinline__ void load_v(const void* p, int dt, size_t i, float* o) {
+    if (VEC == 8) load8_as_f(p, dt, i, o);
+    else o[0] = load_as_f(p, dt, i);
+}
+template <int VEC>
+__device__ __forceinline__ void store_v(void* p, int dt, size_t i, const float* v) {
+    if (VEC == 8) store8_from_f(p, dt, i, v);
+    else store_from_f(p, dt, i, v[0]);
+}
+
+// TAPS > 0: the number of taps is known here and the filter and the last inputs stay in registers; 0: any number, taps are
+// read again for every row.
+template <int VEC, int TAPS>
+__global__ void __launch_bounds__(THREADS)
+causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const void* __restrict__ x_bias, int xb_dt,
+                   const void* __restrict__ w, int w_dt, const void* __restrict__ out_bias, int ob_dt, int add_input,
+                   void* __restrict__ out, int out_dt, long long ldo, float* state, long long slot_stride, int C, int taps_,
+                   const int* __restrict__ seq_row0, const int* __restrict__ seq_len, const int* __restrict__ tok_pos,
+                   const int* __restrict__ slots, int rows) {
+    pdl_wait();
+    const int taps = TAPS > 0 ? TAPS : taps_;
+    const int b = blockIdx.z;
+    const int c0 = (blockIdx.x * THREADS + threadIdx.x) * VEC;
+    if (c0 >= C) return;
+    const int row0 = seq_row0 != nullptr ? seq_row0[b] : b;
+    const int n = seq_len != nullptr ? seq_len[b] : 1;
+    const int r0 = blockIdx.y * rows;                       // first row of this tile within the sequence
+    if (r0 >= n) return;
+    const int r1 = min(r0 + rows, n);
+    const int slot = slots[b];
+    if (slot < 0) {                                         // a row of no sequence
+        float z[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) z[e] = 0.f;
+        for (int r = r0; r < r1; ++r) store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, z);
+        return;
+    }
+    const int first = tok_pos[row0];                        // position of the sequence's first row of this step
+    float* ring = state + (size_t)slot * slot_stride + c0;
+    float xb[VEC], ob[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) xb[e] = ob[e] = 0.f;
+    if (x_bias != nullptr) load_v<VEC>(x_bias, xb_dt, c0, xb);
+    if (out_bias != nullptr) load_v<VEC>(out_bias, ob_dt, c0, ob);
+    // v of row r (may be negative: an earlier step's, or before the sequence)
+    auto input = [&](int r, float* v) {
+        if (r >= 0) {
+            load_v<VEC>(x, x_dt, (size_t)(row0 + r) * ldx + c0, v);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] += xb[e];
+        } else if (first + r >= 0) {
+            const float* cell = ring + (size_t)((first + r) % taps) * C;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] = cell[e];
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) v[e] = 0.f;
+        }
+    };
+    if constexpr (TAPS > 0) {
+        float wv[TAPS][VEC], last[TAPS][VEC];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) wv[j][e] = load_as_f(w, w_dt, (size_t)(c0 + e) * TAPS + j);
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) input(r0 - TAPS + j, last[j]);
+        for (int r = r0; r < r1; ++r) {
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) last[j][e] = last[j + 1][e];
+            input(r, last[TAPS - 1]);
+            float acc[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                acc[e] = 0.f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], last[j][e], acc[e]);
+                acc[e] += ob[e];
+                if (add_input) acc[e] += last[TAPS - 1][e];
+            }
+            store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, acc);
+        }
+    } else {
+        for (int r = r0; r < r1; ++r) {
+            float acc[VEC], v[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = v[e] = 0.f;
+            for (int j = 0; j < taps; ++j) {
+                input(r - taps + 1 + j, v);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) acc[e] = fmaf(load_as_f(w, w_dt, (size_t)(c0 + e) * taps + j), v[e], acc[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] += ob[e] + (add_input ? v[e] : 0.f);
+            store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, acc);
+        }
+    }
+    if (blockIdx.y == 0) {
+        for (int r = max(0, n - taps); r < n; ++r) {
+            float v[VEC];
+            input(r, v);
+            float* cell = ring + (size_t)((first + r) % taps) * C;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) cell[e] = v[e];
+        }
+    }
+}
+
+}  // namespace
+
+// x, out: rows `ldx` / `ldo` elements apart (different buffers).  seq_row0, seq_len (both null: a row per sequence, row b is
+// sequence b's next token): the sequences' rows; the position of a sequence's first row is tok_pos of that row.  state: the
+// ring of slot s lies at state + s * slot_stride floats.
+QNN_API int qnn_causal_conv(const void* x, int x_dt, long long ldx, const void* x_bias, int xb_dt, const void* w, int w_dt,
+                            const void* out_bias, int ob_dt, int add_input, void* out, int out_dt, long long ldo, float* state,
+                            long long slot_stride, int C, int taps, const int* seq_row0, const int* seq_len,
+                            const int* tok_pos, const int* slots, int n_seqs, int longest, cudaStream_t st) {
+    if (n_seqs <= 0 || longest <= 0) return 0;
+    if (C <= 0 || taps < 1 || n_seqs > 65535 || ldx < C || ldo < C || slot_stride < (long long)taps * C) return QNN_ERR_ARGUMENT;
+    const int xs = x_dt == QNN_DT_BF16 ? 2 : 4, os = out_dt == QNN_DT_BF16 ? 2 : 4;
+    const bool vec = C % 8 == 0 && (ldx * xs) % 16 == 0 && (ldo * os) % 16 == 0 &&
+                     (((uintptr_t)x | (uintptr_t)out | (uintptr_t)x_bias | (uintptr_t)out_bias) & 15) == 0;
+    int rows = longest > 1 ? 16 : 1;
+    if (rows < taps) rows = taps;
+    while ((long long)(longest + rows - 1) / rows > 65535) rows *= 2;
+    const int per = THREADS * (vec ? 8 : 1);
+    const dim3 grid((C + per - 1) / per, (longest + rows - 1) / rows, n_seqs);
+#define QNN_CONV(V, TP)                                                                                                \
+    launch_pdl(causal_conv_kernel<V, TP>, grid, dim3(THREADS), 0, st, x, x_dt, ldx, x_bias, xb_dt, w, w_dt, out_bias,   \
+               ob_dt, add_input, out, out_dt, ldo, state, slot_stride, C, taps, seq_row0, seq_len, tok_pos, slots, rows)
+    if (vec) {
+        if (taps == 4) QNN_CONV(8, 4);
+        else if (taps == 3) QNN_CONV(8, 3);
+        else if (taps == 2) QNN_CONV(8, 2);
+        else QNN_CONV(8, 0);
+    } else {
+        QNN_CONV(1, 0);
+    }
+#undef QNN_CONV
+    QNN_LAUNCH_CHECK();
+}

@@ -1,0 +1,167 @@
+// The float32 residual stream of layers that norm what a sublayer gives, scale it, add it, and may then average over depth.
+//
+//   qnn_stream_update   X = resid + mult * rmsnorm(y; w_post);  X -> resid_out
+//                       with a history:  Z = sum_(j < n) a_j X_j + a_n X,  Z -> avg_out   (X_j: rows that earlier layers left)
+//                       out_next = rmsnorm(Z or X; w_next), if asked for
+//
+// One block per row; the row stays in registers between its sums where it fits, eight columns per access where rows allow.
+// Earlier layers' rows are read in the order of the layers and each is used once.  All sums are float32.
+#include "common.cuh"
+
+using namespace qnn;
+
+namespace {
+
+struct Update {
+    const float* resid;
+    const void* y;
+    const void* w_post;
+    const void* w_next;
+    float* resid_out;
+    const float* hist;        // [n_hist][rows][H]; null: no average
+    const void* numbers;      // [n_hist + 1]
+    float* avg_out;
+    void* out_next;
+    long long hist_stride;
+    int y_dt, wp_dt, wn_dt, num_dt, out_dt, n_hist, H;
+    float mult, eps_post, off_post, eps_next, off_next;
+};
+
+template <int CH>
+__global__ void stream_update_vec_kernel(const Update u) {
+    __shared__ float red[32];
+    const size_t base = (size_t)blockIdx.x * u.H;
+    const int nchunks = u.H >> 3;
+    float g1[CH][8], v[CH][8], r[CH][8];
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {                       // weights are written by no kernel of the step
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < nchunks) load8_as_f(u.w_post, u.wp_dt, (size_t)c * 8, g1[i]);
+    }
+    pdl_wait();
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < nchunks) {
+            load8_as_f(u.y, u.y_dt, base + (size_t)c * 8, v[i]);
+            load8_as_f(u.resid, QNN_DT_F32, base + (size_t)c * 8, r[i]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[i][e] = r[i][e] = g1[i][e] = 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += v[i][e] * v[i][e];
+    }
+    ss = block_sum(ss, red);
+    const float inv = rsqrtf(ss / (float)u.H + u.eps_post);
+    float ss2 = 0.f;
+    const float a_last = u.hist != nullptr ? load_as_f(u.numbers, u.num_dt, u.n_hist) : 1.f;
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c >= nchunks) continue;
+        const size_t at = base + (size_t)c * 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) r[i][e] += u.mult * (v[i][e] * inv * (g1[i][e] + u.off_post));
+        store8_from_f(u.resid_out, QNN_DT_F32, at, r[i]);
+        if (u.hist != nullptr) {
+            float z[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z[e] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < u.n_hist; ++j) {
+                float h[8];
+                load8_as_f(u.hist, QNN_DT_F32, (size_t)j * u.hist_stride + at, h);
+                const float a = load_as_f(u.numbers, u.num_dt, j);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) z[e] = fmaf(a, h[e], z[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) r[i][e] = fmaf(a_last, r[i][e], z[e]);
+            store8_from_f(u.avg_out, QNN_DT_F32, at, r[i]);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss2 += r[i][e] * r[i][e];
+    }
+    if (u.out_next == nullptr) return;
+    ss2 = block_sum(ss2, red);
+    const float inv2 = rsqrtf(ss2 / (float)u.H + u.eps_next);
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < nchunks) {
+            float g2[8], o[8];
+            load8_as_f(u.w_next, u.wn_dt, (size_t)c * 8, g2);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (g2[e] + u.off_next);
+            store8_from_f(u.out_next, u.out_dt, base + (size_t)c * 8, o);
+        }
+    }
+}
+
+// Any width: a column at a time, each thread re-reads only what it wrote itself.
+__global__ void stream_update_kernel(const Update u) {
+    __shared__ float red[32];
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * u.H;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < u.H; i += blockDim.x) {
+        const float v = load_as_f(u.y, u.y_dt, base + i);
+        ss += v * v;
+    }
+    ss = block_sum(ss, red);
+    const float inv = rsqrtf(ss / (float)u.H + u.eps_post);
+    float ss2 = 0.f;
+    for (int i = threadIdx.x; i < u.H; i += blockDim.x) {
+        float r = u.resid[base + i] +
+                  u.mult * (load_as_f(u.y, u.y_dt, base + i) * inv * (load_as_f(u.w_post, u.wp_dt, i) + u.off_post));
+        u.resid_out[base + i] = r;
+        if (u.hist != nullptr) {
+            float z = 0.f;
+            for (int j = 0; j < u.n_hist; ++j)
+                z = fmaf(load_as_f(u.numbers, u.num_dt, j), u.hist[(size_t)j * u.hist_stride + base + i], z);
+            r = fmaf(load_as_f(u.numbers, u.num_dt, u.n_hist), r, z);
+            u.avg_out[base + i] = r;
+        }
+        ss2 += r * r;
+    }
+    if (u.out_next == nullptr) return;
+    ss2 = block_sum(ss2, red);
+    const float inv2 = rsqrtf(ss2 / (float)u.H + u.eps_next);
+    const float* from = u.hist != nullptr ? u.avg_out : u.resid_out;
+    for (int i = threadIdx.x; i < u.H; i += blockDim.x)
+        store_from_f(u.out_next, u.out_dt, base + i, from[base + i] * inv2 * (load_as_f(u.w_next, u.wn_dt, i) + u.off_next));
+}
+
+}  // namespace
+
+// resid may be resid_out (in place).  hist (null: no average): rows of n_hist earlier layers, hist_stride floats from one
+// layer's rows to the next's; numbers: n_hist + 1 of them, the last one for X; avg_out may be resid but not resid_out.
+// w_next / out_next null: no norm follows.
+QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, float mult, const void* w_post, int wp_dt,
+                              float eps_post, int unit_post, float* resid_out, const float* hist, long long hist_stride,
+                              int n_hist, const void* numbers, int num_dt, float* avg_out, const void* w_next, int wn_dt,
+                              float eps_next, int unit_next, void* out_next, int out_dt, int T, int H, cudaStream_t st) {
+    if (T <= 0) return 0;
+    if (H <= 0 || (out_next != nullptr && w_next == nullptr)) return QNN_ERR_ARGUMENT;
+    if (hist != nullptr && (n_hist < 0 || numbers == nullptr || avg_out == nullptr || avg_out == resid_out)) return QNN_ERR_ARGUMENT;
+    Update u;
+    u.resid = resid; u.y = y; u.w_post = w_post; u.w_next = w_next; u.resid_out = resid_out; u.hist = hist;
+    u.numbers = numbers; u.avg_out = avg_out; u.out_next = out_next; u.hist_stride = hist_stride;
+    u.y_dt = y_dt; u.wp_dt = wp_dt; u.wn_dt = wn_dt; u.num_dt = num_dt; u.out_dt = out_dt; u.n_hist = n_hist; u.H = H;
+    u.mult = mult; u.eps_post = eps_post; u.off_post = unit_post ? 1.f : 0.f; u.eps_next = eps_next;
+    u.off_next = unit_next ? 1.f : 0.f;
+    const uintptr_t all = (uintptr_t)resid | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)resid_out |
+                          (uintptr_t)hist | (uintptr_t)avg_out | (uintptr_t)out_next;
+    if ((H & 7) == 0 && (all & 15) == 0 && (hist_stride & 3) == 0 && H <= 8 * 2 * 1024) {
+        const int chunks = H >> 3;
+        const int ch = chunks > 1024 ? 2 : 1;
+        const int threads = (((chunks + ch - 1) / ch) + 31) / 32 * 32;
+        if (ch == 1) launch_pdl(stream_update_vec_kernel<1>, dim3(T), dim3(threads), 0, st, u);
+        else launch_pdl(stream_update_vec_kernel<2>, dim3(T), dim3(threads), 0, st, u);
+        QNN_LAUNCH_CHECK();
+    }
+    launch_pdl(stream_update_kernel, dim3(T), dim3(H >= 2048 ? 512 : (H >= 512 ? 256 : 128)), 0, st, u);
+    QNN_LAUNCH_CHECK();
+}

@@ -27,6 +27,15 @@ class WholeSequences:
 
 
 @dataclasses.dataclass
+class DepthHistory:
+    """What the layers of a model that averages over depth leave for the layers after them, for one step."""
+
+    results: torch.Tensor           # [layers + 1, T, width] float32: the embedded rows, then every layer's result
+    stream: torch.Tensor            # [T, width] float32: the average that goes on
+    index: int = 0                  # the executed layer that runs: its result is results[index + 1]
+
+
+@dataclasses.dataclass
 class StepBatch:
     """Device-side description of one step.
 
@@ -76,3 +85,4 @@ class StepBatch:
     # continues sequences appends to a cache line with readers only then, so that the readers still find the ring as
     # earlier steps left it.
     after_layers: List[Any] = dataclasses.field(default_factory=list)
+    depth: Optional[DepthHistory] = None      # set by the model for the length of a forward pass, if it averages over depth

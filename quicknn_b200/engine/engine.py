@@ -47,7 +47,7 @@ class Engine:
         if max_slots is None:
             max_slots = max(1, min(max_tokens // PAGE, 256))
         needs, states = model.cache_needs()
-        self.cache = KVCache(needs, states, max_tokens, max_slots, max_seq, model.dtype, self.device)
+        self.cache = KVCache(needs, states, max_tokens, max_slots, max_seq, model.dtype, self.device, model.block_state_needs())
         self.max_seq, self.max_slots = max_seq, max_slots
         self.tuning: Dict[str, Any] = dict(tuning or {})
         if decode_splits:

@@ -19,7 +19,7 @@ from ..parts.layout import expected_tensors
 from ..parts.linear import project
 from ..parts.spec import ModelSpec
 from ..weights.loader import check_state_dict, load_named_tensors, place
-from .batch import StepBatch
+from .batch import DepthHistory, StepBatch
 
 DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.float32, "fp32": torch.float32}
 
@@ -90,6 +90,15 @@ class Model:
     # ---- what the cache has to provide ------------------------------------------------
     def _check_schedule(self) -> None:
         spec = self.spec
+        if spec.depth_history:
+            if self.positions is not None or self.embedding_norm is not None or any(e.add_embedding for e in spec.schedule):
+                raise ValueError("an average over depth starts from the embedded rows as they are")
+            for i, e in enumerate(spec.schedule):
+                n = getattr(self.blocks[e.layer], "depth_terms", None)
+                if n != i + 2:
+                    raise ValueError(f"executed layer {i} averages over {n} results, there are {i + 2}")
+        elif any(getattr(b, "depth_terms", None) is not None for b in self.blocks):
+            raise ValueError("a layer averages over depth in a model that keeps no history")
         writers: Dict[int, int] = {}
         for e in spec.schedule:
             if not (0 <= e.layer < len(self.blocks)):
@@ -123,6 +132,14 @@ class Model:
                 if mine is not None and kept.window is not None and (mine.window is None or mine.window > kept.window):
                     needs[e.cache] = dataclasses.replace(kept, window=mine.window)
         return needs, states
+
+    def block_state_needs(self) -> List[Optional[StateNeed]]:
+        """The fixed-size states that blocks keep beside their mixers', by cache line."""
+        out: List[Optional[StateNeed]] = [None] * self.spec.n_cache_lines()
+        for e in self.spec.schedule:
+            if e.writes_cache:
+                out[e.cache] = self.blocks[e.layer].state_need()
+        return out
 
     def scratch_need(self, step) -> int:
         """Bytes of scratch that a step of this shape needs: the largest need of the layers that run
@@ -169,6 +186,15 @@ class Model:
             # the normed rows are the stream itself (float32), not a sublayer's input
             x = self.embedding_norm(ops.embed(step.tokens, self.embedding, spec.embedding.scale), torch.float32)
             normed = None
+        elif spec.depth_history:
+            # the embedded rows are the first of the results that later layers average over
+            T, W = step.tokens.numel(), spec.hidden_size
+            results = torch.empty((len(sched) + 1, T, W), dtype=torch.float32, device=step.tokens.device)
+            step.depth = DepthHistory(results, torch.empty((T, W), dtype=torch.float32, device=results.device))
+            if hasattr(first, "of_embedding"):
+                x, normed = first.of_embedding(step.tokens, self.embedding, spec.embedding.scale, step.act_dtype, out=results[0])
+            else:
+                x, normed = ops.embed(step.tokens, self.embedding, spec.embedding.scale, out=results[0]), None
         elif hasattr(first, "of_embedding"):
             # the first layer's first norm in the embedding's kernel; the layer is handed its input normed
             x, normed = first.of_embedding(step.tokens, self.embedding, spec.embedding.scale, step.act_dtype)
@@ -181,6 +207,8 @@ class Model:
             line = cache.line(e.cache, writes=e.writes_cache)
             if line is not None:
                 line.has_readers = e.cache in self._lines_read
+            if step.depth is not None:
+                step.depth.index = i
             if e.add_embedding:
                 first = self.blocks[e.layer].first_norm()
                 if hasattr(first, "add_then"):               # the add and the layer's first norm in one kernel
@@ -198,6 +226,7 @@ class Model:
         for call in step.after_layers:         # appends that waited for the readers of their cache line
             call()
         step.after_layers.clear()
+        step.depth = None
         step.shared_rows.clear()               # what layers handed each other lives no longer than the step
         return self.logits_of_rows(x, None if step.want_every_row else step.want_rows, step.act_dtype, reduce)
 

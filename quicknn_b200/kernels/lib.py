@@ -43,20 +43,20 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_gemm_skinny_tcgen05": [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_float, c_int, c_vp, c_vp],
     "qnn_gemm_skinny_tcgen05_argmax": [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_float, c_vp, c_vp, c_vp],
     "qnn_attn_decode": [c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp, c_int, c_int,
-                        c_int, c_int, c_float, c_float, c_int, c_vp, c_vp, c_int, c_vp, c_ll, c_vp, c_vp],
+                        c_int, c_int, c_float, c_float, c_int, c_vp, c_vp, c_int, c_vp, c_ll, c_vp, c_vp, c_vp],
     "qnn_attn_extend": [c_vp, c_vp, c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_ll, c_vp, c_vp,
-                        c_vp, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_vp, c_vp],
+                        c_vp, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_vp, c_vp, c_vp],
     "qnn_attn_supports": [c_int, c_int, c_int, c_int],
     "qnn_attn_prefill_generic": [c_vp, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_int,
-                                 c_int, c_float, c_float, c_int, c_vp, c_vp],
+                                 c_int, c_float, c_float, c_int, c_vp, c_vp, c_vp],
     "qnn_attn_prefill_mma": [c_vp, c_vp, c_vp, c_ll, c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int,
-                             c_float, c_float, c_int, c_vp, c_vp],
+                             c_float, c_float, c_int, c_vp, c_vp, c_vp],
     "qnn_attn_prefill_tcgen05": [c_vp, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_float,
-                                 c_float, c_int, c_vp, c_vp, c_vp],
+                                 c_float, c_int, c_vp, c_vp, c_vp, c_vp],
     "qnn_attn_extend_gather": [c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_vp],
     "qnn_attn_prefill_paged": [c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_ll, c_vp, c_vp,
-                               c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_vp, c_vp],
+                               c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_vp, c_vp, c_vp],
     "qnn_sample": [c_vp, c_int, c_int, c_int, c_float, c_float, c_float, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp,
                    c_vp, c_vp],
     "qnn_sample_candidates": [c_vp, c_int, c_int, c_int, c_int, c_float, c_float, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp,
@@ -67,7 +67,17 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_rmsnorm_strided": [c_vp, c_int, c_ll, c_vp, c_int, c_float, c_vp, c_int, c_ll, c_vp, c_ll, c_int, c_int, c_vp],
     "qnn_copy_rows": [c_vp, c_int, c_ll, c_vp, c_ll, c_int, c_int, c_vp],
     "qnn_scale_heads": [c_vp, c_int, c_vp, c_int, c_int, c_int, c_vp],
-    "qnn_gate_heads": [c_vp, c_int, c_vp, c_int, c_int, c_vp, c_int, c_int, c_int, c_int, c_vp],
+    "qnn_gate_heads": [c_vp, c_int, c_ll, c_vp, c_int, c_int, c_vp, c_int, c_vp, c_ll, c_float, c_int, c_int, c_int, c_vp],
+    "qnn_causal_conv": [c_vp, c_int, c_ll, c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_int, c_ll, c_vp, c_ll, c_int,
+                        c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_vp],
+    "qnn_stream_update": [c_vp, c_vp, c_int, c_float, c_vp, c_int, c_float, c_int, c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_vp,
+                          c_vp, c_int, c_float, c_int, c_vp, c_int, c_int, c_int, c_vp],
+    "qnn_block_linear": [c_vp, c_int, c_ll, c_ll, c_vp, c_int, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_int, c_int, c_int,
+                         c_int, c_vp],
+    "qnn_linear_recurrence": [c_vp, c_ll, c_vp, c_vp, c_int, c_vp, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_vp, c_int, c_float,
+                              c_vp, c_int, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_vp, c_vp],
+    "qnn_latent_prep": [c_vp, c_int, c_ll, c_int, c_int, c_vp, c_int, c_float, c_int, c_int, c_vp, c_vp, c_ll, c_vp, c_ll,
+                        c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_int, c_int, c_vp],
     "qnn_small_linear_f32": [c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_int, c_vp, c_int, c_float, c_vp],
     "qnn_gla_scan": [c_vp, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_float, c_vp, c_vp, c_vp, c_vp,
                      c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_vp],

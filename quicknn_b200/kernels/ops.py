@@ -79,15 +79,20 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: Optional
 
 
 def embed_rmsnorm(tokens: torch.Tensor, table: torch.Tensor, scale: float, weight: torch.Tensor, eps: float,
-                  unit_offset: bool, out_dtype: torch.dtype):
-    """``embed`` and the first norm of what it gives in one kernel: (rows [T, H] float32, rmsnorm(rows))."""
+                  unit_offset: bool, out_dtype: torch.dtype, out: Optional[torch.Tensor] = None):
+    """``embed`` and the first norm of what it gives in one kernel: (rows [T, H] float32, rmsnorm(rows)).  ``out``: where
+    the rows go."""
     _req(tokens, "tokens", torch.int32, 1)
     _req(table, "table", None, 2)
     _req(weight, "weight", None, 1)
     T, (V, H) = tokens.numel(), table.shape
     if weight.numel() != H:
         raise ValueError(f"norm weight has {weight.numel()} elements for width {H}")
-    out = torch.empty((T, H), dtype=torch.float32, device=tokens.device)
+    if out is None:
+        out = torch.empty((T, H), dtype=torch.float32, device=tokens.device)
+    _req(out, "out", torch.float32, 2)
+    if tuple(out.shape) != (T, H):
+        raise ValueError("embed_rmsnorm: the rows do not fit")
     normed = torch.empty((T, H), dtype=out_dtype, device=tokens.device)
     _lib.check(_lib.load().qnn_embed_rmsnorm(_p(tokens), _p(table), dt_code(table), float(scale), _p(out), _p(weight),
                                              dt_code(weight), float(eps), int(unit_offset), _p(normed), dt_code(normed),
@@ -593,24 +598,26 @@ def linear_refusal(dtype: torch.dtype, inner: int) -> Optional[str]:
     return None
 
 
-def _check_slopes(slopes: Optional[torch.Tensor], n_heads: int) -> None:
-    if slopes is not None:
-        _req(slopes, "slopes", torch.float32, 1)
-        if slopes.numel() != n_heads:
-            raise ValueError(f"attention: {slopes.numel()} distance slopes for {n_heads} query heads")
+def _check_per_head(slopes: Optional[torch.Tensor], sinks: Optional[torch.Tensor], n_heads: int) -> None:
+    for t, what in ((slopes, "distance slopes"), (sinks, "sinks")):
+        if t is not None:
+            _req(t, what, torch.float32, 1)
+            if t.numel() != n_heads:
+                raise ValueError(f"attention: {t.numel()} {what} for {n_heads} query heads")
 
 
 def attn_prefill(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, tok_pos: torch.Tensor,
                  tok_row0: torch.Tensor, scale: float, cap: Optional[float], window: Optional[int],
                  seq_row0: Optional[torch.Tensor] = None, seq_len: Optional[torch.Tensor] = None,
-                 max_len: int = 0, slopes: Optional[torch.Tensor] = None):
+                 max_len: int = 0, slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
     """Causal (optionally windowed) attention of this step's own rows.  qkv: [T, (nq+2nkv)*hd]
     after rotation; returns [T, nq*hd].  bfloat16 with head sizes 64/128/256 runs on the tensor
     cores when the per-sequence arrays (first row, length) are given; everything else takes the
     generic kernel.  ``slopes`` (float32, one per query head, optional): ``slope * (i - j)`` is subtracted from the
-    score of query position i and key position j."""
+    score of query position i and key position j.  ``sinks`` (float32, one per query head, optional): exp(sink) joins the
+    denominator of every row's softmax, without a key, a value, the scale or a bias; all attention wrappers take it."""
     _req(qkv, "qkv", None, 2)
-    _check_slopes(slopes, n_heads)
+    _check_per_head(slopes, sinks, n_heads)
     T = qkv.shape[0]
     out = torch.empty((T, n_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
     es = qkv.element_size()
@@ -626,32 +633,32 @@ def attn_prefill(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, tok_
             code = L.qnn_attn_prefill_tcgen05(
                 _p(qkv), T, _p(out), out.shape[1], _p(seq_row0), _p(seq_len), None, seq_row0.numel(), int(max_len),
                 n_heads, n_kv, head_dim, float(scale), float(cap or 0.0), int(window or 0),
-                _p(_status_word(qkv.device)), _p(slopes), _stream())
+                _p(_status_word(qkv.device)), _p(slopes), _p(sinks), _stream())
             if code != _lib.ERR_UNSUPPORTED:
                 _lib.check(code, "attn_prefill_tcgen05")
                 return out
         code = L.qnn_attn_prefill_mma(
             ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], _p(out),
             out.shape[1], _p(seq_row0), _p(seq_len), seq_row0.numel(), int(max_len), n_heads, n_kv, head_dim,
-            float(scale), float(cap or 0.0), int(window or 0), _p(slopes), _stream())
+            float(scale), float(cap or 0.0), int(window or 0), _p(slopes), _p(sinks), _stream())
         if code != _lib.ERR_UNSUPPORTED:
             _lib.check(code, "attn_prefill_mma")
             return out
     _lib.check(L.qnn_attn_prefill_generic(
         ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], dt_code(qkv),
         _p(out), out.shape[1], _p(tok_pos), _p(tok_row0), T, n_heads, n_kv, head_dim, float(scale),
-        float(cap or 0.0), int(window or 0), _p(slopes), _stream()), "attn_prefill")
+        float(cap or 0.0), int(window or 0), _p(slopes), _p(sinks), _stream()), "attn_prefill")
     return out
 
 
 def attn_prefill_paged(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_pool: torch.Tensor,
                        v_pool: torch.Tensor, page_table: torch.Tensor, page_size: int, ring: int,
                        tok_pos: torch.Tensor, tok_slot: torch.Tensor, scale: float, cap: Optional[float],
-                       window: Optional[int], slopes: Optional[torch.Tensor] = None):
+                       window: Optional[int], slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
     """Several query rows per sequence against the paged cache (keys written earlier in the
     same step by the layer that owns the line).  q = the first nq*hd columns of qkv."""
     _req(qkv, "qkv", None, 2)
-    _check_slopes(slopes, n_heads)
+    _check_per_head(slopes, sinks, n_heads)
     _req(k_pool, "k_pool", qkv.dtype, 4)
     _req(v_pool, "v_pool", qkv.dtype, 4)
     T = qkv.shape[0]
@@ -660,7 +667,7 @@ def attn_prefill_paged(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int
     _lib.check(L.qnn_attn_prefill_paged(
         _p(qkv), qkv.shape[1], dt_code(qkv), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1],
         page_size, ring, _p(out), out.shape[1], _p(tok_pos), _p(tok_slot), T, n_heads, n_kv, head_dim,
-        float(scale), float(cap or 0.0), int(window or 0), _p(slopes), _stream()), "attn_prefill_paged")
+        float(scale), float(cap or 0.0), int(window or 0), _p(slopes), _p(sinks), _stream()), "attn_prefill_paged")
     return out
 
 
@@ -668,7 +675,7 @@ def attn_shared_tensor_core(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: 
                             v_pool: torch.Tensor, page_table: torch.Tensor, page_size: int, ring: int, slots: torch.Tensor,
                             seq_row0: torch.Tensor, seq_len: torch.Tensor, scale: float, cap: Optional[float],
                             window: Optional[int], longest: int, whole=None,
-                            slopes: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                            slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """Attention of query rows ``q`` ([rows, n_heads * head_dim]) whose keys and values, this step's positions included,
     are in the paged cache already (a layer that reads the line another layer wrote earlier in the step), on the
     tensor-core prompt kernel: keys and values are copied out of the pages beside the queries into whole sequences,
@@ -677,7 +684,7 @@ def attn_shared_tensor_core(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: 
     if not (ATTN_TCGEN05 and q.dtype == torch.bfloat16 and head_dim in (64, 128, 256)):
         return None
     _req(q, "q", torch.bfloat16, 2)
-    _check_slopes(slopes, n_heads)
+    _check_per_head(slopes, sinks, n_heads)
     L = _lib.load()
     width = (n_heads + 2 * n_kv) * head_dim
     if whole is None:
@@ -693,7 +700,7 @@ def attn_shared_tensor_core(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: 
     out_rows = torch.empty((total, n_heads * head_dim), dtype=q.dtype, device=q.device)
     code = L.qnn_attn_prefill_tcgen05(
         _p(rows), total, _p(out_rows), out_rows.shape[1], _p(row0), _p(length), _p(start), B, most, n_heads, n_kv,
-        head_dim, float(scale), float(cap or 0.0), int(window or 0), _p(_status_word(q.device)), _p(slopes), _stream())
+        head_dim, float(scale), float(cap or 0.0), int(window or 0), _p(_status_word(q.device)), _p(slopes), _p(sinks), _stream())
     if code == _lib.ERR_UNSUPPORTED:
         return None
     _lib.check(code, "attn_prefill_tcgen05")
@@ -703,7 +710,7 @@ def attn_shared_tensor_core(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: 
 def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                 page_table: torch.Tensor, page_size: int, ring: int, tok_pos: torch.Tensor, tok_row0: torch.Tensor,
                 tok_slot: torch.Tensor, scale: float, cap: Optional[float], window: Optional[int], whole=None,
-                slopes: Optional[torch.Tensor] = None):
+                slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
     """Attention of a step that continues sequences by several tokens: each row sees the cached
     positions before its sequence's first row of this step (from the cache, as earlier steps left it)
     and this step's own rows from there to itself (from ``qkv``, already rotated).  The caller appends
@@ -715,7 +722,7 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     the query tiles that lie before each sequence's new rows, and the new rows' outputs are picked out.
     The generic kernel walks the keys once per row and kv head: it serves float32 and the other head sizes."""
     _req(qkv, "qkv", None, 2)
-    _check_slopes(slopes, n_heads)
+    _check_per_head(slopes, sinks, n_heads)
     _req(k_pool, "k_pool", qkv.dtype, 4)
     _req(v_pool, "v_pool", qkv.dtype, 4)
     for n, t in (("tok_pos", tok_pos), ("tok_row0", tok_row0), ("tok_slot", tok_slot)):
@@ -734,7 +741,7 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
         code = L.qnn_attn_prefill_tcgen05(
             _p(rows), whole.total, _p(out_rows), out_rows.shape[1], _p(whole.row0), _p(whole.length), _p(whole.start), B,
             whole.longest, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0), int(window or 0),
-            _p(_status_word(qkv.device)), _p(slopes), _stream())
+            _p(_status_word(qkv.device)), _p(slopes), _p(sinks), _stream())
         if code != _lib.ERR_UNSUPPORTED:
             _lib.check(code, "attn_prefill_tcgen05")
             return gather_rows(out_rows, whole.tok_row, qkv.dtype)
@@ -748,7 +755,7 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
         ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], dt_code(qkv),
         _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(out), out.shape[1],
         _p(tok_pos), _p(tok_row0), _p(tok_slot), T, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0),
-        int(window or 0), _p(slopes), _stream()), "attn_extend")
+        int(window or 0), _p(slopes), _p(sinks), _stream()), "attn_extend")
     return out
 
 
@@ -756,13 +763,13 @@ def attn_decode(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
                 v_pool: torch.Tensor, page_table: torch.Tensor, page_size: int, ring: int,
                 slots: torch.Tensor, slot_len: torch.Tensor, scale: float, cap: Optional[float],
                 window: Optional[int], n_splits: int, part_o: torch.Tensor, part_ml: torch.Tensor,
-                slopes: Optional[torch.Tensor] = None):
+                slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
     """One query row per sequence against the paged cache.  q = the first nq*hd columns of qkv.
     ``slots``, ``slot_len`` and ``page_table`` must be complete before the kernel that runs just before
     this one on the stream starts (host copies and earlier kernels are): the tensor-core kernel reads
     them while that kernel may still run."""
     _req(qkv, "qkv", None, 2)
-    _check_slopes(slopes, n_heads)
+    _check_per_head(slopes, sinks, n_heads)
     B = qkv.shape[0]
     _req(k_pool, "k_pool", qkv.dtype, 4)
     _req(v_pool, "v_pool", qkv.dtype, 4)
@@ -777,7 +784,7 @@ def attn_decode(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     _lib.check(L.qnn_attn_decode(
         _p(qkv), qkv.shape[1], dt_code(qkv), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1],
         page_size, ring, _p(slots), _p(slot_len), B, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0),
-        int(window or 0), _p(part_o), _p(part_ml), n_splits, _p(out), out.shape[1], _p(slopes), _stream()), "attn_decode", 2)
+        int(window or 0), _p(part_o), _p(part_ml), n_splits, _p(out), out.shape[1], _p(slopes), _p(sinks), _stream()), "attn_decode", 2)
     return out
 
 
@@ -956,18 +963,24 @@ def scale_heads(x: torch.Tensor, gate_logits: torch.Tensor, n_heads: int) -> tor
     return x
 
 
-def gate_heads(o: torch.Tensor, x: torch.Tensor, w_gate: torch.Tensor, n_heads: int) -> torch.Tensor:
-    """o[t, h, :] *= sigmoid(x[t, :] . w_gate[h, :]) in place: ``small_linear_f32`` and ``scale_heads`` in one kernel
-    (the logits and the sigmoid in float32)."""
+def gate_heads(o: torch.Tensor, x: torch.Tensor, w_gate: torch.Tensor, n_heads: int, scale: float = 1.0,
+               out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
+    """o[t, h, :] * scale * sigmoid(x[t, :] . w_gate[h, :]), in place or into the columns ``out_col0 ..`` of ``out``:
+    ``small_linear_f32`` and ``scale_heads`` in one kernel (the logits and the sigmoid in float32)."""
     _req(o, "o", None, 2)
     _req(x, "x", None, 2)
     _req(w_gate, "w_gate", None, 2)
     T, HD = o.shape
-    if HD % n_heads or x.shape[0] != T or tuple(w_gate.shape) != (n_heads, x.shape[1]):
+    if out is None:
+        out, out_col0 = o, 0
+    _req(out, "out", o.dtype, 2)
+    if (HD % n_heads or x.shape[0] != T or tuple(w_gate.shape) != (n_heads, x.shape[1]) or out.shape[0] != T
+            or out_col0 + HD > out.shape[1]):
         raise ValueError("gate_heads: shapes do not agree")
-    _lib.check(_lib.load().qnn_gate_heads(_p(x), dt_code(x), _p(w_gate), dt_code(w_gate), x.shape[1], _p(o), dt_code(o), T,
-                                          n_heads, HD // n_heads, _stream()), "gate_heads")
-    return o
+    _lib.check(_lib.load().qnn_gate_heads(_p(x), dt_code(x), x.shape[1], _p(w_gate), dt_code(w_gate), x.shape[1], _p(o),
+                                          dt_code(o), _col_ptr(out, out_col0), out.shape[1], float(scale), T, n_heads,
+                                          HD // n_heads, _stream()), "gate_heads")
+    return out
 
 
 def small_linear_f32(x: torch.Tensor, w: torch.Tensor, decay_bias: Optional[torch.Tensor] = None,
@@ -1763,3 +1776,172 @@ def sigmoid_attention(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int,
         gate.shape[1] if gate is not None else 0, _p(out), out.shape[1], _p(partial), splits, T, H, G, D, _stream()),
         "sigmoid_attention", 2 if splits > 1 else 1)
     return out
+
+
+# ---- short convolutions, block-diagonal products, the gated linear recurrence, rows of latent attention, averages over depth ----
+
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_row0: Optional[torch.Tensor],
+                seq_len: Optional[torch.Tensor], tok_pos: torch.Tensor, slots: torch.Tensor, n_seqs: int, longest: int = 1, *,
+                col0: int = 0, x_bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None,
+                add_input: bool = False) -> torch.Tensor:
+    """A causal convolution over time per channel: with v = x[:, col0 : col0 + C] + x_bias,
+    out_t = sum_j weight[:, j] v_(t - taps + 1 + j) + out_bias (+ v_t with ``add_input``), zeros before a sequence's first
+    position.  weight: [C, taps].  ``state``: float32 [slots, >= taps * C], whose first taps * C numbers per slot are a ring
+    of the last inputs (position p in row p mod taps).  ``seq_row0`` / ``seq_len`` None: a row per sequence (decode)."""
+    _req(x, "x", None, 2)
+    _req(weight, "weight", None, 2)
+    _req(state, "state", torch.float32)
+    C, taps = weight.shape
+    T = x.shape[0]
+    if col0 + C > x.shape[1] or state[0].numel() < taps * C or slots.numel() < n_seqs:
+        raise ValueError("causal_conv: shapes do not agree")
+    for b in (x_bias, out_bias):
+        if b is not None and b.numel() != C:
+            raise ValueError("causal_conv: a bias per channel")
+    if (seq_row0 is None) != (seq_len is None) or (seq_row0 is None and T < n_seqs):
+        raise ValueError("causal_conv: first rows and row counts come together, or a row per sequence")
+    out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    _lib.check(_lib.load().qnn_causal_conv(
+        _col_ptr(x, col0), dt_code(x), x.shape[1], _p(x_bias), dt_code(x_bias) if x_bias is not None else 0, _p(weight),
+        dt_code(weight), _p(out_bias), dt_code(out_bias) if out_bias is not None else 0, int(add_input), _p(out), dt_code(out),
+        C, _p(state), state.stride(0), C, taps, _p(seq_row0), _p(seq_len), _p(tok_pos), _p(slots), n_seqs,
+        int(longest) if seq_row0 is not None else 1, _stream()), "causal_conv")
+    return out
+
+
+def block_linear(x: torch.Tensor, w: torch.Tensor, *, col0: int = 0, step: Optional[int] = None,
+                 out_dtype: Optional[torch.dtype] = None, gate: Optional[torch.Tensor] = None,
+                 gate_col0: int = 0) -> torch.Tensor:
+    """out[t, b * N : (b + 1) * N] = w[b] x[t, col0 + b * step : ... + K], w: [blocks, N, K]; ``step`` (default K): columns
+    from one part to the next.  ``gate``: rows whose columns ``gate_col0 ..`` gate the outputs by their sigmoid.  float32
+    sums; ``out_dtype`` float32 or x's."""
+    _req(x, "x", None, 2)
+    _req(w, "w", None, 3)
+    B, N, K = w.shape
+    step = K if step is None else int(step)
+    T = x.shape[0]
+    if col0 + (B - 1) * step + K > x.shape[1]:
+        raise ValueError(f"block_linear: {B} parts of {K} columns do not fit rows of {x.shape[1]}")
+    if gate is not None:
+        _req(gate, "gate", None, 2)
+        if gate.shape[0] != T or gate_col0 + B * N > gate.shape[1]:
+            raise ValueError("block_linear: a gate per output")
+    out = torch.empty((T, B * N), dtype=out_dtype or x.dtype, device=x.device)
+    _lib.check(_lib.load().qnn_block_linear(
+        _col_ptr(x, col0), dt_code(x), x.shape[1], step, _p(w), dt_code(w), _p(out), dt_code(out), B * N,
+        _col_ptr(gate, gate_col0) if gate is not None else None, dt_code(gate) if gate is not None else 0,
+        gate.shape[1] if gate is not None else 0, T, B, N, K, _stream()), "block_linear")
+    return out
+
+
+RECURRENCE_SEGMENT = 64       # rows of a segment when sequences are walked in segments side by side; at most 64 segments
+
+
+def linear_recurrence(z: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, decay: torch.Tensor, u: torch.Tensor,
+                      part: int, state: torch.Tensor, state_col0: int, seq_row0: Optional[torch.Tensor],
+                      seq_len: Optional[torch.Tensor], slots: torch.Tensor, n_seqs: int, longest: int = 1, *,
+                      y: Optional[torch.Tensor] = None, y_col0: int = 0, y_bias: Optional[torch.Tensor] = None,
+                      scale: float = 1.0, out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
+    """S_t = a S_(t-1) + sqrt(1 - a^2) i u_t with r, i = sigmoid of the logits plus biases and a = exp(-decay r), from the
+    state of every sequence's slot and back into it; returns scale * S * gelu(y + y_bias) (scale * S without ``y``).
+    z: float32 [rows, 2C] logits, per part of ``part`` channels first r's, then i's (overwritten for long sequences).
+    ``state``: float32 [slots, n], the channels' numbers from ``state_col0`` on."""
+    _req(z, "z", torch.float32, 2)
+    _req(u, "u", None, 2)
+    _req(decay, "decay", torch.float32, 1)
+    _req(state, "state", torch.float32)
+    T, C = u.shape
+    if tuple(z.shape) != (T, 2 * C) or decay.numel() != C or r_bias.numel() != C or i_bias.numel() != C or C % part \
+            or r_bias.dtype != i_bias.dtype:
+        raise ValueError("linear_recurrence: shapes do not agree")
+    if state[0].numel() < state_col0 + C or slots.numel() < n_seqs or (seq_row0 is None and T < n_seqs):
+        raise ValueError("linear_recurrence: the state does not fit, or fewer rows than sequences")
+    if y is not None and (y.shape[0] != T or y_col0 + C > y.shape[1]):
+        raise ValueError("linear_recurrence: the output gate's rows do not fit")
+    if out is None:
+        out, out_col0 = torch.empty((T, C), dtype=u.dtype, device=u.device), 0
+    if out.shape[0] != T or out_col0 + C > out.shape[1]:
+        raise ValueError("linear_recurrence: the result does not fit")
+    longest = int(longest) if seq_row0 is not None else 1
+    seg = RECURRENCE_SEGMENT
+    while -(-longest // seg) > 64:
+        seg *= 2
+    nseg = -(-longest // seg) if longest > 2 * seg else 1
+    seg = seg if nseg > 1 else max(1, longest)
+    scratch = torch.empty((n_seqs, nseg, 3, C), dtype=torch.float32, device=u.device) if nseg > 1 else None
+    _lib.check(_lib.load().qnn_linear_recurrence(
+        _p(z), z.shape[1], _p(r_bias), _p(i_bias), dt_code(r_bias), _p(decay), _p(u), dt_code(u), C,
+        _col_ptr(y, y_col0) if y is not None else None, dt_code(y) if y is not None else 0, y.shape[1] if y is not None else 0,
+        _p(y_bias), dt_code(y_bias) if y_bias is not None else 0, float(scale), _col_ptr(out, out_col0), dt_code(out),
+        out.shape[1], ctypes.c_void_p(state.data_ptr() + 4 * state_col0), state.stride(0), _p(seq_row0), _p(seq_len),
+        _p(slots), n_seqs, C, int(part), seg, nseg, _p(scratch), _stream()), "linear_recurrence", 2 if nseg > 1 else 1)
+    return out
+
+
+def latent_prep(a: torch.Tensor, c_col: int, r_col: int, weight: torch.Tensor, eps: float, rot_dim: int,
+                inv_freq: torch.Tensor, q: torch.Tensor, n_heads: int, head_dim: int, tok_pos: torch.Tensor,
+                tok_slot: torch.Tensor, line, append: bool, packed: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The rows of latent attention.  Key row: the ``rot_dim`` columns of ``a`` from ``r_col`` on, rotated, then the latent
+    (``weight.numel()`` columns from ``c_col`` on) RMS-normed with the plain weight, then zeros up to ``head_dim``.  The first
+    ``rot_dim`` columns of every query head of ``q`` ([rows, heads * head_dim]) are rotated, in place, or, with ``packed``
+    ([rows, (heads + 2) * head_dim]), into that buffer with the key row twice behind them.  ``append``: the key row goes to
+    the cache line."""
+    _req(a, "a", None, 2)
+    _req(q, "q", a.dtype, 2)
+    _req(weight, "weight", None, 1)
+    T, rank = a.shape[0], weight.numel()
+    dst = q if packed is None else packed
+    _req(dst, "packed", a.dtype, 2)
+    if (q.shape != (T, n_heads * head_dim) or head_dim < rank + rot_dim or c_col + rank > a.shape[1]
+            or r_col + rot_dim > a.shape[1] or dst.shape[0] != T or (packed is not None and dst.shape[1] != (n_heads + 2) * head_dim)):
+        raise ValueError("latent_prep: shapes do not agree")
+    if rot_dim:
+        _req(inv_freq, "inv_freq", torch.float32, 1)
+        if inv_freq.numel() != rot_dim // 2:
+            raise ValueError("latent_prep: a frequency per rotated pair")
+    pool = table = slot_len = None
+    max_pages = page_size = ring = 0
+    if append:
+        _req(line.k, "cache", a.dtype, 4)
+        if tuple(line.k.shape[1:]) != (1, line.page_size, head_dim):
+            raise ValueError("latent_prep: the cache line has another shape")
+        pool, table, slot_len, max_pages = line.k, line.page_table, line.slot_len, line.page_table.shape[1]
+        page_size, ring = line.page_size, line.ring
+    _lib.check(_lib.load().qnn_latent_prep(
+        _p(a), dt_code(a), a.shape[1], int(c_col), int(r_col), _p(weight), dt_code(weight), float(eps), rank, int(rot_dim),
+        _p(inv_freq) if rot_dim else None, _p(q), q.shape[1], _p(dst), dst.shape[1], n_heads, head_dim,
+        n_heads * head_dim if packed is not None else -1, _p(tok_pos), _p(tok_slot), _p(pool), _p(table), max_pages, page_size,
+        ring, _p(slot_len), int(append), T, _stream()), "latent_prep")
+    return dst
+
+
+def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: torch.Tensor, eps_post: float, unit_post: bool,
+                  out: Optional[torch.Tensor] = None, *, hist: Optional[torch.Tensor] = None,
+                  numbers: Optional[torch.Tensor] = None, avg_out: Optional[torch.Tensor] = None,
+                  w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0, unit_next: bool = False,
+                  out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """X = resid + mult * rmsnorm(y, w_post), written to ``out`` (default: resid, in place).  With ``hist`` ([n, rows, width]
+    float32, contiguous layers) and ``numbers`` (n + 1): avg_out = sum_j numbers[j] hist[j] + numbers[n] X.  Returns
+    rmsnorm(the average, or X; w_next) when ``w_next`` is given.  One kernel, float32 sums."""
+    _req(resid, "resid", torch.float32, 2)
+    _req(y, "y", None, 2)
+    _req(w_post, "w_post", None, 1)
+    T, H = resid.shape
+    out = resid if out is None else out
+    _req(out, "out", torch.float32, 2)
+    if tuple(y.shape) != (T, H) or tuple(out.shape) != (T, H) or w_post.numel() != H or (w_next is not None and w_next.numel() != H):
+        raise ValueError("stream_update: shapes do not agree")
+    n = 0
+    if hist is not None:
+        _req(hist, "hist", torch.float32, 3)
+        _req(avg_out, "avg_out", torch.float32, 2)
+        n = hist.shape[0]
+        if tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
+            raise ValueError("stream_update: an average takes a number per earlier layer's rows and one for these")
+    normed = torch.empty((T, H), dtype=out_dtype, device=resid.device) if w_next is not None else None
+    _lib.check(_lib.load().qnn_stream_update(
+        _p(resid), _p(y), dt_code(y), float(mult), _p(w_post), dt_code(w_post), float(eps_post), int(unit_post), _p(out),
+        _p(hist), hist.stride(0) if hist is not None else 0, n, _p(numbers), dt_code(numbers) if numbers is not None else 0,
+        _p(avg_out), _p(w_next), dt_code(w_next) if w_next is not None else 0, float(eps_next), int(unit_next), _p(normed),
+        dt_code(normed) if normed is not None else 0, T, H, _stream()), "stream_update")
+    return normed

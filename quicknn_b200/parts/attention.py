@@ -23,6 +23,10 @@ Options beyond that (all off unless the spec gives them):
   key position j (a bias that grows with the distance, in float32 inside the attention kernels).
 * ``out_gate``: the concatenated heads are multiplied, element by element, by sigmoid(``g_proj`` x) before the output
   product.
+* ``sink``: a learned number per query head (``sink``) that joins the denominator of the softmax as exp(sink); it has no
+  key and no value, takes neither the scale nor a bias and counts once (float32 inside the attention kernels).
+* ``head_gate``: every head's output is multiplied by one number, sigmoid((``head_gate`` x)_h), before the output product
+  (the logit in float32).
 * ``shared_kv``: the layer has no keys and values of its own; its schedule entry reads the cache line that another
   layer writes (whose head counts, sizes and rotation are the same), with its own queries.
 
@@ -72,9 +76,14 @@ class AttentionMixer(Mixer):
         if self._slope_values is not None and len(self._slope_values) != self.n_heads:
             raise ValueError(f"{len(self._slope_values)} distance slopes for {self.n_heads} heads")
         self.slopes: Optional[torch.Tensor] = None
+        self.has_sink = bool(p.get("sink", False))
+        self.sinks: Optional[torch.Tensor] = None
+        self.has_head_gate = bool(p.get("head_gate", False))
+        self.w_head_gate: Optional[torch.Tensor] = None
         self.w_out_gate: Optional[torch.Tensor] = None
         if p.get("v_head_dim") and (self.value_dim != self.key_dim or self.key_dim % 8):
             self.head_dim = (max(self.key_dim, self.value_dim) + 7) // 8 * 8
+        self.out_width = self.n_heads * self.head_dim            # columns that the output matrix reads
         self.heads = HeadShape(self.n_heads, 0 if self.shared_kv else self.n_kv, self.head_dim)
         pos: PartSpec = p["position"]
         if self.head_dim != self.key_dim and "head_dim" in pos.params:
@@ -110,6 +119,10 @@ class AttentionMixer(Mixer):
                 out["k_norm"] = ((nkv * hd if whole else hd,), S)
         if p.get("out_gate", False):
             out["g_proj"] = ((nq * vd, H), M)
+        if p.get("sink", False):
+            out["sink"] = ((nq,), B)
+        if p.get("head_gate", False):
+            out["head_gate"] = ((nq, H), M)
         return out
 
     def _carried(self, t: torch.Tensor, heads: int, size: int) -> torch.Tensor:
@@ -148,6 +161,10 @@ class AttentionMixer(Mixer):
                 self.w_qkv, self.w_out_gate = self.w_qkvg[:n], self.w_qkvg[n:]
         if self._slope_values is not None:
             self.slopes = torch.tensor(self._slope_values, dtype=torch.float32, device=device)
+        if self.has_sink:
+            self.sinks = tensors["sink"].to(torch.float32).contiguous()
+        if self.has_head_gate:
+            self.w_head_gate = tensors["head_gate"].contiguous()
         if self.has_bias or self.qk_norm:
             self.prep = HeadPrep(
                 bias=torch.cat([b.to(torch.float32) for b in biases]).contiguous() if biases else None,
@@ -169,7 +186,7 @@ class AttentionMixer(Mixer):
         self._resident = sms * max(1, min(8, 512 // max(1, self.head_dim)))
 
     def weight_bytes(self) -> int:
-        ws = [self.w_qkv, self.w_o, self.out_bias, self.w_out_gate]
+        ws = [self.w_qkv, self.w_o, self.out_bias, self.w_out_gate, self.w_head_gate, self.sinks]
         if self.prep is not None:
             ws += [self.prep.bias, self.prep.q_norm, self.prep.k_norm]
         return sum(w.numel() * w.element_size() for w in ws if w is not None)
@@ -226,7 +243,21 @@ class AttentionMixer(Mixer):
             return 0
         return step.n_seqs * self.n_heads * self.decode_splits(step) * (self.head_dim + 2) * 4
 
+    def before_output(self, x: torch.Tensor, step, line, scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                      out_col0: int = 0) -> torch.Tensor:
+        """What the output matrix multiplies, times ``scale``, into the columns ``out_col0 ..`` of ``out`` when given: the
+        gated heads of a layer with a gate per head."""
+        if not self.has_head_gate:
+            raise ValueError("attention: rows before the output product are offered by layers with a gate per head")
+        return ops.gate_heads(self._heads_of(x, step, line), x, self.w_head_gate, self.n_heads, scale, out, out_col0)
+
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
+        a = self.before_output(x, step, line) if self.has_head_gate else self._heads_of(x, step, line)
+        y = project(a, self.w_o)
+        return y if (self.out_bias is None or self.defer_out_bias) else ops.add_bias_(y, self.out_bias)
+
+    def _heads_of(self, x: torch.Tensor, step, line) -> torch.Tensor:
+        """The concatenated heads (with the gate per element, where the layer has one)."""
         h = self.heads
         extend = step.mode == "extend"
         fusable = not extend and self.prep is None and not self.shared_kv
@@ -248,8 +279,7 @@ class AttentionMixer(Mixer):
             a = ops.sigmoid_gate_(a, qkv, gate_col)
         elif self.out_gate:
             a = ops.sigmoid_gate_(a, project(x, self.w_out_gate))
-        y = project(a, self.w_o)
-        return y if (self.out_bias is None or self.defer_out_bias) else ops.add_bias_(y, self.out_bias)
+        return a
 
     def _attend_rows_of(self, left, q: torch.Tensor, step, line) -> torch.Tensor:
         """Attention of the query rows ``q`` (the first columns of its rows) over the keys and values in the packed rows
@@ -266,9 +296,9 @@ class AttentionMixer(Mixer):
         if step.mode == "extend":
             return ops.attn_extend(packed, self.n_heads, nkv, D, line.k, line.v, line.page_table, line.page_size,
                                    line.ring, step.tok_pos, step.tok_row0, step.tok_slot, self.scale, self.softcap,
-                                   self.window, whole=getattr(step, "whole", None), slopes=self.slopes)
+                                   self.window, whole=getattr(step, "whole", None), slopes=self.slopes, sinks=self.sinks)
         return ops.attn_prefill(packed, self.n_heads, nkv, D, step.tok_pos, step.tok_row0, self.scale, self.softcap,
-                                self.window, step.seq_row0, step.seq_len, step.max_q_len, slopes=self.slopes)
+                                self.window, step.seq_row0, step.seq_len, step.max_q_len, slopes=self.slopes, sinks=self.sinks)
 
     def attend(self, qkv: torch.Tensor, step, line) -> torch.Tensor:
         """Attention of the packed q|k|v rows of a step, by the step's mode.  In prefill and decode the keys and
@@ -281,7 +311,7 @@ class AttentionMixer(Mixer):
             # so that the first rows still find the ring cells that the last rows overwrite
             a = ops.attn_extend(qkv, h.n_heads, h.n_kv_heads, h.head_dim, line.k, line.v, line.page_table,
                                 line.page_size, line.ring, step.tok_pos, step.tok_row0, step.tok_slot, self.scale,
-                                self.softcap, self.window, whole=getattr(step, "whole", None), slopes=self.slopes)
+                                self.softcap, self.window, whole=getattr(step, "whole", None), slopes=self.slopes, sinks=self.sinks)
             append = lambda: ops.cache_append(qkv, h.n_heads, h.n_kv_heads, h.head_dim, step.tok_pos, step.tok_slot, line)  # noqa: E731
             if line.has_readers and hasattr(step, "after_layers"):
                 step.after_layers.append(append)             # the line's readers come first: see _attend_rows_of
@@ -308,15 +338,15 @@ class AttentionMixer(Mixer):
                 a = ops.attn_shared_tensor_core(qkv, self.n_heads, self.n_kv, self.head_dim, line.k, line.v,
                                                 line.page_table, line.page_size, line.ring, step.slots, step.seq_row0,
                                                 step.seq_len, self.scale, self.softcap, self.window, step.max_q_len,
-                                                whole=whole, slopes=self.slopes)
+                                                whole=whole, slopes=self.slopes, sinks=self.sinks)
             if a is None:
                 a = ops.attn_prefill_paged(qkv, self.n_heads, self.n_kv, self.head_dim, line.k, line.v,
                                            line.page_table, line.page_size, line.ring, step.tok_pos, step.tok_slot,
-                                           self.scale, self.softcap, self.window, slopes=self.slopes)
+                                           self.scale, self.softcap, self.window, slopes=self.slopes, sinks=self.sinks)
         elif step.mode == "prefill":
             a = ops.attn_prefill(qkv, self.n_heads, self.n_kv, self.head_dim, step.tok_pos, step.tok_row0,
                                  self.scale, self.softcap, self.window, step.seq_row0, step.seq_len, step.max_q_len,
-                                 slopes=self.slopes)
+                                 slopes=self.slopes, sinks=self.sinks)
         else:
             splits = self.decode_splits(step)
             n = step.n_seqs * self.n_heads * splits
@@ -324,5 +354,5 @@ class AttentionMixer(Mixer):
             a = ops.attn_decode(qkv, self.n_heads, self.n_kv, self.head_dim, line.k, line.v, line.page_table,
                                 line.page_size, line.ring, step.slots, line.slot_len, self.scale, self.softcap,
                                 self.window, splits, part[:n * self.head_dim], part[n * self.head_dim:n * (self.head_dim + 2)],
-                                slopes=self.slopes)
+                                slopes=self.slopes, sinks=self.sinks)
         return a

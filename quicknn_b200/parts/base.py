@@ -128,6 +128,7 @@ class Part:
     PARAM_ROLE_MATRIX = "matrix"
     PARAM_ROLE_NORM = "norm"          # drawn around 0: weights applied as 1 + w, biases
     PARAM_ROLE_SCALE = "scale"        # drawn around 1: weights that multiply as they are
+    PARAM_ROLE_AVERAGE = "average"    # drawn around 1/n, n the number of elements: weights of a sum of n terms
 
     def __init__(self, spec: PartSpec):
         self.spec = spec
@@ -204,6 +205,10 @@ class FeedForward(Part):
 
 
 class Block(Part):
+    def state_need(self) -> Optional[StateNeed]:
+        """Fixed-size state of the block itself (beside the mixer's)."""
+        return None
+
     def first_norm(self):
         """The norm that this block applies to its input first, or None.  When it gives one,
         the block that runs before it may apply it (fused with its own last add) and hand

@@ -2,7 +2,10 @@
 
 ``sandwich`` (Gemma 2, src/models/QuickNN.Models.Gemma2.pas:166-189): a norm before
 and after each sublayer, the post-norm applied to the sublayer's output before it
-is added:  x += post(mixer(pre(x)));  x += post(ff(pre(x))).
+is added:  x += post(mixer(pre(x)));  x += post(ff(pre(x))).  Options: ``residual_mult`` (what is added is multiplied by it);
+a layer may lack the feed-forward; ``input_conv`` = taps (what the mixer reads is h + conv(h), a causal convolution over time
+per channel, whose last inputs are a state of the block); ``depth_average`` = n (what the layer gives is kept, and what goes on
+is the sum of its and all earlier results, the embedded rows among them, with n learned numbers).
 ``prenorm``: x += m mixer(pre(x));  x += m ff(pre(x)), with a constant m (``residual_mult``, 1 unless given) and a
 feed-forward that a layer may lack.  The add and the norm that follows are one kernel for an RMSNorm and for every norm
 that offers ``add_then`` (the dynamic tanh).
@@ -22,12 +25,12 @@ may be asked to apply the first norm of the layer that runs next (``next_norm``)
 """
 from __future__ import annotations
 
-from typing import Dict, Tuple
+from typing import Dict, Optional, Tuple
 
 import torch
 
 from ..kernels import ops
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, StateNeed
 from .norm import GroupRMSNorm, LayerNorm, NoNorm, RMSNorm
 from .parallel import ParallelMixer
 from .spec import LayerSpec, PartSpec
@@ -91,8 +94,77 @@ class _LayerParts(Block):
 class SandwichBlock(_LayerParts):
     NORM_NAMES = ("pre_mixer", "post_mixer", "pre_ff", "post_ff")
 
+    def __init__(self, layer: LayerSpec):
+        super().__init__(layer)
+        b = layer.block
+        self.mult = float(b.get("residual_mult", 1.0))
+        self.conv_taps = b.get("input_conv")
+        self.depth_terms = b.get("depth_average")
+        self.hidden = int(b.get("hidden_size", 0))
+        self.conv: Optional[torch.Tensor] = None             # [hidden, taps]
+        self.depth: Optional[torch.Tensor] = None            # [n]
+        # the plain arrangement (two kernels around a feed-forward that is there) or the general one
+        self.general = self.mult != 1.0 or self.conv_taps is not None or self.depth_terms is not None or self.ff is None
+        if self.general and not all(isinstance(n, RMSNorm) for n in self.norms.values()):
+            raise ValueError("sandwich: a multiplier, an input convolution, an average over depth and a missing "
+                             "feed-forward go with RMS norms")
+
+    @classmethod
+    def layer_param_shapes(cls, layer: LayerSpec) -> Dict[str, Tuple[Tuple[int, ...], str]]:
+        out = super().layer_param_shapes(layer)
+        b = layer.block
+        if b.get("input_conv") is not None:
+            out["input_conv"] = ((int(b.params["hidden_size"]), int(b.get("input_conv"))), cls.PARAM_ROLE_MATRIX)
+        if b.get("depth_average") is not None:
+            out["depth_average"] = ((int(b.get("depth_average")),), cls.PARAM_ROLE_AVERAGE)
+        return out
+
+    def load(self, tensors, compute_dtype, device) -> None:
+        super().load(tensors, compute_dtype, device)
+        if self.conv_taps is not None:
+            self.conv = tensors["input_conv"].contiguous()
+        if self.depth_terms is not None:
+            self.depth = tensors["depth_average"].contiguous()
+
+    def weight_bytes(self) -> int:
+        return super().weight_bytes() + sum(w.numel() * w.element_size() for w in (self.conv, self.depth) if w is not None)
+
+    def state_need(self) -> Optional[StateNeed]:
+        return None if self.conv_taps is None else StateNeed((int(self.conv_taps), self.hidden), "float32")
+
     def first_norm(self):
         return self.norms["pre_mixer"]
+
+    def _update(self, resid, y, post: str, then, step, out, closes: bool):
+        """out = resid + mult * post(y); when that closes the layer and the model averages over depth, the average goes to
+        ``step.depth.stream``.  Returns then(the new stream) when ``then`` is an RMSNorm."""
+        p, d = self.norms[post], step.depth
+        kw = {}
+        if closes and self.depth is not None:
+            kw.update(hist=d.results[:d.index + 1], numbers=self.depth, avg_out=d.stream)
+        if isinstance(then, RMSNorm):
+            kw.update(w_next=then.weight, eps_next=then.eps, unit_next=then.unit_offset, out_dtype=step.act_dtype)
+        return ops.stream_update(resid, y, self.mult, p.weight, p.eps, p.unit_offset, out, **kw)
+
+    def _forward_general(self, resid: torch.Tensor, step, line, n, next_norm):
+        if self.conv is not None:
+            decode = step.mode == "decode"
+            n = ops.causal_conv(n, self.conv, line.block_state, None if decode else step.seq_row0,
+                                None if decode else step.seq_len, step.tok_pos, step.slots, step.n_seqs,
+                                1 if decode else step.max_q_len, add_input=True)
+        y = self.mixer.forward(n, step, line)
+        # with an average over depth the layer's result has a place of its own; the stream that came in is not touched
+        out = resid if self.depth is None else step.depth.results[step.depth.index + 1]
+        if self.ff is None:
+            n = self._update(resid, y, "post_mixer", next_norm, step, out, True)
+        else:
+            n = self._update(resid, y, "post_mixer", self.norms["pre_ff"], step, out, False)
+            y = self.ff.forward(n, step)
+            n = self._update(out, y, "post_ff", next_norm, step, out, True)
+        stream = out if self.depth is None else step.depth.stream
+        if next_norm is None:
+            return stream
+        return stream, (n if isinstance(next_norm, RMSNorm) else next_norm(stream, step.act_dtype))
 
     def forward(self, resid: torch.Tensor, step, line, normed=None, next_norm=None):
         """Returns the residual stream, or (residual stream, next_norm(residual stream)) when
@@ -100,6 +172,8 @@ class SandwichBlock(_LayerParts):
         nm = self.norms
         act = step.act_dtype
         n = normed if normed is not None else nm["pre_mixer"](resid, act)
+        if self.general:
+            return self._forward_general(resid, step, line, n, next_norm)
         y = self.mixer.forward(n, step, line)
         if isinstance(nm["post_mixer"], RMSNorm) and isinstance(nm["pre_ff"], RMSNorm):
             n = nm["post_mixer"].add_to(resid, y, then=nm["pre_ff"], out_dtype=act)

@@ -45,9 +45,11 @@ class RMSNorm(Norm):
     def __call__(self, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         return ops.rmsnorm(x, self.weight, self.eps, self.unit_offset, out_dtype)
 
-    def of_embedding(self, tokens: torch.Tensor, table: torch.Tensor, scale: float, out_dtype: torch.dtype):
-        """(embedded rows, self(embedded rows)) in one kernel: the first norm of a model's first layer."""
-        return ops.embed_rmsnorm(tokens, table, scale, self.weight, self.eps, self.unit_offset, out_dtype)
+    def of_embedding(self, tokens: torch.Tensor, table: torch.Tensor, scale: float, out_dtype: torch.dtype,
+                     out: Optional[torch.Tensor] = None):
+        """(embedded rows, self(embedded rows)) in one kernel: the first norm of a model's first layer.  ``out``: where the
+        embedded rows go."""
+        return ops.embed_rmsnorm(tokens, table, scale, self.weight, self.eps, self.unit_offset, out_dtype, out)
 
     def add_to(self, resid: torch.Tensor, y: torch.Tensor, then: Optional["RMSNorm"] = None,
                out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:

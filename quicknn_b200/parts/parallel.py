@@ -1,7 +1,14 @@
-"""Mixers side by side: several mixers read the same input, each output is RMS-normed over the model width with a
-plain weight of its own, and the mixer's output is their mean.
+"""Mixers side by side: several mixers read the same input.  Either each output is RMS-normed over the model width with a
+plain weight of its own and the mixer's output is their mean,
 
     y = (1/n) sum_b  rmsnorm(branch_b(x)) * w_b
+
+or, with ``scales`` = {branch: number}, the outputs are summed with fixed numbers,
+
+    y = sum_b  scale_b branch_b(x)
+
+which is one product: the branches leave what their output matrices multiply, already scaled (``before_output``), side by side
+in one row, and the output matrices are stacked along their inner size.
 
 ``branches`` maps a name to the branch's ``PartSpec`` (any registered mixer); the branch's parameters are this mixer's
 ``<name>.<parameter>`` and its weight ``<name>.out``.  The branches share one cache line: at most one of them may keep
@@ -16,6 +23,7 @@ import torch
 
 from ..kernels import ops
 from .base import MIXERS, CacheNeed, Mixer, StateNeed
+from .linear import project
 from .spec import PartSpec
 
 
@@ -35,6 +43,11 @@ class ParallelMixer(Mixer):
         if sum(b.state_need() is not None for b in self.branches) > 1:
             raise ValueError("parallel: at most one branch may keep a state")
         self.out_weights: List[torch.Tensor] = []
+        scales = p.get("scales")
+        self.scales: Optional[List[float]] = None if scales is None else [float(scales[n]) for n in self.names]
+        self.w_o: Optional[torch.Tensor] = None          # with scales: the branches' output matrices side by side
+        if self.scales is not None and not all(hasattr(b, "before_output") for b in self.branches):
+            raise ValueError("parallel: branches with fixed scales offer their rows before the output product")
 
     @classmethod
     def param_shapes(cls, spec: PartSpec) -> Dict[str, Tuple[Tuple[int, ...], str]]:
@@ -43,7 +56,8 @@ class ParallelMixer(Mixer):
         for name, sub in p["branches"].items():
             for k, v in MIXERS.get(sub.kind).param_shapes(sub).items():
                 out[f"{name}.{k}"] = v
-            out[f"{name}.out"] = ((int(p["hidden_size"]),), cls.PARAM_ROLE_SCALE)
+            if p.get("scales") is None:
+                out[f"{name}.out"] = ((int(p["hidden_size"]),), cls.PARAM_ROLE_SCALE)
         return out
 
     def load(self, tensors, compute_dtype, device) -> None:
@@ -52,10 +66,18 @@ class ParallelMixer(Mixer):
             pre = name + "."
             b.load({k[len(pre):]: v for k, v in tensors.items() if k.startswith(pre) and k != pre + "out"},
                    compute_dtype, device)
-            self.out_weights.append(tensors[pre + "out"].contiguous())
+            if self.scales is None:
+                self.out_weights.append(tensors[pre + "out"].contiguous())
+        if self.scales is not None:
+            ws = [b.w_o for b in self.branches]
+            wide = torch.float32 if any(w.dtype == torch.float32 for w in ws) else ws[0].dtype
+            self.w_o = torch.cat([w.to(wide) for w in ws], dim=1).contiguous()
+            for b in self.branches:                      # a branch's output matrix is a range of this one's columns
+                b.w_o = None
 
     def weight_bytes(self) -> int:
-        return sum(b.weight_bytes() for b in self.branches) + sum(w.numel() * w.element_size() for w in self.out_weights)
+        own = self.out_weights + ([self.w_o] if self.w_o is not None else [])
+        return sum(b.weight_bytes() for b in self.branches) + sum(w.numel() * w.element_size() for w in own)
 
     def cache_need(self) -> Optional[CacheNeed]:
         for b in self.branches:
@@ -80,4 +102,11 @@ class ParallelMixer(Mixer):
         return [b.forward(x, step, line) for b in self.branches]
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
+        if self.scales is not None:
+            rows = torch.empty((x.shape[0], self.w_o.shape[1]), dtype=x.dtype, device=x.device)
+            col = 0
+            for b, s in zip(self.branches, self.scales):
+                b.before_output(x, step, line, s, rows, col)
+                col += b.out_width
+            return project(rows, self.w_o)
         return ops.mean_rmsnorm(self.forward_branches(x, step, line), self.out_weights, self.eps, x.dtype)

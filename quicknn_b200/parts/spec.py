@@ -84,6 +84,8 @@ class ModelSpec:
     head: HeadSpec
     max_positions: int
     stop_ids: Tuple[int, ...] = ()
+    # every layer's result is kept for the layers after it (blocks with ``depth_average``)
+    depth_history: bool = False
     # standard deviations that the random-weights mode uses: matrices, norm weights
     init_std: float = 0.02
     init_norm_std: float = 0.1

@@ -10,6 +10,7 @@ from __future__ import annotations
 
 import hashlib
 import json
+import math
 import os
 from typing import Dict, Iterator, Optional, Tuple
 
@@ -33,9 +34,12 @@ def random_tensors(arch: Architecture, cfg: ModelConfig, seed: int, dtype: torch
     for name, (shape, role) in expected_tensors(spec).items():
         g = torch.Generator(device=device)
         g.manual_seed(_tensor_seed(seed, name))
-        std = nstd if role in (Part.PARAM_ROLE_NORM, Part.PARAM_ROLE_SCALE) else spec.init_std
+        std = nstd if role in (Part.PARAM_ROLE_NORM, Part.PARAM_ROLE_SCALE, Part.PARAM_ROLE_AVERAGE) else spec.init_std
+        mean = 1.0 if role == Part.PARAM_ROLE_SCALE else 0.0
+        if role == Part.PARAM_ROLE_AVERAGE:
+            mean = 1.0 / max(1, math.prod(shape))
         t = torch.empty(shape, dtype=torch.float32, device=device)
-        t.normal_(1.0 if role == Part.PARAM_ROLE_SCALE else 0.0, std, generator=g)
+        t.normal_(mean, std, generator=g)
         yield name, t.to(dtype)
 
 
