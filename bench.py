@@ -268,7 +268,8 @@ def design_sizes(name, design="fuposun"):
     dense, latent attention + experts; Tumudra's: windowed attention beside a matrix memory, attention, retention,
     attention on the keys and values of the attention layer before it (all with the dense feed-forward); Gunirax's:
     six layers of which the second and third run twice (chunked sigmoid attention beside a lightning memory, and HGRN2,
-    with dense and routed feed-forwards in turn)."""
+    with dense and routed feed-forwards in turn); Linedra's: windowed attention beside a linear recurrence as wide as the
+    model, latent attention in every fourth layer, routed experts everywhere."""
     W, ff, heads, hd, kvh, layers, vocab, window = {
         "2b": (2304, 9216, 8, 256, 4, 8, 32768, 4096), "1b": (1536, 6144, 8, 128, 4, 8, 32768, 2048)}[name]
     rank, qr, d = (256, 768, 128) if name == "2b" else (128, 512, 64)
@@ -287,6 +288,17 @@ def design_sizes(name, design="fuposun"):
                  query_pre_attn_scalar=hd)
     if design == "fuposun":
         return [("fuposun", fupo), ("gemma2", gemma)]
+    if design == "linedra":
+        rot = d // 2
+        par = ("parallel", {"left": {"heads": heads, "kv_heads": kvh, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window}},
+                            "right": {"width": W, "blocks": 8, "conv": 4}, "left_scale": 1.25, "right_scale": 0.75})
+        # the row that the latent layers cache, latent and rotated part together, has Fuposun's latent size
+        lat = ("latent_attention", {"heads": H, "dim": d, "rot_dim": rot, "vdim": d, "q_rank": qr, "kv_rank": rank - rot,
+                                    "scale": (d + rot) ** -0.5, "rot": {"base": 1e4, "dims": rot}})
+        lmoe = {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": ff // 4, "limit": 7.0}}
+        line = dict(architecture="Linedra", vocab=vocab, width=W, embedding={"scale": W ** 0.5}, norm={"eps": 1e-6},
+                    canon={"taps": 4}, residual_mult=0.5, logit_softcap=50.0,
+                    layers=[{"type": t, "mixer": m, "mlp": lmoe} for t, m in ((par, lat, par, par) * layers)[:layers]])
     if design == "gunirax":
         # eight executed layers from six: the second and third run twice over (the loop).  Chunked sigmoid attention
         # with the other models' heads beside a lightning memory, HGRN2 layers, dense and routed feed-forwards.
@@ -331,6 +343,8 @@ def design_sizes(name, design="fuposun"):
             mixer = ("attention", dict(att, kv_from=i - 2))
         tlayers.append({"type": mixer[0], "mixer": mixer[1], "mlp": dense})
     tumu = dict(architecture="Tumudra", vocab=vocab, width=W, embedding={"scale": 1.0}, norm={"eps": 1e-6}, layers=tlayers)
+    if design == "linedra":
+        return [("linedra", line), ("fuposun", fupo), ("tumudra", tumu), ("gemma2", gemma)]
     if design == "gunirax":
         return [("gunirax", guni), ("tumudra", tumu), ("fuposun", fupo), ("gemma2", gemma)]
     return [("tumudra", tumu), ("fuposun", fupo), ("gemma2", gemma)]
@@ -412,7 +426,7 @@ def main():
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-baseline", action="store_true", help="do not time the plain PyTorch / NumPy baselines")
-    ap.add_argument("--design", default=None, choices=["fuposun", "tumudra", "mubasun", "gunirax"],
+    ap.add_argument("--design", default=None, choices=["fuposun", "tumudra", "mubasun", "gunirax", "linedra"],
                     help="instead of the record: this design beside the library's other models at equal size "
                          "(prefill, decode, kernels)")
     ap.add_argument("--design-sizes", default="1b,2b", help="with --design: which of 1b, 2b")

@@ -673,10 +673,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 
 
 template <int HD, bool FIXED>
-int launch_attn(const void* qkv, long long total_rows, void* out, long long out_stride, const int* seq_row0,
+int launch_attn(const void* qkv, long long ld, long long total_rows, void* out, long long out_stride, const int* seq_row0,
                 const int* seq_len, const int* seq_q0, int B, int max_len, int nq, int nkv, float scale, float cap,
                 int window, int* status, const float* slopes, const float* sinks, cudaStream_t st) {
-    const long long width = (long long)(nq + 2 * nkv) * HD;
+    const long long width = ld;                    // the rows may be wider than what is read of them
     CUtensorMap map_q, map_kv;
     int rc = make_map(&map_q, qkv, total_rows, width, BM);
     if (rc) return rc;
@@ -754,7 +754,7 @@ int launch_attn(const void* qkv, long long total_rows, void* out, long long out_
 
 }  // namespace
 
-// qkv: this step's projections, [T rows, (nq + 2 nkv) * hd] bfloat16, rotated; sequence b occupies rows
+// qkv: this step's projections, [T rows, (nq + 2 nkv) * hd] bfloat16, rotated, rows ld elements apart; sequence b occupies rows
 // seq_row0[b] .. + seq_len[b] - 1.  seq_q0 (may be null): row seq_q0[b] of sequence b is the first whose output is
 // wanted; the rows before it bring keys and values only (qnn_attn_extend_gather lays cached tokens out that way) and
 // their output rows hold nothing of use.  Head sizes 64, 128 and 256; QNN_ERR_UNSUPPORTED for others.  `status` as in
@@ -762,7 +762,7 @@ int launch_attn(const void* qkv, long long total_rows, void* out, long long out_
 // the other half of a pair).  seq_row0 and seq_len are read before the kernel waits for the kernel launched
 // in front of it on the stream: that kernel must not be the one that writes them (copies from the host and
 // kernels further back are complete by then).
-QNN_API int qnn_attn_prefill_tcgen05(const void* qkv, long long total_rows, void* out, long long out_stride,
+QNN_API int qnn_attn_prefill_tcgen05(const void* qkv, long long ld, long long total_rows, void* out, long long out_stride,
                                      const int* seq_row0, const int* seq_len, const int* seq_q0, int B, int max_len,
                                      int nq, int nkv, int hd, float scale, float cap, int window, int* status,
                                      const float* slopes, const float* sinks, cudaStream_t st) {
@@ -770,8 +770,9 @@ QNN_API int qnn_attn_prefill_tcgen05(const void* qkv, long long total_rows, void
     if (hd != 64 && hd != 128 && hd != 256) return QNN_ERR_UNSUPPORTED;
     if (nkv <= 0 || nq % nkv) return QNN_ERR_ARGUMENT;
     if (B > 65535 || nq > 32767 || (max_len + BM - 1) / BM > 65535) return QNN_ERR_UNSUPPORTED;
-    if (((uintptr_t)qkv & 15) || ((uintptr_t)out & 15) || (out_stride * 2) % 16) return QNN_ERR_UNSUPPORTED;
-#define QNN_ATTN_ARGS qkv, total_rows, out, out_stride, seq_row0, seq_len, seq_q0, B, max_len, nq, nkv, scale, cap, window, status, slopes, sinks, st
+    if (ld < (long long)(nq + 2 * nkv) * hd) return QNN_ERR_ARGUMENT;
+    if ((ld & 7) || ((uintptr_t)qkv & 15) || ((uintptr_t)out & 15) || (out_stride * 2) % 16) return QNN_ERR_UNSUPPORTED;
+#define QNN_ATTN_ARGS qkv, ld, total_rows, out, out_stride, seq_row0, seq_len, seq_q0, B, max_len, nq, nkv, scale, cap, window, status, slopes, sinks, st
     // With a softcap up to 70 the exponent cap * log2(e) stays below 101, so that neither exp(score) nor a row's
     // sum over a million keys leaves float32: the fixed-reference softmax with both groups of warps.  QNN_ATTN_FIXED=0
     // keeps the running maximum (for comparisons).

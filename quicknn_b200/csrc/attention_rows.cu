@@ -252,7 +252,7 @@ QNN_API int qnn_attn_prefill_paged(const void* q, long long q_stride, int dtype,
 // qnn_attn_prefill_tcgen05 with seq_q0 = seq_start then computes the new rows against everything before them.
 // grid (longest whole sequence, sequences).
 // ---------------------------------------------------------------------------------
-__global__ void extend_gather_kernel(const bf16* __restrict__ qkv, const bf16* __restrict__ k_pool,
+__global__ void extend_gather_kernel(const bf16* __restrict__ qkv, long long ld, const bf16* __restrict__ k_pool,
                                      const bf16* __restrict__ v_pool, const int* __restrict__ page_table, int max_pages,
                                      int page_size, int ring, const int* __restrict__ slots,
                                      const int* __restrict__ seq_start, const int* __restrict__ seq_row0,
@@ -270,7 +270,7 @@ __global__ void extend_gather_kernel(const bf16* __restrict__ qkv, const bf16* _
         // the step's own projections: the whole row, or (queries_only: rows of a layer that reads another layer's
         // cache line) the queries alone, the keys and values of every position coming from the cache below
         const int src_chunks = queries_only ? qc : chunks;
-        const uint4* src = reinterpret_cast<const uint4*>(qkv + ((size_t)seq_row0[b] + (p - start)) * (src_chunks * 8));
+        const uint4* src = reinterpret_cast<const uint4*>(qkv + ((size_t)seq_row0[b] + (p - start)) * ld);
         for (int c = threadIdx.x; c < src_chunks; c += blockDim.x) dst[c] = src[c];
         if (!queries_only) return;
     }
@@ -297,16 +297,16 @@ __global__ void extend_gather_kernel(const bf16* __restrict__ qkv, const bf16* _
     }
 }
 
-// queries_only: qkv holds [rows, nq * hd] queries; keys and values of the step's own positions are in the cache already
+// qkv: rows ld elements apart.  queries_only: qkv holds [rows, nq * hd] queries; keys and values of the step's own positions are in the cache already
 // (another layer appended them earlier in the step).  seq_start may be null: every sequence starts at position 0.
-QNN_API int qnn_attn_extend_gather(const void* qkv, const void* k_pool, const void* v_pool, const int* page_table,
+QNN_API int qnn_attn_extend_gather(const void* qkv, long long ld, const void* k_pool, const void* v_pool, const int* page_table,
                                    int max_pages, int page_size, int ring, const int* slots, const int* seq_start,
                                    const int* seq_row0, const int* seq_len, const int* whole_row0, void* whole, int B,
                                    int longest, int nq, int nkv, int hd, int queries_only, cudaStream_t st) {
     if (B <= 0 || longest <= 0) return 0;
-    if (hd <= 0 || (hd & 7) || page_size <= 0 || B > 65535) return QNN_ERR_UNSUPPORTED;
+    if (hd <= 0 || (hd & 7) || page_size <= 0 || B > 65535 || (ld & 7)) return QNN_ERR_UNSUPPORTED;
     if ((((uintptr_t)qkv | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)whole) & 15)) return QNN_ERR_ARGUMENT;
-    qnn::launch_pdl(extend_gather_kernel, dim3((unsigned)longest, (unsigned)B), dim3(128), 0, st, (const bf16*)qkv,
+    qnn::launch_pdl(extend_gather_kernel, dim3((unsigned)longest, (unsigned)B), dim3(128), 0, st, (const bf16*)qkv, ld,
                     (const bf16*)k_pool, (const bf16*)v_pool, page_table, max_pages, page_size, ring, slots, seq_start,
                     seq_row0, seq_len, whole_row0, (bf16*)whole, nq, nkv, hd, queries_only);
     QNN_LAUNCH_CHECK();

@@ -123,7 +123,7 @@ small_linear_thread_kernel(const TX* __restrict__ x, const TW* __restrict__ w, f
     out[(size_t)(t0 + r) * N + n0 + c] = finish(d, bias, bias_dt, inv_tau, n0 + c);
 }
 
-// out[t, h, :] = o[t, h, :] * scale * sigmoid(x[t, :] . w[h, :]) (out may be o): the gate per head formed (float32) and
+// out[t, h, :] = o[t, h, :] * scale * sigmoid(x[t, :] . w[h, :]) (out may be o; without w: sigmoid(x[t, h])): the gate per head formed (float32) and
 // applied in one kernel; a block per row, the warps share the heads.  A lane's terms and the order of their sum depend on
 // the width only.
 template <typename TX, typename TW>
@@ -135,7 +135,9 @@ __global__ void gate_heads_kernel(const TX* __restrict__ x, long long ldx, const
     const TX* xr = x + (size_t)blockIdx.x * ldx;
     constexpr int VX = Vec16<TX>::N, VW = Vec16<TW>::N, V = VX > VW ? VX : VW;
     const bool vec = (W % V) == 0 && (ldx % V) == 0 && ((((uintptr_t)x | (uintptr_t)w) & 15) == 0);
-    for (int h = warp; h < H; h += nwarp) {
+    if (w == nullptr)
+        for (int h = threadIdx.x; h < H; h += blockDim.x) gate[h] = scale * (1.f / (1.f + expf(-to_f(xr[h]))));
+    for (int h = warp; h < H && w != nullptr; h += nwarp) {
         const TW* wr = w + (size_t)h * W;
         float d = 0.f;
         if (vec) {                                          // 16-byte loads where the rows allow
@@ -231,7 +233,7 @@ QNN_API int qnn_small_linear_f32(const void* x, int x_dt, const void* w, int w_d
     QNN_LAUNCH_CHECK();
 }
 
-// x: rows of pitch ldx; o: dense rows [T, H * D]; out: rows of pitch ldo in o's element type (o itself with ldo = H * D).
+// x: rows of pitch ldx (w null: the logits themselves, H of them); o: dense rows [T, H * D]; out: rows of pitch ldo in o's element type (o itself with ldo = H * D).
 QNN_API int qnn_gate_heads(const void* x, int x_dt, long long ldx, const void* w, int w_dt, int W, const void* o, int o_dt,
                            void* out, long long ldo, float scale, int T, int H, int D, cudaStream_t st) {
     if (T <= 0) return 0;

@@ -17,7 +17,7 @@
 using namespace qnn;
 
 template <typename T>
-__global__ void rope_cache_kernel(T* __restrict__ qkv, int nq, int nkv, int hd, int rot,
+__global__ void rope_cache_kernel(T* __restrict__ qkv, long long ld, int nq, int nkv, int hd, int rot,
                                   const float* __restrict__ inv_freq, const int* __restrict__ tok_pos,
                                   const int* __restrict__ tok_slot, T* __restrict__ k_pool, T* __restrict__ v_pool,
                                   const int* __restrict__ page_table, int max_pages, int page_size, int ring,
@@ -27,7 +27,7 @@ __global__ void rope_cache_kernel(T* __restrict__ qkv, int nq, int nkv, int hd, 
     const int pos = tok_pos[t];
     const int slot = tok_slot[t];
     const int half = hd / 2, rh = rot / 2;
-    const size_t row = (size_t)t * (nq + 2 * nkv) * hd;
+    const size_t row = (size_t)t * ld;
     T* q = qkv + row;
     T* k = q + (size_t)nq * hd;
     T* v = k + (size_t)nkv * hd;
@@ -81,7 +81,7 @@ __global__ void rope_cache_kernel(T* __restrict__ qkv, int nq, int nkv, int hd, 
 // partners half the rotated width away) or copies VEC values.  Needs rot/2, hd - rot and hd to be
 // multiples of VEC.
 template <typename T>
-__global__ void rope_cache_vec_kernel(T* __restrict__ qkv, int nq, int nkv, int hd, int rot,
+__global__ void rope_cache_vec_kernel(T* __restrict__ qkv, long long ld, int nq, int nkv, int hd, int rot,
                                       const float* __restrict__ inv_freq, const int* __restrict__ tok_pos,
                                       const int* __restrict__ tok_slot, T* __restrict__ k_pool,
                                       T* __restrict__ v_pool, const int* __restrict__ page_table, int max_pages,
@@ -92,7 +92,7 @@ __global__ void rope_cache_vec_kernel(T* __restrict__ qkv, int nq, int nkv, int 
     const int pos = tok_pos[t];
     const int slot = tok_slot[t];
     const int rh = rot / 2;
-    T* q = qkv + (size_t)t * (nq + 2 * nkv) * hd;
+    T* q = qkv + (size_t)t * ld;
     T* k = q + (size_t)nq * hd;
     T* v = k + (size_t)nkv * hd;
     size_t cache_base = 0;
@@ -155,15 +155,17 @@ __global__ void rope_cache_vec_kernel(T* __restrict__ qkv, int nq, int nkv, int 
     }
 }
 
-QNN_API int qnn_rope_cache_write(void* qkv, int dtype, int T, int nq, int nkv, int hd, int rot,
+// qkv: rows ld elements apart.
+QNN_API int qnn_rope_cache_write(void* qkv, long long ld, int dtype, int T, int nq, int nkv, int hd, int rot,
                                  const float* inv_freq, const int* tok_pos, const int* tok_slot, void* k_pool,
                                  void* v_pool, const int* page_table, int max_pages, int page_size, int ring,
                                  const int* slot_len, int write_cache, cudaStream_t st) {
     if (T <= 0) return 0;
     if (hd % 2 || rot % 2 || rot > hd || rot < 0) return QNN_ERR_UNSUPPORTED;
+    if (ld < (long long)(nq + 2 * nkv) * hd) return QNN_ERR_ARGUMENT;
     const int vec = dtype == QNN_DT_BF16 ? 8 : 4;
     const bool aligned = ((((uintptr_t)qkv | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15) == 0);
-    if (aligned && hd % vec == 0 && (rot / 2) % vec == 0 && (hd - rot) % vec == 0) {
+    if (aligned && ld % vec == 0 && hd % vec == 0 && (rot / 2) % vec == 0 && (hd - rot) % vec == 0) {
         const int items = (nq + nkv) * (rot / 2) / vec + nkv * (hd - rot) / vec + nkv * hd / vec;
         // a token per block; few tokens: many threads each (the step waits for this kernel's latency); many tokens:
         // small blocks, more of them on an SM (measured at 12 heads of 256: 2048 tokens 9.4 us with 64 threads,
@@ -172,11 +174,11 @@ QNN_API int qnn_rope_cache_write(void* qkv, int dtype, int T, int nq, int nkv, i
         if (T > 1024) threads = 64;
         else if (T > 256 && threads > 128) threads = 128;
         if (dtype == QNN_DT_BF16)
-            qnn::launch_pdl(rope_cache_vec_kernel<bf16>, dim3(T), dim3(threads), (size_t)(rot / 2) * sizeof(float2), st, (bf16*)qkv, nq, nkv, hd, rot,
+            qnn::launch_pdl(rope_cache_vec_kernel<bf16>, dim3(T), dim3(threads), (size_t)(rot / 2) * sizeof(float2), st, (bf16*)qkv, ld, nq, nkv, hd, rot,
                             inv_freq, tok_pos, tok_slot, (bf16*)k_pool, (bf16*)v_pool, page_table, max_pages, page_size,
                             ring, slot_len, write_cache);
         else
-            qnn::launch_pdl(rope_cache_vec_kernel<float>, dim3(T), dim3(threads), (size_t)(rot / 2) * sizeof(float2), st, (float*)qkv, nq, nkv, hd, rot,
+            qnn::launch_pdl(rope_cache_vec_kernel<float>, dim3(T), dim3(threads), (size_t)(rot / 2) * sizeof(float2), st, (float*)qkv, ld, nq, nkv, hd, rot,
                             inv_freq, tok_pos, tok_slot, (float*)k_pool, (float*)v_pool, page_table, max_pages,
                             page_size, ring, slot_len, write_cache);
         QNN_LAUNCH_CHECK();
@@ -184,11 +186,11 @@ QNN_API int qnn_rope_cache_write(void* qkv, int dtype, int T, int nq, int nkv, i
     const int work = (nq + nkv) * hd / 2;
     const int threads = work >= 1024 ? 256 : (work >= 256 ? 128 : 64);
     if (dtype == QNN_DT_BF16)
-        qnn::launch_pdl(rope_cache_kernel<bf16>, dim3(T), dim3(threads), 0, st, (bf16*)qkv, nq, nkv, hd, rot, inv_freq,
+        qnn::launch_pdl(rope_cache_kernel<bf16>, dim3(T), dim3(threads), 0, st, (bf16*)qkv, ld, nq, nkv, hd, rot, inv_freq,
                         tok_pos, tok_slot, (bf16*)k_pool, (bf16*)v_pool, page_table, max_pages, page_size, ring,
                         slot_len, write_cache);
     else
-        qnn::launch_pdl(rope_cache_kernel<float>, dim3(T), dim3(threads), 0, st, (float*)qkv, nq, nkv, hd, rot,
+        qnn::launch_pdl(rope_cache_kernel<float>, dim3(T), dim3(threads), 0, st, (float*)qkv, ld, nq, nkv, hd, rot,
                         inv_freq, tok_pos, tok_slot, (float*)k_pool, (float*)v_pool, page_table, max_pages, page_size,
                         ring, slot_len, write_cache);
     QNN_LAUNCH_CHECK();

@@ -3,6 +3,9 @@
 //   qnn_stream_update   X = resid + mult * rmsnorm(y; w_post);  X -> resid_out
 //                       with a history:  Z = sum_(j < n) a_j X_j + a_n X,  Z -> avg_out   (X_j: rows that earlier layers left)
 //                       out_next = rmsnorm(Z or X; w_next), if asked for
+//                       with a filter (decode steps, a row per sequence): h = out_next + conv(out_next), the causal
+//                       convolution of short_conv.cu over the sequence's last normed rows, in the place of out_next
+//   y may come in `terms` rows per row (the outputs of a row's experts), summed in their order.
 //
 // One block per row; the row stays in registers between its sums where it fits, eight columns per access where rows allow.
 // Earlier layers' rows are read in the order of the layers and each is used once.  All sums are float32.
@@ -22,10 +25,41 @@ struct Update {
     const void* numbers;      // [n_hist + 1]
     float* avg_out;
     void* out_next;
-    long long hist_stride;
+    const void* conv;         // [H, taps]; null: no convolution
+    float* ring;              // slot s: ring + s * slot_stride, [taps][H]: position p in row p mod taps
+    const int* tok_pos;
+    const int* slots;
+    long long hist_stride, slot_stride;
+    int terms, conv_dt, taps;
     int y_dt, wp_dt, wn_dt, num_dt, out_dt, n_hist, H;
     float mult, eps_post, off_post, eps_next, off_next;
 };
+
+// h = n + conv(n) of 8 columns from column c on, n already rounded as it is stored; the row's n joins the ring.
+__device__ __forceinline__ void conv8(const Update& u, int t, int c, float* n) {
+    const int slot = u.slots[t], pos = u.tok_pos[t];
+    if (slot < 0) return;
+    float* ring = u.ring + (size_t)slot * u.slot_stride + c;
+    float acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+    for (int j = 0; j < u.taps; ++j) {
+        const int q = pos - u.taps + 1 + j;
+        if (q < 0) continue;
+        float x[8];
+        if (q == pos) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = n[e];
+        } else {
+            load8_as_f(ring + (size_t)(q % u.taps) * u.H, QNN_DT_F32, 0, x);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(load_as_f(u.conv, u.conv_dt, (size_t)(c + e) * u.taps + j), x[e], acc[e]);
+    }
+    store8_from_f(ring + (size_t)(pos % u.taps) * u.H, QNN_DT_F32, 0, n);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) n[e] += acc[e];
+}
 
 template <int CH>
 __global__ void stream_update_vec_kernel(const Update u) {
@@ -44,7 +78,14 @@ __global__ void stream_update_vec_kernel(const Update u) {
     for (int i = 0; i < CH; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
         if (c < nchunks) {
-            load8_as_f(u.y, u.y_dt, base + (size_t)c * 8, v[i]);
+            const size_t yat = (size_t)blockIdx.x * u.terms * u.H + (size_t)c * 8;
+            load8_as_f(u.y, u.y_dt, yat, v[i]);
+            for (int k = 1; k < u.terms; ++k) {
+                float z[8];
+                load8_as_f(u.y, u.y_dt, yat + (size_t)k * u.H, z);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[i][e] += z[e];
+            }
             load8_as_f(u.resid, QNN_DT_F32, base + (size_t)c * 8, r[i]);
         } else {
 #pragma unroll
@@ -95,6 +136,12 @@ __global__ void stream_update_vec_kernel(const Update u) {
             load8_as_f(u.w_next, u.wn_dt, (size_t)c * 8, g2);
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (g2[e] + u.off_next);
+            if (u.conv != nullptr) {
+                if (u.out_dt == QNN_DT_BF16)
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) o[e] = __bfloat162float(__float2bfloat16_rn(o[e]));
+                conv8(u, blockIdx.x, c * 8, o);
+            }
             store8_from_f(u.out_next, u.out_dt, base + (size_t)c * 8, o);
         }
     }
@@ -105,9 +152,15 @@ __global__ void stream_update_kernel(const Update u) {
     __shared__ float red[32];
     pdl_wait();
     const size_t base = (size_t)blockIdx.x * u.H;
+    auto y_of = [&](int i) {
+        const size_t at = (size_t)blockIdx.x * u.terms * u.H + i;
+        float v = load_as_f(u.y, u.y_dt, at);
+        for (int k = 1; k < u.terms; ++k) v += load_as_f(u.y, u.y_dt, at + (size_t)k * u.H);
+        return v;
+    };
     float ss = 0.f;
     for (int i = threadIdx.x; i < u.H; i += blockDim.x) {
-        const float v = load_as_f(u.y, u.y_dt, base + i);
+        const float v = y_of(i);
         ss += v * v;
     }
     ss = block_sum(ss, red);
@@ -115,7 +168,7 @@ __global__ void stream_update_kernel(const Update u) {
     float ss2 = 0.f;
     for (int i = threadIdx.x; i < u.H; i += blockDim.x) {
         float r = u.resid[base + i] +
-                  u.mult * (load_as_f(u.y, u.y_dt, base + i) * inv * (load_as_f(u.w_post, u.wp_dt, i) + u.off_post));
+                  u.mult * (y_of(i) * inv * (load_as_f(u.w_post, u.wp_dt, i) + u.off_post));
         u.resid_out[base + i] = r;
         if (u.hist != nullptr) {
             float z = 0.f;
@@ -138,12 +191,17 @@ __global__ void stream_update_kernel(const Update u) {
 
 // resid may be resid_out (in place).  hist (null: no average): rows of n_hist earlier layers, hist_stride floats from one
 // layer's rows to the next's; numbers: n_hist + 1 of them, the last one for X; avg_out may be resid but not resid_out.
-// w_next / out_next null: no norm follows.
-QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, float mult, const void* w_post, int wp_dt,
+// w_next / out_next null: no norm follows.  terms: rows of y per row, summed.  conv (null: none; needs out_next and rows of
+// whole eights on 16 bytes, else QNN_ERR_UNSUPPORTED): row t is the next token, at tok_pos[t], of the sequence in slots[t].
+QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, int terms, float mult, const void* w_post, int wp_dt,
                               float eps_post, int unit_post, float* resid_out, const float* hist, long long hist_stride,
                               int n_hist, const void* numbers, int num_dt, float* avg_out, const void* w_next, int wn_dt,
-                              float eps_next, int unit_next, void* out_next, int out_dt, int T, int H, cudaStream_t st) {
+                              float eps_next, int unit_next, void* out_next, int out_dt, const void* conv, int conv_dt,
+                              int taps, float* ring, long long slot_stride, const int* tok_pos, const int* slots, int T, int H,
+                              cudaStream_t st) {
     if (T <= 0) return 0;
+    if (H <= 0 || terms < 1 || (conv != nullptr && (out_next == nullptr || ring == nullptr || taps < 1 || slot_stride < (long long)taps * H)))
+        return QNN_ERR_ARGUMENT;
     if (H <= 0 || (out_next != nullptr && w_next == nullptr)) return QNN_ERR_ARGUMENT;
     if (hist != nullptr && (n_hist < 0 || numbers == nullptr || avg_out == nullptr || avg_out == resid_out)) return QNN_ERR_ARGUMENT;
     Update u;
@@ -152,9 +210,11 @@ QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, float
     u.y_dt = y_dt; u.wp_dt = wp_dt; u.wn_dt = wn_dt; u.num_dt = num_dt; u.out_dt = out_dt; u.n_hist = n_hist; u.H = H;
     u.mult = mult; u.eps_post = eps_post; u.off_post = unit_post ? 1.f : 0.f; u.eps_next = eps_next;
     u.off_next = unit_next ? 1.f : 0.f;
+    u.terms = terms; u.conv = conv; u.conv_dt = conv_dt; u.taps = taps; u.ring = ring; u.slot_stride = slot_stride;
+    u.tok_pos = tok_pos; u.slots = slots;
     const uintptr_t all = (uintptr_t)resid | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)resid_out |
-                          (uintptr_t)hist | (uintptr_t)avg_out | (uintptr_t)out_next;
-    if ((H & 7) == 0 && (all & 15) == 0 && (hist_stride & 3) == 0 && H <= 8 * 2 * 1024) {
+                          (uintptr_t)hist | (uintptr_t)avg_out | (uintptr_t)out_next | (uintptr_t)ring;
+    if ((H & 7) == 0 && (all & 15) == 0 && (hist_stride & 3) == 0 && (slot_stride & 3) == 0 && H <= 8 * 2 * 1024) {
         const int chunks = H >> 3;
         const int ch = chunks > 1024 ? 2 : 1;
         const int threads = (((chunks + ch - 1) / ch) + 31) / 32 * 32;
@@ -162,6 +222,7 @@ QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, float
         else launch_pdl(stream_update_vec_kernel<2>, dim3(T), dim3(threads), 0, st, u);
         QNN_LAUNCH_CHECK();
     }
+    if (conv != nullptr) return QNN_ERR_UNSUPPORTED;
     launch_pdl(stream_update_kernel, dim3(T), dim3(H >= 2048 ? 512 : (H >= 512 ? 256 : 128)), 0, st, u);
     QNN_LAUNCH_CHECK();
 }

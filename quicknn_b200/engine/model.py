@@ -174,7 +174,7 @@ class Model:
         output head first and may return its result without the logits ever being written."""
         spec = self.spec
         sched = spec.schedule
-        first = self.blocks[sched[0].layer].first_norm() if sched else None
+        first = self.blocks[sched[0].layer].entry(step, cache.line(sched[0].cache, writes=sched[0].writes_cache)) if sched else None
         if self.positions is not None and self.embedding_norm is None:
             # a learned vector per position joins the looked-up row; the first layer's norm in the same kernel
             if hasattr(first, "of_embedding_rows"):
@@ -220,7 +220,8 @@ class Model:
             # that adds this layer's last sublayer to the residual stream (not where the embedded rows come between)
             nxt = None
             if i + 1 < len(sched) and not sched[i + 1].add_embedding:
-                nxt = self.blocks[sched[i + 1].layer].first_norm()
+                after = sched[i + 1]
+                nxt = self.blocks[after.layer].entry(step, cache.line(after.cache, writes=after.writes_cache))
             out = self.blocks[e.layer].forward(x, step, line, normed=normed, next_norm=nxt)
             x, normed = out if nxt is not None else (out, None)
         for call in step.after_layers:         # appends that waited for the readers of their cache line

@@ -75,6 +75,7 @@ class StepProfiler:
         self._patch(RMSNorm, "add_to", "norms and residual")
         self._patch(ops, "add_", "norms and residual")
         self._patch(ops, "add_scaled_rmsnorm", "norms and residual")
+        self._patch(ops, "stream_update", "norms and residual")
         self._patch(ops, "embed", "embedding")
         self._patch(ops, "embed_rmsnorm", "embedding")
         self._patch(model, "logits_of_rows", "head")
@@ -259,6 +260,31 @@ class OpTimer:
             rows = ff2 + (ff2 // 2 if kw.get("gated", True) else ff2)        # rows of an expert's matrices
             flops = 2.0 * T * top * rows * W
             byts = float(used * rows * W * wgu.element_size() + _nbytes(x) + _nbytes(out))
+        elif name == "causal_conv":
+            byts = float(2 * _nbytes(out) + _nbytes(a[1]))
+        elif name == "block_linear":
+            x, w, gate = a[0], a[1], kw.get("gate")
+            flops = 2.0 * x.shape[0] * w.numel()
+            byts = float(x.shape[0] * w.shape[0] * w.shape[2] * x.element_size() + _nbytes(w) + _nbytes(out)
+                         + (x.shape[0] * w.shape[0] * w.shape[1] * gate.element_size() if gate is not None else 0))
+        elif name == "linear_recurrence":
+            z, u, y = a[0], a[4], kw.get("y")
+            byts = float(_nbytes(z) + 2 * _nbytes(u) + (_nbytes(u) if y is not None else 0) + 2 * a[11] * u.shape[1] * 4)
+        elif name == "recurrent_step":
+            p, conv, w = a[0], a[5], a[7]
+            C, rows = conv.shape[0], p.shape[0]
+            flops = 2.0 * rows * w.numel()
+            byts = float(_nbytes(w) + rows * C * (3 * p.element_size() + 4 * (conv.shape[1] + 2)))
+        elif name == "latent_prep":
+            row = a[3].numel() + int(a[5])               # latent and rotated part
+            q, packed = a[7], kw.get("packed", a[14] if len(a) > 14 else None)
+            turned = q.shape[0] * int(a[8]) * int(a[5]) * q.element_size()
+            byts = float(q.shape[0] * row * q.element_size() + (_nbytes(q) + _nbytes(packed) if packed is not None else 2 * turned))
+        elif name == "stream_update":
+            resid, y = a[0], a[1]
+            byts = float(2 * _nbytes(resid) + _nbytes(y) + _nbytes(kw.get("hist")) + _nbytes(kw.get("avg_out")) + _nbytes(out))
+        elif name == "gate_heads":
+            byts = float(2 * _nbytes(a[0]) + _nbytes(a[1]) + _nbytes(a[2]))
         elif name in ("rope_cache_write",):
             byts = float(2 * _nbytes(a[0]))
         elif name.startswith("embed"):               # the rows that are looked up, not the table

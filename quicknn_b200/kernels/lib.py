@@ -29,7 +29,7 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_gather_rows": [c_vp, c_int, c_vp, c_vp, c_int, c_int, c_int, c_vp],
     "qnn_cast": [c_vp, c_int, c_vp, c_int, c_ll, c_vp],
     "qnn_check_finite": [c_vp, c_ll, c_vp, c_vp],
-    "qnn_rope_cache_write": [c_vp, c_int, c_int, c_int, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp,
+    "qnn_rope_cache_write": [c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp,
                              c_vp, c_int, c_int, c_int, c_vp, c_int, c_vp],
     "qnn_skinny_bf16": [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_float, c_vp],
     "qnn_skinny_argmax": [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_float, c_vp, c_vp],
@@ -51,9 +51,9 @@ _SIGNATURES: Dict[str, list] = {
                                  c_int, c_float, c_float, c_int, c_vp, c_vp, c_vp],
     "qnn_attn_prefill_mma": [c_vp, c_vp, c_vp, c_ll, c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int,
                              c_float, c_float, c_int, c_vp, c_vp, c_vp],
-    "qnn_attn_prefill_tcgen05": [c_vp, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_float,
+    "qnn_attn_prefill_tcgen05": [c_vp, c_ll, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_float,
                                  c_float, c_int, c_vp, c_vp, c_vp, c_vp],
-    "qnn_attn_extend_gather": [c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_int,
+    "qnn_attn_extend_gather": [c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_vp],
     "qnn_attn_prefill_paged": [c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_ll, c_vp, c_vp,
                                c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_vp, c_vp, c_vp],
@@ -70,8 +70,11 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_gate_heads": [c_vp, c_int, c_ll, c_vp, c_int, c_int, c_vp, c_int, c_vp, c_ll, c_float, c_int, c_int, c_int, c_vp],
     "qnn_causal_conv": [c_vp, c_int, c_ll, c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_int, c_ll, c_vp, c_ll, c_int,
                         c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_vp],
-    "qnn_stream_update": [c_vp, c_vp, c_int, c_float, c_vp, c_int, c_float, c_int, c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_vp,
-                          c_vp, c_int, c_float, c_int, c_vp, c_int, c_int, c_int, c_vp],
+    "qnn_stream_update": [c_vp, c_vp, c_int, c_int, c_float, c_vp, c_int, c_float, c_int, c_vp, c_vp, c_ll, c_int, c_vp, c_int,
+                          c_vp, c_vp, c_int, c_float, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_ll, c_vp, c_vp, c_int,
+                          c_int, c_vp],
+    "qnn_recurrent_step": [c_vp, c_ll, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_vp, c_vp, c_vp, c_vp, c_float, c_vp, c_ll,
+                           c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_int, c_int, c_vp],
     "qnn_block_linear": [c_vp, c_int, c_ll, c_ll, c_vp, c_int, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_int, c_int, c_int,
                          c_int, c_vp],
     "qnn_linear_recurrence": [c_vp, c_ll, c_vp, c_vp, c_int, c_vp, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_vp, c_int, c_float,

@@ -65,6 +65,17 @@ def _req(t: torch.Tensor, name: str, dtype=None, dim=None) -> None:
         raise ValueError(f"{name} must have {dim} dimensions, got {tuple(t.shape)}")
 
 
+def _rows(t: torch.Tensor, name: str, dtype=None) -> int:
+    """Check rows that may lie further apart than they are wide (a range of columns of wider rows) and return their pitch."""
+    if not t.is_cuda:
+        raise _lib.KernelError(f"{name} must be a CUDA tensor: quicknn_b200 has no CPU path")
+    if t.dim() != 2 or (t.shape[1] > 1 and t.stride(1) != 1) or (t.shape[0] > 1 and t.stride(0) < t.shape[1]):
+        raise ValueError(f"{name} must be rows of consecutive elements")
+    if dtype is not None and t.dtype != dtype:
+        raise TypeError(f"{name} must be {dtype}, got {t.dtype}")
+    return t.stride(0) if t.shape[0] > 1 else max(t.stride(0), t.shape[1])
+
+
 def embed(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None):
     _req(tokens, "tokens", torch.int32, 1)
     _req(table, "table", None, 2)
@@ -200,7 +211,7 @@ def rope_cache_write(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, 
                      k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
                      page_table: Optional[torch.Tensor], page_size: int, ring: int,
                      slot_len: Optional[torch.Tensor], write_cache: bool):
-    _req(qkv, "qkv", None, 2)
+    ld = _rows(qkv, "qkv")
     T = qkv.shape[0]
     if qkv.shape[1] != (n_heads + 2 * n_kv) * head_dim:
         raise ValueError("rope_cache_write: qkv width does not match the head counts")
@@ -220,7 +231,7 @@ def rope_cache_write(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, 
         _req(slot_len, "slot_len", torch.int32, 1)
     L = _lib.load()
     _lib.check(L.qnn_rope_cache_write(
-        _p(qkv), dt_code(qkv), T, n_heads, n_kv, head_dim, rot_dim, _p(inv_freq), _p(tok_pos), _p(tok_slot),
+        _p(qkv), ld, dt_code(qkv), T, n_heads, n_kv, head_dim, rot_dim, _p(inv_freq), _p(tok_pos), _p(tok_slot),
         _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1] if page_table is not None else 0,
         page_size, ring, _p(slot_len), int(write_cache), _stream()), "rope_cache_write")
 
@@ -615,8 +626,9 @@ def attn_prefill(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, tok_
     cores when the per-sequence arrays (first row, length) are given; everything else takes the
     generic kernel.  ``slopes`` (float32, one per query head, optional): ``slope * (i - j)`` is subtracted from the
     score of query position i and key position j.  ``sinks`` (float32, one per query head, optional): exp(sink) joins the
-    denominator of every row's softmax, without a key, a value, the scale or a bias; all attention wrappers take it."""
-    _req(qkv, "qkv", None, 2)
+    denominator of every row's softmax, without a key, a value, the scale or a bias; all attention wrappers take it.
+    The rows of ``qkv`` may be a range of columns of wider rows."""
+    ld = _rows(qkv, "qkv")
     _check_per_head(slopes, sinks, n_heads)
     T = qkv.shape[0]
     out = torch.empty((T, n_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
@@ -631,21 +643,21 @@ def attn_prefill(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, tok_
         _req(seq_len, "seq_len", torch.int32, 1)
         if ATTN_TCGEN05:
             code = L.qnn_attn_prefill_tcgen05(
-                _p(qkv), T, _p(out), out.shape[1], _p(seq_row0), _p(seq_len), None, seq_row0.numel(), int(max_len),
+                _p(qkv), ld, T, _p(out), out.shape[1], _p(seq_row0), _p(seq_len), None, seq_row0.numel(), int(max_len),
                 n_heads, n_kv, head_dim, float(scale), float(cap or 0.0), int(window or 0),
                 _p(_status_word(qkv.device)), _p(slopes), _p(sinks), _stream())
             if code != _lib.ERR_UNSUPPORTED:
                 _lib.check(code, "attn_prefill_tcgen05")
                 return out
         code = L.qnn_attn_prefill_mma(
-            ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], _p(out),
+            ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), ld, _p(out),
             out.shape[1], _p(seq_row0), _p(seq_len), seq_row0.numel(), int(max_len), n_heads, n_kv, head_dim,
             float(scale), float(cap or 0.0), int(window or 0), _p(slopes), _p(sinks), _stream())
         if code != _lib.ERR_UNSUPPORTED:
             _lib.check(code, "attn_prefill_mma")
             return out
     _lib.check(L.qnn_attn_prefill_generic(
-        ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], dt_code(qkv),
+        ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), ld, dt_code(qkv),
         _p(out), out.shape[1], _p(tok_pos), _p(tok_row0), T, n_heads, n_kv, head_dim, float(scale),
         float(cap or 0.0), int(window or 0), _p(slopes), _p(sinks), _stream()), "attn_prefill")
     return out
@@ -695,11 +707,11 @@ def attn_shared_tensor_core(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: 
         start, row0, length, new_row0, new_len = whole.start, whole.row0, whole.length, whole.new_row0, whole.new_len
     rows = torch.empty((total, width), dtype=q.dtype, device=q.device)
     _lib.check(L.qnn_attn_extend_gather(
-        _p(q), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(slots), _p(start),
+        _p(q), q.shape[1], _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(slots), _p(start),
         _p(new_row0), _p(new_len), _p(row0), _p(rows), B, most, n_heads, n_kv, head_dim, 1, _stream()), "attn_extend_gather")
     out_rows = torch.empty((total, n_heads * head_dim), dtype=q.dtype, device=q.device)
     code = L.qnn_attn_prefill_tcgen05(
-        _p(rows), total, _p(out_rows), out_rows.shape[1], _p(row0), _p(length), _p(start), B, most, n_heads, n_kv,
+        _p(rows), width, total, _p(out_rows), out_rows.shape[1], _p(row0), _p(length), _p(start), B, most, n_heads, n_kv,
         head_dim, float(scale), float(cap or 0.0), int(window or 0), _p(_status_word(q.device)), _p(slopes), _p(sinks), _stream())
     if code == _lib.ERR_UNSUPPORTED:
         return None
@@ -721,7 +733,7 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     kernel: the cached keys and values are copied out of the pages into that layout, the kernel leaves out
     the query tiles that lie before each sequence's new rows, and the new rows' outputs are picked out.
     The generic kernel walks the keys once per row and kv head: it serves float32 and the other head sizes."""
-    _req(qkv, "qkv", None, 2)
+    ld = _rows(qkv, "qkv")
     _check_per_head(slopes, sinks, n_heads)
     _req(k_pool, "k_pool", qkv.dtype, 4)
     _req(v_pool, "v_pool", qkv.dtype, 4)
@@ -734,12 +746,12 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
         B = whole.row0.numel()
         rows = torch.empty((whole.total, qkv.shape[1]), dtype=qkv.dtype, device=qkv.device)
         _lib.check(L.qnn_attn_extend_gather(
-            _p(qkv), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(whole.slots),
+            _p(qkv), ld, _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(whole.slots),
             _p(whole.start), _p(whole.new_row0), _p(whole.new_len), _p(whole.row0), _p(rows), B, whole.longest,
             n_heads, n_kv, head_dim, 0, _stream()), "attn_extend_gather")
         out_rows = torch.empty((whole.total, n_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
         code = L.qnn_attn_prefill_tcgen05(
-            _p(rows), whole.total, _p(out_rows), out_rows.shape[1], _p(whole.row0), _p(whole.length), _p(whole.start), B,
+            _p(rows), rows.shape[1], whole.total, _p(out_rows), out_rows.shape[1], _p(whole.row0), _p(whole.length), _p(whole.start), B,
             whole.longest, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0), int(window or 0),
             _p(_status_word(qkv.device)), _p(slopes), _p(sinks), _stream())
         if code != _lib.ERR_UNSUPPORTED:
@@ -752,7 +764,7 @@ def attn_extend(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     v_ptr = k_ptr + n_kv * head_dim * es
     L = _lib.load()
     _lib.check(L.qnn_attn_extend(
-        ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), qkv.shape[1], dt_code(qkv),
+        ctypes.c_void_p(q_ptr), ctypes.c_void_p(k_ptr), ctypes.c_void_p(v_ptr), ld, dt_code(qkv),
         _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1], page_size, ring, _p(out), out.shape[1],
         _p(tok_pos), _p(tok_row0), _p(tok_slot), T, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0),
         int(window or 0), _p(slopes), _p(sinks), _stream()), "attn_extend")
@@ -768,7 +780,7 @@ def attn_decode(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     ``slots``, ``slot_len`` and ``page_table`` must be complete before the kernel that runs just before
     this one on the stream starts (host copies and earlier kernels are): the tensor-core kernel reads
     them while that kernel may still run."""
-    _req(qkv, "qkv", None, 2)
+    ld = _rows(qkv, "qkv")
     _check_per_head(slopes, sinks, n_heads)
     B = qkv.shape[0]
     _req(k_pool, "k_pool", qkv.dtype, 4)
@@ -782,7 +794,7 @@ def attn_decode(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, k_poo
     out = torch.empty((B, n_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
     L = _lib.load()
     _lib.check(L.qnn_attn_decode(
-        _p(qkv), qkv.shape[1], dt_code(qkv), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1],
+        _p(qkv), ld, dt_code(qkv), _p(k_pool), _p(v_pool), _p(page_table), page_table.shape[1],
         page_size, ring, _p(slots), _p(slot_len), B, n_heads, n_kv, head_dim, float(scale), float(cap or 0.0),
         int(window or 0), _p(part_o), _p(part_ml), n_splits, _p(out), out.shape[1], _p(slopes), _p(sinks), _stream()), "attn_decode", 2)
     return out
@@ -963,22 +975,26 @@ def scale_heads(x: torch.Tensor, gate_logits: torch.Tensor, n_heads: int) -> tor
     return x
 
 
-def gate_heads(o: torch.Tensor, x: torch.Tensor, w_gate: torch.Tensor, n_heads: int, scale: float = 1.0,
-               out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
+def gate_heads(o: torch.Tensor, x: torch.Tensor, w_gate: Optional[torch.Tensor], n_heads: int, scale: float = 1.0,
+               out: Optional[torch.Tensor] = None, out_col0: int = 0, x_col0: int = 0) -> torch.Tensor:
     """o[t, h, :] * scale * sigmoid(x[t, :] . w_gate[h, :]), in place or into the columns ``out_col0 ..`` of ``out``:
-    ``small_linear_f32`` and ``scale_heads`` in one kernel (the logits and the sigmoid in float32)."""
+    ``small_linear_f32`` and ``scale_heads`` in one kernel (the logits and the sigmoid in float32).  ``w_gate`` None: the
+    logits are the columns ``x_col0 ..`` of ``x`` themselves."""
     _req(o, "o", None, 2)
     _req(x, "x", None, 2)
-    _req(w_gate, "w_gate", None, 2)
     T, HD = o.shape
     if out is None:
         out, out_col0 = o, 0
     _req(out, "out", o.dtype, 2)
-    if (HD % n_heads or x.shape[0] != T or tuple(w_gate.shape) != (n_heads, x.shape[1]) or out.shape[0] != T
-            or out_col0 + HD > out.shape[1]):
+    if w_gate is not None:
+        _req(w_gate, "w_gate", None, 2)
+        if x_col0 or tuple(w_gate.shape) != (n_heads, x.shape[1]):
+            raise ValueError("gate_heads: shapes do not agree")
+    if HD % n_heads or x.shape[0] != T or x_col0 + n_heads > x.shape[1] or out.shape[0] != T or out_col0 + HD > out.shape[1]:
         raise ValueError("gate_heads: shapes do not agree")
-    _lib.check(_lib.load().qnn_gate_heads(_p(x), dt_code(x), x.shape[1], _p(w_gate), dt_code(w_gate), x.shape[1], _p(o),
-                                          dt_code(o), _col_ptr(out, out_col0), out.shape[1], float(scale), T, n_heads,
+    _lib.check(_lib.load().qnn_gate_heads(_col_ptr(x, x_col0), dt_code(x), x.shape[1], _p(w_gate),
+                                          dt_code(w_gate if w_gate is not None else x), x.shape[1] if w_gate is not None else n_heads,
+                                          _p(o), dt_code(o), _col_ptr(out, out_col0), out.shape[1], float(scale), T, n_heads,
                                           HD // n_heads, _stream()), "gate_heads")
     return out
 
@@ -1118,7 +1134,8 @@ MOE_GROUPED_FROM = 64        # rows per expert (on average) from which prompts t
 def moe_experts(x: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, top: int, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, activation: int, limit: float, alpha: float, weight_on_input: bool,
                 shared: Optional[torch.Tensor] = None, grouped: Optional[bool] = None,
-                shared_gate: Optional[torch.Tensor] = None, identity: bool = False, gated: bool = True) -> torch.Tensor:
+                shared_gate: Optional[torch.Tensor] = None, identity: bool = False, gated: bool = True,
+                summed: bool = True) -> torch.Tensor:
     """sum over a row's chosen experts of down_e(act(gate_e(x'), up_e(x'))) (+ ``shared``), float32 [rows, width].
     ``activation``: ``GATED_CLAMPED`` or the code of a plain gate (act(g) * u, e.g. ``ACT_CODES["silu"]``).
     ``identity``: expert ids from the number of experts on are identity experts (their output is the row itself
@@ -1127,7 +1144,8 @@ def moe_experts(x: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, top: 
     The score multiplies the expert's input (x' = score * x) or its output.  w_gate_up: [experts, 2*ff, width]
     (gate rows, then up rows); w_down: [experts, width, ff].  Everything stays on the device.
     ``gated`` False: the experts are down_e(act(up_e(x'))); w_gate_up is then [experts, ff, width] (up rows alone) and
-    ``activation`` one of ``ACT_CODES``.
+    ``activation`` one of ``ACT_CODES``.  ``summed`` False (no shared expert, no identity experts): the experts' outputs
+    themselves, [rows * top, width], a row's ``top`` ones after another.
 
     Three kinds of tile: with many rows per expert (prompts; bfloat16, the clamped activation, widths in whole 16-byte
     pieces) the rows are gathered expert after expert and both products are grouped tcgen05 GEMMs over tiles of 128
@@ -1152,6 +1170,8 @@ def moe_experts(x: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, top: 
                    and (activation in (GATED_CLAMPED, ACT_CODES["silu"]) or not gated) and W % 8 == 0 and ff % 8 == 0)
     if activation != GATED_CLAMPED:
         limit = 0.0                                 # the grouped product's epilogue reads "no limit" as silu(g) * u
+    if not summed and (shared is not None or identity):
+        raise ValueError("moe_experts: what is not summed has neither a shared expert nor identity experts")
     extra = (shared_gate, (sel_e, sel_w, E, x) if identity else None)
     tile_rows = 128 if grouped else int(L.qnn_moe_tile_rows(n, E, dt_code(x), W, ff))   # else 16, or 64 with many rows each
     max_tiles = int(L.qnn_moe_max_tiles(n, E, tile_rows))
@@ -1173,19 +1193,19 @@ def moe_experts(x: torch.Tensor, sel_e: torch.Tensor, sel_w: torch.Tensor, top: 
                                  0 if gated else int(activation), float(limit), float(alpha), status, _stream())
         if code == _lib.ERR_UNSUPPORTED:           # sizes the grouped product refuses: the other tiles
             return moe_experts(x, sel_e, sel_w, top, w_gate_up, w_down, activation, limit, alpha, weight_on_input, shared,
-                               grouped=False, shared_gate=shared_gate, identity=identity, gated=gated)
+                               grouped=False, shared_gate=shared_gate, identity=identity, gated=gated, summed=summed)
         _lib.check(code, "moe_tcgen05")
         _lib.check(L.qnn_moe_tcgen05(_p(hidden), _p(w_down), _p(ys), n, E, W, ff, EPI_NONE, _p(offsets), _p(perm), _p(sel_w),
                                      _p(tiles), _p(n_tiles), max_tiles, int(not weight_on_input), 0.0, 0.0, status,
                                      _stream()), "moe_tcgen05")
-        return _moe_sum(L, ys, top, shared, T, W, *extra)
+        return _moe_sum(L, ys, top, shared, T, W, *extra) if summed else ys
     _lib.check(L.qnn_moe_gate_up(_p(x), dt_code(x), W, _p(w_gate_up), ff, _p(offsets), _p(perm), _p(sel_w), _p(tiles),
                                  _p(n_tiles), max_tiles, tile_rows, top, int(weight_on_input),
                                  int(activation) + (0 if gated else ACT_ALONE), float(limit),
                                  float(alpha), _p(hidden), _stream()), "moe_gate_up")
     _lib.check(L.qnn_moe_down(_p(hidden), dt_code(x), ff, _p(w_down), W, _p(offsets), _p(perm), _p(sel_w), _p(tiles),
                               _p(n_tiles), max_tiles, tile_rows, int(not weight_on_input), _p(ys), _stream()), "moe_down")
-    return _moe_sum(L, ys, top, shared, T, W, *extra)
+    return _moe_sum(L, ys, top, shared, T, W, *extra) if summed else ys
 
 
 def _moe_sum(L, ys: torch.Tensor, top: int, shared: Optional[torch.Tensor], T: int, W: int,
@@ -1915,21 +1935,53 @@ def latent_prep(a: torch.Tensor, c_col: int, r_col: int, weight: torch.Tensor, e
     return dst
 
 
+def recurrent_step(p: torch.Tensor, y_col0: int, x_col0: int, x_bias: torch.Tensor, y_bias: torch.Tensor, conv: torch.Tensor,
+                   conv_bias: torch.Tensor, w_gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
+                   decay: torch.Tensor, state: torch.Tensor, tok_pos: torch.Tensor, slots: torch.Tensor, scale: float,
+                   out: torch.Tensor, out_col0: int = 0) -> bool:
+    """``causal_conv``, ``block_linear`` and ``linear_recurrence`` of one token per sequence in one kernel (bfloat16, parts in
+    whole 16-byte pieces).  False where the kernel does not take the sizes or element types: nothing has run then."""
+    _req(p, "p", None, 2)
+    _req(w_gates, "w_gates", None, 3)
+    _req(out, "out", None, 2)
+    _req(state, "state", torch.float32)
+    C, taps = conv.shape
+    B, part = slots.numel(), w_gates.shape[2]
+    vecs = (x_bias, y_bias, conv, conv_bias)
+    if p.dtype != torch.bfloat16 or w_gates.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 \
+            or any(v.dtype != conv.dtype for v in vecs):
+        return False
+    if (p.shape[0] != B or w_gates.shape[0] * part != C or w_gates.shape[1] != 2 * part or out.shape[0] != B
+            or out_col0 + C > out.shape[1] or max(y_col0, x_col0) + C > p.shape[1] or state[0].numel() < (taps + 1) * C):
+        raise ValueError("recurrent_step: shapes do not agree")
+    code = _lib.load().qnn_recurrent_step(
+        _p(p), p.shape[1], int(y_col0), int(x_col0), _p(x_bias), _p(y_bias), _p(conv), _p(conv_bias), dt_code(conv), _p(w_gates),
+        _p(r_bias), _p(i_bias), _p(decay), float(scale), _col_ptr(out, out_col0), out.shape[1], _p(state), state.stride(0),
+        _p(tok_pos), _p(slots), B, C, part, taps, _stream())
+    if code == _lib.ERR_UNSUPPORTED:
+        return False
+    _lib.check(code, "recurrent_step")
+    return True
+
+
 def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: torch.Tensor, eps_post: float, unit_post: bool,
-                  out: Optional[torch.Tensor] = None, *, hist: Optional[torch.Tensor] = None,
+                  out: Optional[torch.Tensor] = None, *, terms: int = 1, hist: Optional[torch.Tensor] = None,
                   numbers: Optional[torch.Tensor] = None, avg_out: Optional[torch.Tensor] = None,
                   w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0, unit_next: bool = False,
-                  out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
-    """X = resid + mult * rmsnorm(y, w_post), written to ``out`` (default: resid, in place).  With ``hist`` ([n, rows, width]
-    float32, contiguous layers) and ``numbers`` (n + 1): avg_out = sum_j numbers[j] hist[j] + numbers[n] X.  Returns
-    rmsnorm(the average, or X; w_next) when ``w_next`` is given.  One kernel, float32 sums."""
+                  out_dtype: Optional[torch.dtype] = None, conv: Optional[tuple] = None) -> Optional[torch.Tensor]:
+    """X = resid + mult * rmsnorm(y, w_post), written to ``out`` (default: resid, in place).  ``terms``: y has that many rows
+    per row, which are summed first.  With ``hist`` ([n, rows, width] float32, contiguous layers) and ``numbers`` (n + 1):
+    avg_out = sum_j numbers[j] hist[j] + numbers[n] X.  Returns n = rmsnorm(the average, or X; w_next) when ``w_next`` is given;
+    with ``conv`` = (weight [width, taps], ring state, tok_pos, slots), a row per sequence, n + conv(n) (``causal_conv`` with
+    ``add_input``).  One kernel, float32 sums."""
     _req(resid, "resid", torch.float32, 2)
     _req(y, "y", None, 2)
     _req(w_post, "w_post", None, 1)
     T, H = resid.shape
     out = resid if out is None else out
     _req(out, "out", torch.float32, 2)
-    if tuple(y.shape) != (T, H) or tuple(out.shape) != (T, H) or w_post.numel() != H or (w_next is not None and w_next.numel() != H):
+    if tuple(y.shape) != (T * terms, H) or tuple(out.shape) != (T, H) or w_post.numel() != H \
+            or (w_next is not None and w_next.numel() != H):
         raise ValueError("stream_update: shapes do not agree")
     n = 0
     if hist is not None:
@@ -1939,9 +1991,26 @@ def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: tor
         if tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
             raise ValueError("stream_update: an average takes a number per earlier layer's rows and one for these")
     normed = torch.empty((T, H), dtype=out_dtype, device=resid.device) if w_next is not None else None
-    _lib.check(_lib.load().qnn_stream_update(
-        _p(resid), _p(y), dt_code(y), float(mult), _p(w_post), dt_code(w_post), float(eps_post), int(unit_post), _p(out),
-        _p(hist), hist.stride(0) if hist is not None else 0, n, _p(numbers), dt_code(numbers) if numbers is not None else 0,
-        _p(avg_out), _p(w_next), dt_code(w_next) if w_next is not None else 0, float(eps_next), int(unit_next), _p(normed),
-        dt_code(normed) if normed is not None else 0, T, H, _stream()), "stream_update")
+    cw = state = pos = slots = None
+    if conv is not None:
+        cw, state, pos, slots = conv
+        _req(state, "state", torch.float32)
+        if w_next is None or cw.shape[0] != H or state[0].numel() < cw.numel() or slots.numel() != T:
+            raise ValueError("stream_update: a convolution follows a norm, a filter per column, a row per sequence")
+
+    def call(with_conv: bool) -> int:
+        return _lib.load().qnn_stream_update(
+            _p(resid), _p(y), dt_code(y), int(terms), float(mult), _p(w_post), dt_code(w_post), float(eps_post), int(unit_post),
+            _p(out), _p(hist), hist.stride(0) if hist is not None else 0, n, _p(numbers),
+            dt_code(numbers) if numbers is not None else 0, _p(avg_out), _p(w_next), dt_code(w_next) if w_next is not None else 0,
+            float(eps_next), int(unit_next), _p(normed), dt_code(normed) if normed is not None else 0,
+            _p(cw) if with_conv else None, dt_code(cw) if with_conv else 0, cw.shape[1] if with_conv else 0,
+            _p(state) if with_conv else None, state.stride(0) if with_conv else 0, _p(pos) if with_conv else None,
+            _p(slots) if with_conv else None, T, H, _stream())
+
+    code = call(conv is not None)
+    if conv is not None and code == _lib.ERR_UNSUPPORTED:              # rows of other widths: the convolution on its own
+        _lib.check(call(False), "stream_update")
+        return causal_conv(normed, cw, state, None, None, pos, slots, T, add_input=True)
+    _lib.check(code, "stream_update")
     return normed

@@ -243,16 +243,32 @@ class AttentionMixer(Mixer):
             return 0
         return step.n_seqs * self.n_heads * self.decode_splits(step) * (self.head_dim + 2) * 4
 
-    def before_output(self, x: torch.Tensor, step, line, scale: float = 1.0, out: Optional[torch.Tensor] = None,
-                      out_col0: int = 0) -> torch.Tensor:
-        """What the output matrix multiplies, times ``scale``, into the columns ``out_col0 ..`` of ``out`` when given: the
-        gated heads of a layer with a gate per head."""
-        if not self.has_head_gate:
-            raise ValueError("attention: rows before the output product are offered by layers with a gate per head")
-        return ops.gate_heads(self._heads_of(x, step, line), x, self.w_head_gate, self.n_heads, scale, out, out_col0)
+    def input_matrix(self) -> torch.Tensor:
+        """Everything that multiplies the input in one matrix, for a mixer that stacks it with its other branches': q | k | v |
+        the gate's rows, in whole 16-byte pieces."""
+        if not self.has_head_gate or self.shared_kv or self.prep is not None or self.out_gate:
+            raise ValueError("attention: rows before the output product are offered by layers with a gate per head and "
+                             "without biases and head norms")
+        pad = torch.zeros(((-self.n_heads) % 8, self.hidden), dtype=self.w_qkv.dtype, device=self.w_qkv.device)
+        return stack_rows([self.w_qkv, self.w_head_gate, pad])
+
+    def release_inputs(self) -> None:
+        """Forget the input matrices: they live on in the stacked one."""
+        self.w_qkv = self.w_head_gate = None
+
+    def before_output(self, p: torch.Tensor, col0: int, step, line, scale: float, out: torch.Tensor, out_col0: int) -> torch.Tensor:
+        """What the output matrix multiplies, times ``scale``, into the columns ``out_col0 ..`` of ``out``: the gated heads.
+        p: rows whose columns from ``col0`` on are the input times ``input_matrix``."""
+        n = self.heads.width
+        qkv = p[:, col0:col0 + n]
+        self.position.place(qkv, self.heads, step, line, append=step.mode != "extend")
+        a = self.attend(qkv, step, line)
+        return ops.gate_heads(a, p, None, self.n_heads, scale, out, out_col0, x_col0=col0 + n)
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
-        a = self.before_output(x, step, line) if self.has_head_gate else self._heads_of(x, step, line)
+        a = self._heads_of(x, step, line)
+        if self.has_head_gate:
+            a = ops.gate_heads(a, x, self.w_head_gate, self.n_heads)
         y = project(a, self.w_o)
         return y if (self.out_bias is None or self.defer_out_bias) else ops.add_bias_(y, self.out_bias)
 

@@ -205,6 +205,12 @@ class FeedForward(Part):
 
 
 class Block(Part):
+    def entry(self, step, line):
+        """What this block does to the stream first, for the block that runs before it (or the embedding) to apply: what it
+        returns for a step may depend on the step's mode and on the block's cache line.  ``normed`` in ``forward`` is its
+        result."""
+        return self.first_norm()
+
     def state_need(self) -> Optional[StateNeed]:
         """Fixed-size state of the block itself (beside the mixer's)."""
         return None

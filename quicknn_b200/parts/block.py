@@ -36,6 +36,26 @@ from .parallel import ParallelMixer
 from .spec import LayerSpec, PartSpec
 
 
+class NormThenConv:
+    """A norm and the causal convolution over time that follows it: h = n + conv(n), n = norm(x).  What a block with an input
+    convolution does first, bound to a step and to the block's state."""
+
+    def __init__(self, norm: RMSNorm, weight: torch.Tensor, state: torch.Tensor, step):
+        self.norm, self.weight, self.state, self.step = norm, weight, state, step
+
+    def after(self, n: torch.Tensor) -> torch.Tensor:
+        s, decode = self.step, self.step.mode == "decode"
+        return ops.causal_conv(n, self.weight, self.state, None if decode else s.seq_row0, None if decode else s.seq_len,
+                               s.tok_pos, s.slots, s.n_seqs, 1 if decode else s.max_q_len, add_input=True)
+
+    def __call__(self, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+        return self.after(self.norm(x, out_dtype))
+
+    def of_embedding(self, tokens: torch.Tensor, table: torch.Tensor, scale: float, out_dtype: torch.dtype, out=None):
+        x, n = self.norm.of_embedding(tokens, table, scale, out_dtype, out)
+        return x, self.after(n)
+
+
 class _LayerParts(Block):
     NORM_NAMES: Tuple[str, ...] = ()
 
@@ -135,23 +155,29 @@ class SandwichBlock(_LayerParts):
     def first_norm(self):
         return self.norms["pre_mixer"]
 
-    def _update(self, resid, y, post: str, then, step, out, closes: bool):
+    def entry(self, step, line):
+        norm = self.first_norm()
+        return norm if self.conv is None else NormThenConv(norm, self.conv, line.block_state, step)
+
+    def _update(self, resid, y, post: str, then, step, out, closes: bool, terms: int = 1):
         """out = resid + mult * post(y); when that closes the layer and the model averages over depth, the average goes to
-        ``step.depth.stream``.  Returns then(the new stream) when ``then`` is an RMSNorm."""
+        ``step.depth.stream``.  Returns then(the new stream) when ``then`` is an RMSNorm, alone or with a convolution behind
+        it (in the same kernel for the single rows of a decode step)."""
         p, d = self.norms[post], step.depth
-        kw = {}
+        kw = {"terms": terms}
+        conv = None
+        if isinstance(then, NormThenConv):
+            conv, then = then, then.norm
+            if step.mode == "decode":
+                kw["conv"] = (conv.weight, conv.state, step.tok_pos, step.slots)
         if closes and self.depth is not None:
             kw.update(hist=d.results[:d.index + 1], numbers=self.depth, avg_out=d.stream)
         if isinstance(then, RMSNorm):
             kw.update(w_next=then.weight, eps_next=then.eps, unit_next=then.unit_offset, out_dtype=step.act_dtype)
-        return ops.stream_update(resid, y, self.mult, p.weight, p.eps, p.unit_offset, out, **kw)
+        n = ops.stream_update(resid, y, self.mult, p.weight, p.eps, p.unit_offset, out, **kw)
+        return n if conv is None or step.mode == "decode" else conv.after(n)
 
     def _forward_general(self, resid: torch.Tensor, step, line, n, next_norm):
-        if self.conv is not None:
-            decode = step.mode == "decode"
-            n = ops.causal_conv(n, self.conv, line.block_state, None if decode else step.seq_row0,
-                                None if decode else step.seq_len, step.tok_pos, step.slots, step.n_seqs,
-                                1 if decode else step.max_q_len, add_input=True)
         y = self.mixer.forward(n, step, line)
         # with an average over depth the layer's result has a place of its own; the stream that came in is not touched
         out = resid if self.depth is None else step.depth.results[step.depth.index + 1]
@@ -159,21 +185,22 @@ class SandwichBlock(_LayerParts):
             n = self._update(resid, y, "post_mixer", next_norm, step, out, True)
         else:
             n = self._update(resid, y, "post_mixer", self.norms["pre_ff"], step, out, False)
-            y = self.ff.forward(n, step)
-            n = self._update(out, y, "post_ff", next_norm, step, out, True)
+            y, terms = self.ff.forward_terms(n, step) if hasattr(self.ff, "forward_terms") else (self.ff.forward(n, step), 1)
+            n = self._update(out, y, "post_ff", next_norm, step, out, True, terms)
         stream = out if self.depth is None else step.depth.stream
         if next_norm is None:
             return stream
-        return stream, (n if isinstance(next_norm, RMSNorm) else next_norm(stream, step.act_dtype))
+        return stream, (n if isinstance(next_norm, (RMSNorm, NormThenConv)) else next_norm(stream, step.act_dtype))
 
     def forward(self, resid: torch.Tensor, step, line, normed=None, next_norm=None):
         """Returns the residual stream, or (residual stream, next_norm(residual stream)) when
         ``next_norm`` (an RMSNorm) is given."""
         nm = self.norms
         act = step.act_dtype
-        n = normed if normed is not None else nm["pre_mixer"](resid, act)
         if self.general:
+            n = normed if normed is not None else self.entry(step, line)(resid, act)
             return self._forward_general(resid, step, line, n, next_norm)
+        n = normed if normed is not None else nm["pre_mixer"](resid, act)
         y = self.mixer.forward(n, step, line)
         if isinstance(nm["post_mixer"], RMSNorm) and isinstance(nm["pre_ff"], RMSNorm):
             n = nm["post_mixer"].add_to(resid, y, then=nm["pre_ff"], out_dtype=act)

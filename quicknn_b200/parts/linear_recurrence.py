@@ -22,6 +22,7 @@ from .linear import project, stack_rows
 from .spec import PartSpec
 
 DECAY = 8.0
+STEP_MAX_ROWS = 64             # decode rows up to which the whole step is one kernel (it forms u once per 32 channels of a part)
 
 
 @MIXERS.register("rglru")
@@ -76,23 +77,33 @@ class RealGatedRecurrence(Mixer):
     def state_need(self) -> Optional[StateNeed]:
         return StateNeed((self.taps + 1, self.width), "float32")
 
-    def before_output(self, x: torch.Tensor, step, line, scale: float = 1.0, out: Optional[torch.Tensor] = None,
-                      out_col0: int = 0) -> torch.Tensor:
-        """scale * S * y: what the output matrix multiplies, into the columns ``out_col0 ..`` of ``out`` when given."""
+    def input_matrix(self) -> torch.Tensor:
+        """What multiplies the input, for a mixer that stacks it with its other branches'."""
+        return self.w_in
+
+    def release_inputs(self) -> None:
+        """Forget the input matrix: it lives on in the stacked one."""
+        self.w_in = None
+
+    def before_output(self, p: torch.Tensor, col0: int, step, line, scale: float, out: torch.Tensor, out_col0: int) -> torch.Tensor:
+        """scale * S * y: what the output matrix multiplies, into the columns ``out_col0 ..`` of ``out``.  p: rows whose columns
+        from ``col0`` on are the input times ``input_matrix`` (y | x)."""
         D = self.width
         decode = step.mode == "decode"
+        if decode and step.n_seqs <= STEP_MAX_ROWS and ops.recurrent_step(
+                p, col0, col0 + D, self.x_bias, self.y_bias, self.conv, self.conv_bias, self.w_gates, self.r_bias, self.i_bias,
+                self.decay, line.state, step.tok_pos, step.slots, scale, out, out_col0):
+            return out
         row0, lens = (None, None) if decode else (step.seq_row0, step.seq_len)
         longest = 1 if decode else step.max_q_len
-        p = project(x, self.w_in)                                                            # y | x
-        u = ops.causal_conv(p, self.conv, line.state, row0, lens, step.tok_pos, step.slots, step.n_seqs, longest, col0=D,
+        u = ops.causal_conv(p, self.conv, line.state, row0, lens, step.tok_pos, step.slots, step.n_seqs, longest, col0=col0 + D,
                             x_bias=self.x_bias, out_bias=self.conv_bias)
         ug = u if u.dtype == self.w_gates.dtype else ops.cast(u, self.w_gates.dtype)
         z = ops.block_linear(ug, self.w_gates, out_dtype=torch.float32)                      # the gates' logits, float32
-        if out is None:
-            out, out_col0 = torch.empty((x.shape[0], D), dtype=x.dtype, device=x.device), 0
         return ops.linear_recurrence(z, self.r_bias, self.i_bias, self.decay, u, self.part, line.state, self.taps * D, row0,
-                                     lens, step.slots, step.n_seqs, longest, y=p, y_bias=self.y_bias, scale=scale, out=out,
-                                     out_col0=out_col0)
+                                     lens, step.slots, step.n_seqs, longest, y=p, y_col0=col0, y_bias=self.y_bias, scale=scale,
+                                     out=out, out_col0=out_col0)
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
-        return project(self.before_output(x, step, line), self.w_o)
+        out = torch.empty((x.shape[0], self.width), dtype=x.dtype, device=x.device)
+        return project(self.before_output(project(x, self.w_in), 0, step, line, 1.0, out, 0), self.w_o)

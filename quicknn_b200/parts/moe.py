@@ -159,7 +159,14 @@ class RoutedExperts(FeedForward):
                                                        self.w_shared_gate) if w is not None)
         return n + (self.shared.weight_bytes() if self.shared is not None else 0)
 
-    def forward(self, x: torch.Tensor, step) -> torch.Tensor:
+    def forward_terms(self, x: torch.Tensor, step) -> Tuple[torch.Tensor, int]:
+        """(rows, n): the output is the sum of n rows each, for whoever can sum them in a kernel of its own; n = 1 where the
+        sum is formed here (a shared expert, identity experts)."""
+        if self.shared is not None or self.identity > 0:
+            return self.forward(x, step), 1
+        return self.forward(x, step, summed=False), self.top
+
+    def forward(self, x: torch.Tensor, step, summed: bool = True) -> torch.Tensor:
         if self.w_router_and_gate is not None:
             sel_e, sel_w, gate = ops.moe_route(x, self.w_router_and_gate, self.top, self.score, self.renormalize,
                                                self.correction, self.route_scale, extra=1, groups=self.groups)
@@ -172,4 +179,4 @@ class RoutedExperts(FeedForward):
         act = ops.GATED_CLAMPED if self.activation == "clamped" else ops.ACT_CODES[self.activation]
         return ops.moe_experts(xe, sel_e, sel_w, self.top, self.w_gate_up, self.w_down, act, self.limit,
                                self.alpha, self.weight_on_input, shared, shared_gate=gate, identity=self.identity > 0,
-                               gated=self.gated)
+                               gated=self.gated, summed=summed)

@@ -7,8 +7,9 @@ or, with ``scales`` = {branch: number}, the outputs are summed with fixed number
 
     y = sum_b  scale_b branch_b(x)
 
-which is one product: the branches leave what their output matrices multiply, already scaled (``before_output``), side by side
-in one row, and the output matrices are stacked along their inner size.
+which is two products: the branches' input matrices are stacked (``input_matrix``), every branch works on its columns of the
+product's rows, and the branches leave what their output matrices multiply, already scaled, side by side in one row
+(``before_output``), the output matrices being stacked along their inner size.
 
 ``branches`` maps a name to the branch's ``PartSpec`` (any registered mixer); the branch's parameters are this mixer's
 ``<name>.<parameter>`` and its weight ``<name>.out``.  The branches share one cache line: at most one of them may keep
@@ -23,7 +24,7 @@ import torch
 
 from ..kernels import ops
 from .base import MIXERS, CacheNeed, Mixer, StateNeed
-from .linear import project
+from .linear import project, stack_rows
 from .spec import PartSpec
 
 
@@ -45,7 +46,9 @@ class ParallelMixer(Mixer):
         self.out_weights: List[torch.Tensor] = []
         scales = p.get("scales")
         self.scales: Optional[List[float]] = None if scales is None else [float(scales[n]) for n in self.names]
-        self.w_o: Optional[torch.Tensor] = None          # with scales: the branches' output matrices side by side
+        self.w_in: Optional[torch.Tensor] = None         # with scales: the branches' input matrices one below the other
+        self.w_o: Optional[torch.Tensor] = None          # and their output matrices side by side
+        self.in_cols: List[int] = []
         if self.scales is not None and not all(hasattr(b, "before_output") for b in self.branches):
             raise ValueError("parallel: branches with fixed scales offer their rows before the output product")
 
@@ -72,11 +75,16 @@ class ParallelMixer(Mixer):
             ws = [b.w_o for b in self.branches]
             wide = torch.float32 if any(w.dtype == torch.float32 for w in ws) else ws[0].dtype
             self.w_o = torch.cat([w.to(wide) for w in ws], dim=1).contiguous()
-            for b in self.branches:                      # a branch's output matrix is a range of this one's columns
+            ins = [b.input_matrix() for b in self.branches]
+            self.in_cols = [sum(w.shape[0] for w in ins[:i]) for i in range(len(ins))]
+            pad = torch.zeros(((-sum(w.shape[0] for w in ins)) % 8, self.hidden), dtype=ins[0].dtype, device=ins[0].device)
+            self.w_in = stack_rows(ins + [pad])          # rows of whole 16-byte pieces
+            for b in self.branches:                      # the branches' own matrices are ranges of these from here on
                 b.w_o = None
+                b.release_inputs()
 
     def weight_bytes(self) -> int:
-        own = self.out_weights + ([self.w_o] if self.w_o is not None else [])
+        own = self.out_weights + ([self.w_in, self.w_o] if self.w_o is not None else [])
         return sum(b.weight_bytes() for b in self.branches) + sum(w.numel() * w.element_size() for w in own)
 
     def cache_need(self) -> Optional[CacheNeed]:
@@ -103,10 +111,11 @@ class ParallelMixer(Mixer):
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
         if self.scales is not None:
+            p = project(x, self.w_in)
             rows = torch.empty((x.shape[0], self.w_o.shape[1]), dtype=x.dtype, device=x.device)
             col = 0
-            for b, s in zip(self.branches, self.scales):
-                b.before_output(x, step, line, s, rows, col)
+            for b, s, c in zip(self.branches, self.scales, self.in_cols):
+                b.before_output(p, c, step, line, s, rows, col)
                 col += b.out_width
             return project(rows, self.w_o)
         return ops.mean_rmsnorm(self.forward_branches(x, step, line), self.out_weights, self.eps, x.dtype)
