@@ -8,8 +8,9 @@
 // tap that falls before the step's first row comes from the ring, any other from the step's rows.  Sums are float32 in
 // the order of the taps, so they do not depend on how a sequence was cut into steps.
 //
-// A thread owns VEC channels of `rows` consecutive rows of one sequence.  The threads of a sequence's first tile read the
-// ring (tiles have at least taps - 1 rows) and, after that, write the same channels' new rows into it.
+// A thread owns VEC channels of `rows` consecutive rows of one sequence; it asks for all of a tile's rows before it uses the
+// first.  The threads of a sequence's first tile read the ring (tiles have at least taps - 1 rows) and, after that, write
+// the same channels' new rows into it.
 #include "common.cuh"
 
 using namespace qnn;
@@ -29,23 +30,39 @@ __device__ __forceinline__ void store_v(void* p, int dt, size_t i, const float* 
     else store_from_f(p, dt, i, v[0]);
 }
 
-// TAPS > 0: the number of taps is known here and the filter and the last inputs stay in registers; 0: any number, taps are
-// read again for every row.
-template <int VEC, int TAPS>
+// TAPS > 0: the number of taps and of rows per tile (ROWS) is known here, and the filter and the tile's inputs stay in
+// registers; 0: any numbers, inputs are read again for every tap.
+template <int VEC, int TAPS, int ROWS>
 __global__ void __launch_bounds__(THREADS)
 causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const void* __restrict__ x_bias, int xb_dt,
                    const void* __restrict__ w, int w_dt, const void* __restrict__ out_bias, int ob_dt, int add_input,
                    void* __restrict__ out, int out_dt, long long ldo, float* state, long long slot_stride, int C, int taps_,
                    const int* __restrict__ seq_row0, const int* __restrict__ seq_len, const int* __restrict__ tok_pos,
-                   const int* __restrict__ slots, int rows) {
+                   const int* __restrict__ slots, int rows_) {
+    const int taps = TAPS > 0 ? TAPS : taps_, rows = TAPS > 0 ? ROWS : rows_;
+    const int b = blockIdx.y;
+    const int groups = (C + VEC - 1) / VEC;                 // of channels; consecutive threads take consecutive groups
+    const unsigned at = blockIdx.x * (unsigned)THREADS + threadIdx.x;
+    const int tile = (int)(at / (unsigned)groups), c0 = (int)(at - (unsigned)tile * groups) * VEC;
+    const int r0 = tile * rows;                             // first row of this tile within the sequence
+    float wv[TAPS > 0 ? TAPS : 1][VEC], xb[VEC], ob[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) xb[e] = ob[e] = 0.f;
+    // filters and biases are written by no kernel of the step: asked for before the wait for the kernel in front
+    if (x_bias != nullptr) load_v<VEC>(x_bias, xb_dt, c0, xb);
+    if (out_bias != nullptr) load_v<VEC>(out_bias, ob_dt, c0, ob);
+    if constexpr (TAPS > 0) {
+        float flat[TAPS * VEC];                             // [channel][tap], VEC * TAPS numbers in a row
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) load_v<VEC>(w, w_dt, (size_t)c0 * TAPS + i * VEC, flat + i * VEC);
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) wv[j][e] = flat[e * TAPS + j];
+    }
     pdl_wait();
-    const int taps = TAPS > 0 ? TAPS : taps_;
-    const int b = blockIdx.z;
-    const int c0 = (blockIdx.x * THREADS + threadIdx.x) * VEC;
-    if (c0 >= C) return;
     const int row0 = seq_row0 != nullptr ? seq_row0[b] : b;
     const int n = seq_len != nullptr ? seq_len[b] : 1;
-    const int r0 = blockIdx.y * rows;                       // first row of this tile within the sequence
     if (r0 >= n) return;
     const int r1 = min(r0 + rows, n);
     const int slot = slots[b];
@@ -58,11 +75,6 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
     }
     const int first = tok_pos[row0];                        // position of the sequence's first row of this step
     float* ring = state + (size_t)slot * slot_stride + c0;
-    float xb[VEC], ob[VEC];
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) xb[e] = ob[e] = 0.f;
-    if (x_bias != nullptr) load_v<VEC>(x_bias, xb_dt, c0, xb);
-    if (out_bias != nullptr) load_v<VEC>(out_bias, ob_dt, c0, ob);
     // v of row r (may be negative: an earlier step's, or before the sequence)
     auto input = [&](int r, float* v) {
         if (r >= 0) {
@@ -79,29 +91,25 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
         }
     };
     if constexpr (TAPS > 0) {
-        float wv[TAPS][VEC], last[TAPS][VEC];
+        float v[ROWS + TAPS - 1][VEC];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j)
+        for (int i = 0; i < ROWS + TAPS - 1; ++i) {
+            const int r = r0 - TAPS + 1 + i;
+            if (r < r1) input(r, v[i]);
+        }
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) wv[j][e] = load_as_f(w, w_dt, (size_t)(c0 + e) * TAPS + j);
-#pragma unroll
-        for (int j = 1; j < TAPS; ++j) input(r0 - TAPS + j, last[j]);
-        for (int r = r0; r < r1; ++r) {
-#pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j)
-#pragma unroll
-                for (int e = 0; e < VEC; ++e) last[j][e] = last[j + 1][e];
-            input(r, last[TAPS - 1]);
+        for (int i = 0; i < ROWS; ++i) {
+            if (r0 + i >= r1) continue;
             float acc[VEC];
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
                 acc[e] = 0.f;
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], last[j][e], acc[e]);
+                for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], v[i + j][e], acc[e]);
                 acc[e] += ob[e];
-                if (add_input) acc[e] += last[TAPS - 1][e];
+                if (add_input) acc[e] += v[i + TAPS - 1][e];
             }
-            store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, acc);
+            store_v<VEC>(out, out_dt, (size_t)(row0 + r0 + i) * ldo + c0, acc);
         }
     } else {
         for (int r = r0; r < r1; ++r) {
@@ -118,7 +126,7 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
             store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, acc);
         }
     }
-    if (blockIdx.y == 0) {
+    if (r0 == 0) {
         for (int r = max(0, n - taps); r < n; ++r) {
             float v[VEC];
             input(r, v);
@@ -142,23 +150,25 @@ QNN_API int qnn_causal_conv(const void* x, int x_dt, long long ldx, const void* 
     if (C <= 0 || taps < 1 || n_seqs > 65535 || ldx < C || ldo < C || slot_stride < (long long)taps * C) return QNN_ERR_ARGUMENT;
     const int xs = x_dt == QNN_DT_BF16 ? 2 : 4, os = out_dt == QNN_DT_BF16 ? 2 : 4;
     const bool vec = C % 8 == 0 && (ldx * xs) % 16 == 0 && (ldo * os) % 16 == 0 &&
-                     (((uintptr_t)x | (uintptr_t)out | (uintptr_t)x_bias | (uintptr_t)out_bias) & 15) == 0;
-    int rows = longest > 1 ? 16 : 1;
-    if (rows < taps) rows = taps;
-    while ((long long)(longest + rows - 1) / rows > 65535) rows *= 2;
-    const int per = THREADS * (vec ? 8 : 1);
-    const dim3 grid((C + per - 1) / per, (longest + rows - 1) / rows, n_seqs);
-#define QNN_CONV(V, TP)                                                                                                \
-    launch_pdl(causal_conv_kernel<V, TP>, grid, dim3(THREADS), 0, st, x, x_dt, ldx, x_bias, xb_dt, w, w_dt, out_bias,   \
+                     (((uintptr_t)x | (uintptr_t)out | (uintptr_t)x_bias | (uintptr_t)out_bias | (uintptr_t)w) & 15) == 0;
+    const bool known = vec && taps >= 2 && taps <= 4;
+    int rows = longest > 1 ? 8 : 1;
+    if (!known && rows < taps) rows = taps;
+    const long long work = (long long)((longest + rows - 1) / rows) * ((C + (vec ? 7 : 0)) / (vec ? 8 : 1));
+    if (work + THREADS > 0xffffffffLL) return QNN_ERR_UNSUPPORTED;
+    const dim3 grid((unsigned)((work + THREADS - 1) / THREADS), n_seqs);
+#define QNN_CONV(V, TP, R)                                                                                             \
+    launch_pdl(causal_conv_kernel<V, TP, R>, grid, dim3(THREADS), 0, st, x, x_dt, ldx, x_bias, xb_dt, w, w_dt, out_bias, \
                ob_dt, add_input, out, out_dt, ldo, state, slot_stride, C, taps, seq_row0, seq_len, tok_pos, slots, rows)
-    if (vec) {
-        if (taps == 4) QNN_CONV(8, 4);
-        else if (taps == 3) QNN_CONV(8, 3);
-        else if (taps == 2) QNN_CONV(8, 2);
-        else QNN_CONV(8, 0);
-    } else {
-        QNN_CONV(1, 0);
-    }
+#define QNN_CONV_TAPS(R)               \
+    if (taps == 4) QNN_CONV(8, 4, R);  \
+    else if (taps == 3) QNN_CONV(8, 3, R); \
+    else QNN_CONV(8, 2, R);
+    if (known && rows == 8) { QNN_CONV_TAPS(8) }
+    else if (known) { QNN_CONV_TAPS(1) }
+    else if (vec) QNN_CONV(8, 0, 1);
+    else QNN_CONV(1, 0, 1);
+#undef QNN_CONV_TAPS
 #undef QNN_CONV
     QNN_LAUNCH_CHECK();
 }

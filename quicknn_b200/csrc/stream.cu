@@ -35,69 +35,85 @@ struct Update {
     float mult, eps_post, off_post, eps_next, off_next;
 };
 
-// h = n + conv(n) of 8 columns from column c on, n already rounded as it is stored; the row's n joins the ring.
-__device__ __forceinline__ void conv8(const Update& u, int t, int c, float* n) {
-    const int slot = u.slots[t], pos = u.tok_pos[t];
-    if (slot < 0) return;
-    float* ring = u.ring + (size_t)slot * u.slot_stride + c;
-    float acc[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
-    for (int j = 0; j < u.taps; ++j) {
-        const int q = pos - u.taps + 1 + j;
-        if (q < 0) continue;
-        float x[8];
-        if (q == pos) {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = n[e];
-        } else {
-            load8_as_f(ring + (size_t)(q % u.taps) * u.H, QNN_DT_F32, 0, x);
-        }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(load_as_f(u.conv, u.conv_dt, (size_t)(c + e) * u.taps + j), x[e], acc[e]);
-    }
-    store8_from_f(ring + (size_t)(pos % u.taps) * u.H, QNN_DT_F32, 0, n);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) n[e] += acc[e];
-}
-
-template <int CH>
-__global__ void stream_update_vec_kernel(const Update u) {
+// TAPS > 0: h = n + conv(n), that many taps, of the normed row n (rounded as it is stored), a row per sequence; the row's n joins the ring.
+// What waits for no sum (weights before the wait for the kernel in front; the ring's earlier rows; the earlier layers' rows,
+// summed in the order of the layers) is asked for before the first sum.
+constexpr int MAX_TAPS = 4;
+template <int TAPS>
+__global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kernel(const Update u) {
+    constexpr bool CONV = TAPS > 0;
+    constexpr int CH = 1;             // groups of eight columns per thread
     __shared__ float red[32];
     const size_t base = (size_t)blockIdx.x * u.H;
     const int nchunks = u.H >> 3;
-    float g1[CH][8], v[CH][8], r[CH][8];
+    float g1[CH][8], g2[CH][8], v[CH][8], r[CH][8], z[CH][8];
+    float wv[CONV ? TAPS * 8 : 1], prev[TAPS > 1 ? TAPS - 1 : 1][8];
+    const bool in0 = (int)threadIdx.x < nchunks;
 #pragma unroll
     for (int i = 0; i < CH; ++i) {                       // weights are written by no kernel of the step
         const int c = threadIdx.x + i * blockDim.x;
-        if (c < nchunks) load8_as_f(u.w_post, u.wp_dt, (size_t)c * 8, g1[i]);
+        if (c < nchunks) {
+            load8_as_f(u.w_post, u.wp_dt, (size_t)c * 8, g1[i]);
+            if (u.out_next != nullptr) load8_as_f(u.w_next, u.wn_dt, (size_t)c * 8, g2[i]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) g1[i][e] = g2[i][e] = 0.f;
+        }
     }
+    int slot = -1, pos = 0;
+    float* ring = nullptr;
+    if constexpr (CONV) {                                // CH = 1; [channel][tap], taps * 8 numbers in a row
+        slot = u.slots[blockIdx.x];
+        pos = u.tok_pos[blockIdx.x];
+        ring = u.ring + (size_t)(slot < 0 ? 0 : slot) * u.slot_stride + threadIdx.x * 8;
+        if (in0)
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) load8_as_f(u.conv, u.conv_dt, (size_t)threadIdx.x * 8 * TAPS + j * 8, wv + j * 8);
+    }
+    const float a_last = u.hist != nullptr ? load_as_f(u.numbers, u.num_dt, u.n_hist) : 1.f;
     pdl_wait();
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = r[i][e] = z[i][e] = 0.f;
         if (c < nchunks) {
-            const size_t yat = (size_t)blockIdx.x * u.terms * u.H + (size_t)c * 8;
+            const size_t yat = (size_t)blockIdx.x * u.terms * u.H + (size_t)c * 8, at = base + (size_t)c * 8;
             load8_as_f(u.y, u.y_dt, yat, v[i]);
+            load8_as_f(u.resid, QNN_DT_F32, at, r[i]);
             for (int k = 1; k < u.terms; ++k) {
-                float z[8];
-                load8_as_f(u.y, u.y_dt, yat + (size_t)k * u.H, z);
+                float t[8];
+                load8_as_f(u.y, u.y_dt, yat + (size_t)k * u.H, t);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) v[i][e] += z[e];
+                for (int e = 0; e < 8; ++e) v[i][e] += t[e];
             }
-            load8_as_f(u.resid, QNN_DT_F32, base + (size_t)c * 8, r[i]);
-        } else {
+            if (u.hist != nullptr) {
+#pragma unroll 4
+                for (int j = 0; j < u.n_hist; ++j) {
+                    float h[8];
+                    load8_as_f(u.hist, QNN_DT_F32, (size_t)j * u.hist_stride + at, h);
+                    const float a = load_as_f(u.numbers, u.num_dt, j);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v[i][e] = r[i][e] = g1[i][e] = 0.f;
+                    for (int e = 0; e < 8; ++e) z[i][e] = fmaf(a, h[e], z[i][e]);
+                }
+            }
         }
 #pragma unroll
         for (int e = 0; e < 8; ++e) ss += v[i][e] * v[i][e];
     }
+    if constexpr (CONV) {
+#pragma unroll
+        for (int d = 1; d < TAPS; ++d) {                 // prev[d - 1]: the row d positions back
+            if (in0 && slot >= 0 && pos - d >= 0) load8_as_f(ring + (size_t)((pos - d) % TAPS) * u.H, QNN_DT_F32, 0, prev[d - 1]);
+            else
+#pragma unroll
+                for (int e = 0; e < 8; ++e) prev[d - 1][e] = 0.f;
+        }
+    }
     ss = block_sum(ss, red);
     const float inv = rsqrtf(ss / (float)u.H + u.eps_post);
     float ss2 = 0.f;
-    const float a_last = u.hist != nullptr ? load_as_f(u.numbers, u.num_dt, u.n_hist) : 1.f;
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
@@ -107,19 +123,8 @@ __global__ void stream_update_vec_kernel(const Update u) {
         for (int e = 0; e < 8; ++e) r[i][e] += u.mult * (v[i][e] * inv * (g1[i][e] + u.off_post));
         store8_from_f(u.resid_out, QNN_DT_F32, at, r[i]);
         if (u.hist != nullptr) {
-            float z[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) z[e] = 0.f;
-#pragma unroll 4
-            for (int j = 0; j < u.n_hist; ++j) {
-                float h[8];
-                load8_as_f(u.hist, QNN_DT_F32, (size_t)j * u.hist_stride + at, h);
-                const float a = load_as_f(u.numbers, u.num_dt, j);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) z[e] = fmaf(a, h[e], z[e]);
-            }
-#pragma unroll
-            for (int e = 0; e < 8; ++e) r[i][e] = fmaf(a_last, r[i][e], z[e]);
+            for (int e = 0; e < 8; ++e) r[i][e] = fmaf(a_last, r[i][e], z[i][e]);
             store8_from_f(u.avg_out, QNN_DT_F32, at, r[i]);
         }
 #pragma unroll
@@ -131,19 +136,29 @@ __global__ void stream_update_vec_kernel(const Update u) {
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
-        if (c < nchunks) {
-            float g2[8], o[8];
-            load8_as_f(u.w_next, u.wn_dt, (size_t)c * 8, g2);
+        if (c >= nchunks) continue;
+        float o[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (g2[e] + u.off_next);
-            if (u.conv != nullptr) {
+        for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (g2[i][e] + u.off_next);
+        if constexpr (CONV) {
+            if (slot >= 0) {
                 if (u.out_dt == QNN_DT_BF16)
 #pragma unroll
                     for (int e = 0; e < 8; ++e) o[e] = __bfloat162float(__float2bfloat16_rn(o[e]));
-                conv8(u, blockIdx.x, c * 8, o);
+                store8_from_f(ring + (size_t)(pos % TAPS) * u.H, QNN_DT_F32, 0, o);
+                float acc[8];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll
+                for (int d = TAPS - 1; d >= 0; --d)      // the oldest tap first
+#pragma unroll
+                    for (int e = 0; e < 8; ++e)
+                        acc[e] = fmaf(wv[e * TAPS + (TAPS - 1 - d)], d == 0 ? o[e] : prev[d > 0 ? d - 1 : 0][e], acc[e]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[e] += acc[e];
             }
-            store8_from_f(u.out_next, u.out_dt, base + (size_t)c * 8, o);
         }
+        store8_from_f(u.out_next, u.out_dt, base + (size_t)c * 8, o);
     }
 }
 
@@ -191,8 +206,8 @@ __global__ void stream_update_kernel(const Update u) {
 
 // resid may be resid_out (in place).  hist (null: no average): rows of n_hist earlier layers, hist_stride floats from one
 // layer's rows to the next's; numbers: n_hist + 1 of them, the last one for X; avg_out may be resid but not resid_out.
-// w_next / out_next null: no norm follows.  terms: rows of y per row, summed.  conv (null: none; needs out_next and rows of
-// whole eights on 16 bytes, else QNN_ERR_UNSUPPORTED): row t is the next token, at tok_pos[t], of the sequence in slots[t].
+// w_next / out_next null: no norm follows.  terms: rows of y per row, summed.  conv (null: none; needs out_next, rows of
+// whole eights on 16 bytes, at most 4096 columns and four taps, else QNN_ERR_UNSUPPORTED): row t is the next token, at tok_pos[t], of the sequence in slots[t].
 QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, int terms, float mult, const void* w_post, int wp_dt,
                               float eps_post, int unit_post, float* resid_out, const float* hist, long long hist_stride,
                               int n_hist, const void* numbers, int num_dt, float* avg_out, const void* w_next, int wn_dt,
@@ -214,12 +229,17 @@ QNN_API int qnn_stream_update(const float* resid, const void* y, int y_dt, int t
     u.tok_pos = tok_pos; u.slots = slots;
     const uintptr_t all = (uintptr_t)resid | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)resid_out |
                           (uintptr_t)hist | (uintptr_t)avg_out | (uintptr_t)out_next | (uintptr_t)ring;
-    if ((H & 7) == 0 && (all & 15) == 0 && (hist_stride & 3) == 0 && (slot_stride & 3) == 0 && H <= 8 * 2 * 1024) {
-        const int chunks = H >> 3;
-        const int ch = chunks > 1024 ? 2 : 1;
-        const int threads = (((chunks + ch - 1) / ch) + 31) / 32 * 32;
-        if (ch == 1) launch_pdl(stream_update_vec_kernel<1>, dim3(T), dim3(threads), 0, st, u);
-        else launch_pdl(stream_update_vec_kernel<2>, dim3(T), dim3(threads), 0, st, u);
+    if ((H & 7) == 0 && (all & 15) == 0 && (hist_stride & 3) == 0 && (slot_stride & 3) == 0 && H <= 8 * 1024) {
+        const int threads = ((H >> 3) + 31) / 32 * 32;
+        if (conv != nullptr) {
+            if (threads > 512 || taps > MAX_TAPS || ((uintptr_t)conv & 15)) return QNN_ERR_UNSUPPORTED;
+            if (taps == 4) launch_pdl(stream_update_vec_kernel<4>, dim3(T), dim3(threads), 0, st, u);
+            else if (taps == 3) launch_pdl(stream_update_vec_kernel<3>, dim3(T), dim3(threads), 0, st, u);
+            else if (taps == 2) launch_pdl(stream_update_vec_kernel<2>, dim3(T), dim3(threads), 0, st, u);
+            else launch_pdl(stream_update_vec_kernel<1>, dim3(T), dim3(threads), 0, st, u);
+        } else {
+            launch_pdl(stream_update_vec_kernel<0>, dim3(T), dim3(threads), 0, st, u);
+        }
         QNN_LAUNCH_CHECK();
     }
     if (conv != nullptr) return QNN_ERR_UNSUPPORTED;

@@ -268,8 +268,9 @@ class OpTimer:
             byts = float(x.shape[0] * w.shape[0] * w.shape[2] * x.element_size() + _nbytes(w) + _nbytes(out)
                          + (x.shape[0] * w.shape[0] * w.shape[1] * gate.element_size() if gate is not None else 0))
         elif name == "linear_recurrence":
-            z, u, y = a[0], a[4], kw.get("y")
-            byts = float(_nbytes(z) + 2 * _nbytes(u) + (_nbytes(u) if y is not None else 0) + 2 * a[11] * u.shape[1] * 4)
+            u, w, y = a[0], a[1], kw.get("y")
+            flops = 2.0 * u.shape[0] * w.numel()
+            byts = float(_nbytes(w) + 2 * _nbytes(u) + (_nbytes(u) if y is not None else 0) + 2 * a[10] * u.shape[1] * 4)
         elif name == "recurrent_step":
             p, conv, w = a[0], a[5], a[7]
             C, rows = conv.shape[0], p.shape[0]

@@ -78,7 +78,10 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_block_linear": [c_vp, c_int, c_ll, c_ll, c_vp, c_int, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_int, c_int, c_int,
                          c_int, c_vp],
     "qnn_linear_recurrence": [c_vp, c_ll, c_vp, c_vp, c_int, c_vp, c_vp, c_int, c_ll, c_vp, c_int, c_ll, c_vp, c_int, c_float,
-                              c_vp, c_int, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_vp, c_vp],
+                              c_vp, c_int, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_int, c_int, c_vp, c_int,
+                              c_vp],
+    "qnn_recurrence_gates": [c_vp, c_ll, c_vp, c_vp, c_vp, c_vp, c_vp, c_ll, c_vp, c_ll, c_vp, c_vp, c_vp, c_vp, c_int, c_int,
+                             c_int, c_int, c_int, c_vp],
     "qnn_latent_prep": [c_vp, c_int, c_ll, c_int, c_int, c_vp, c_int, c_float, c_int, c_int, c_vp, c_vp, c_ll, c_vp, c_ll,
                         c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_int, c_int, c_vp],
     "qnn_small_linear_f32": [c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_int, c_vp, c_int, c_float, c_vp],

@@ -1854,25 +1854,28 @@ def block_linear(x: torch.Tensor, w: torch.Tensor, *, col0: int = 0, step: Optio
     return out
 
 
-RECURRENCE_SEGMENT = 64       # rows of a segment when sequences are walked in segments side by side; at most 64 segments
+RECURRENCE_SEGMENT = 32       # rows of a segment when sequences are walked in segments side by side
+RECURRENCE_GATES_FUSED = True
 
 
-def linear_recurrence(z: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, decay: torch.Tensor, u: torch.Tensor,
-                      part: int, state: torch.Tensor, state_col0: int, seq_row0: Optional[torch.Tensor],
-                      seq_len: Optional[torch.Tensor], slots: torch.Tensor, n_seqs: int, longest: int = 1, *,
-                      y: Optional[torch.Tensor] = None, y_col0: int = 0, y_bias: Optional[torch.Tensor] = None,
-                      scale: float = 1.0, out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
-    """S_t = a S_(t-1) + sqrt(1 - a^2) i u_t with r, i = sigmoid of the logits plus biases and a = exp(-decay r), from the
-    state of every sequence's slot and back into it; returns scale * S * gelu(y + y_bias) (scale * S without ``y``).
-    z: float32 [rows, 2C] logits, per part of ``part`` channels first r's, then i's (overwritten for long sequences).
-    ``state``: float32 [slots, n], the channels' numbers from ``state_col0`` on."""
-    _req(z, "z", torch.float32, 2)
+def linear_recurrence(u: torch.Tensor, w_gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor, decay: torch.Tensor,
+                      state: torch.Tensor, state_col0: int, seq_row0: Optional[torch.Tensor], seq_len: Optional[torch.Tensor],
+                      slots: torch.Tensor, n_seqs: int, longest: int = 1, *, y: Optional[torch.Tensor] = None, y_col0: int = 0,
+                      y_bias: Optional[torch.Tensor] = None, scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                      out_col0: int = 0) -> torch.Tensor:
+    """S_t = a S_(t-1) + sqrt(1 - a^2) i u_t, r and i the sigmoids of block-diagonal products of u plus biases, a = exp(-decay r),
+    from the state of every sequence's slot and back into it; returns scale * S * gelu(y + y_bias) (scale * S without ``y``).
+    ``w_gates``: [blocks, 2 * part, part], per part r's rows, then i's; the biases float32 [C].  ``state``: float32 [slots, n],
+    the channels' numbers from ``state_col0`` on.  Sequences of more than 32 rows are walked in segments side by side;
+    results differ from the walk in one piece by rounding only."""
     _req(u, "u", None, 2)
-    _req(decay, "decay", torch.float32, 1)
+    _req(w_gates, "w_gates", None, 3)
+    for t, what in ((decay, "decay"), (r_bias, "r_bias"), (i_bias, "i_bias")):
+        _req(t, what, torch.float32, 1)
     _req(state, "state", torch.float32)
     T, C = u.shape
-    if tuple(z.shape) != (T, 2 * C) or decay.numel() != C or r_bias.numel() != C or i_bias.numel() != C or C % part \
-            or r_bias.dtype != i_bias.dtype:
+    B, _, part = w_gates.shape
+    if B * part != C or w_gates.shape[1] != 2 * part or decay.numel() != C or r_bias.numel() != C or i_bias.numel() != C:
         raise ValueError("linear_recurrence: shapes do not agree")
     if state[0].numel() < state_col0 + C or slots.numel() < n_seqs or (seq_row0 is None and T < n_seqs):
         raise ValueError("linear_recurrence: the state does not fit, or fewer rows than sequences")
@@ -1882,19 +1885,33 @@ def linear_recurrence(z: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tenso
         out, out_col0 = torch.empty((T, C), dtype=u.dtype, device=u.device), 0
     if out.shape[0] != T or out_col0 + C > out.shape[1]:
         raise ValueError("linear_recurrence: the result does not fit")
+    L = _lib.load()
     longest = int(longest) if seq_row0 is not None else 1
     seg = RECURRENCE_SEGMENT
-    while -(-longest // seg) > 64:
-        seg *= 2
-    nseg = -(-longest // seg) if longest > 2 * seg else 1
-    seg = seg if nseg > 1 else max(1, longest)
+    nseg = max(1, -(-longest // seg))
     scratch = torch.empty((n_seqs, nseg, 3, C), dtype=torch.float32, device=u.device) if nseg > 1 else None
-    _lib.check(_lib.load().qnn_linear_recurrence(
-        _p(z), z.shape[1], _p(r_bias), _p(i_bias), dt_code(r_bias), _p(decay), _p(u), dt_code(u), C,
+    state_ptr = ctypes.c_void_p(state.data_ptr() + 4 * state_col0)
+    z = None
+    if nseg > 1 and RECURRENCE_GATES_FUSED and u.dtype == torch.bfloat16 and w_gates.dtype == torch.bfloat16:
+        # the gates' product and the first pass over the segments in one kernel
+        z = torch.empty((T, 2 * C), dtype=torch.float32, device=u.device)
+        code = L.qnn_recurrence_gates(_p(u), C, _p(w_gates), _p(r_bias), _p(i_bias), _p(decay), _p(z), 2 * C, state_ptr,
+                                      state.stride(0), _p(scratch), _p(seq_row0), _p(seq_len), _p(slots), n_seqs, longest, C,
+                                      part, nseg, _stream())
+        if code == _lib.ERR_UNSUPPORTED:
+            z = None
+        else:
+            _lib.check(code, "recurrence_gates")
+    done = z is not None
+    if z is None:
+        z = block_linear(u if u.dtype == w_gates.dtype else cast(u, w_gates.dtype), w_gates, out_dtype=torch.float32)
+    _lib.check(L.qnn_linear_recurrence(
+        _p(z), 2 * C, _p(r_bias), _p(i_bias), F32, _p(decay), _p(u), dt_code(u), C,
         _col_ptr(y, y_col0) if y is not None else None, dt_code(y) if y is not None else 0, y.shape[1] if y is not None else 0,
         _p(y_bias), dt_code(y_bias) if y_bias is not None else 0, float(scale), _col_ptr(out, out_col0), dt_code(out),
-        out.shape[1], ctypes.c_void_p(state.data_ptr() + 4 * state_col0), state.stride(0), _p(seq_row0), _p(seq_len),
-        _p(slots), n_seqs, C, int(part), seg, nseg, _p(scratch), _stream()), "linear_recurrence", 2 if nseg > 1 else 1)
+        out.shape[1], state_ptr, state.stride(0), _p(seq_row0), _p(seq_len), _p(slots), n_seqs, C, part, seg if nseg > 1 else longest,
+        nseg, _p(scratch), int(done), _stream()), "linear_recurrence",
+        1 + (1 if nseg > 1 and not done else 0) + (1 if nseg > 64 else 0))
     return out
 
 

@@ -98,10 +98,8 @@ class RealGatedRecurrence(Mixer):
         longest = 1 if decode else step.max_q_len
         u = ops.causal_conv(p, self.conv, line.state, row0, lens, step.tok_pos, step.slots, step.n_seqs, longest, col0=col0 + D,
                             x_bias=self.x_bias, out_bias=self.conv_bias)
-        ug = u if u.dtype == self.w_gates.dtype else ops.cast(u, self.w_gates.dtype)
-        z = ops.block_linear(ug, self.w_gates, out_dtype=torch.float32)                      # the gates' logits, float32
-        return ops.linear_recurrence(z, self.r_bias, self.i_bias, self.decay, u, self.part, line.state, self.taps * D, row0,
-                                     lens, step.slots, step.n_seqs, longest, y=p, y_col0=col0, y_bias=self.y_bias, scale=scale,
+        return ops.linear_recurrence(u, self.w_gates, self.r_bias, self.i_bias, self.decay, line.state, self.taps * D, row0, lens,
+                                     step.slots, step.n_seqs, longest, y=p, y_col0=col0, y_bias=self.y_bias, scale=scale,
                                      out=out, out_col0=out_col0)
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
