@@ -2005,7 +2005,7 @@ def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: tor
         _req(hist, "hist", torch.float32, 3)
         _req(avg_out, "avg_out", torch.float32, 2)
         n = hist.shape[0]
-        if tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
+        if n < 1 or tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
             raise ValueError("stream_update: an average takes a number per earlier layer's rows and one for these")
     normed = torch.empty((T, H), dtype=out_dtype, device=resid.device) if w_next is not None else None
     cw = state = pos = slots = None
