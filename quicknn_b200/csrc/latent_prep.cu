@@ -31,6 +31,22 @@ __global__ void latent_prep_kernel(const T* __restrict__ a, long long lda, int c
     const int t = blockIdx.x, half = rot / 2;
     const int pos = tok_pos[t], slot = tok_slot[t];
     const T* row = a + (size_t)t * lda;
+    // what passes unturned from one buffer to the other waits for nothing below
+    const T* qr = q + (size_t)t * ldq;
+    T* qo = q_out + (size_t)t * ldo;
+    const bool in_place = q == q_out;
+    if (VEC && !in_place) {
+        constexpr int V = Vec16<T>::N;
+        const int cc = (hd - rot) / V;
+#pragma unroll 4
+        for (int i = threadIdx.x; i < H * cc; i += blockDim.x) {
+            const int h = i / cc;
+            const size_t at = (size_t)h * hd + rot + (i - h * cc) * V;
+            Vec16<T> v;
+            v.load(qr + at);
+            *reinterpret_cast<decltype(v.raw)*>(qo + at) = v.raw;
+        }
+    }
     float ss = 0.f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) {
         const float v = to_f(row[c_col + i]);
@@ -56,16 +72,13 @@ __global__ void latent_prep_kernel(const T* __restrict__ a, long long lda, int c
         key[i] = from_f<T>(v);
     }
     // the queries
-    const T* qr = q + (size_t)t * ldq;
-    T* qo = q_out + (size_t)t * ldo;
-    const bool in_place = q == q_out;
     if (VEC) {
         constexpr int V = Vec16<T>::N;
-        const int rc = half / V, cc = (hd - rot) / V, per = rc + (in_place ? 0 : cc);
-        for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
-            const int h = i / per, e = i - h * per;
+        const int rc = half / V;
+        for (int i = threadIdx.x; i < H * rc; i += blockDim.x) {
+            const int h = i / rc, e = i - h * rc;
             const size_t head = (size_t)h * hd;
-            if (e < rc) {
+            {
                 const int j = e * V;
                 Vec16<T> uv, xv;
                 uv.load(qr + head + j);
@@ -81,11 +94,6 @@ __global__ void latent_prep_kernel(const T* __restrict__ a, long long lda, int c
                 }
                 Vec16<T>::store(qo + head + j, p);
                 Vec16<T>::store(qo + head + half + j, s);
-            } else {
-                Vec16<T> v;
-                const int d = rot + (e - rc) * V;
-                v.load(qr + head + d);
-                *reinterpret_cast<decltype(v.raw)*>(qo + head + d) = v.raw;
             }
         }
     } else {

@@ -24,7 +24,7 @@ using namespace qnn;
 namespace {
 
 constexpr int THREADS = 128;
-constexpr int INLINE_PREFIX = 64;       // segments up to which a segment forms its own starting state
+constexpr int INLINE_PREFIX = 8;        // segments up to which a segment forms its own starting state
 
 struct Rec {
     float* z;                   // logits [rows][ldz]: channel c of block b = c / part: columns 2 b part + (c - b part), + part for i
@@ -42,7 +42,7 @@ struct Rec {
     const int* seq_len;
     const int* slots;
     long long ldz, ldu, ldy, ldo, slot_stride;
-    int b_dt, u_dt, y_dt, yb_dt, out_dt, C, part, seg, nseg, prefixed;
+    int b_dt, yb_dt, C, part, seg, nseg, prefixed;
     float scale;
 };
 
@@ -54,7 +54,8 @@ __device__ __forceinline__ float2 gates(float zr, float zi, float br, float bi, 
     return make_float2(expf(la), sqrtf(-expm1f(2.f * la)) * sigmoid_f(zi + bi) * u);
 }
 
-template <bool AGGREGATE>       // true: the first of the two kernels; false with nseg > 1: the second; nseg 1: the only one
+template <bool AGGREGATE, typename T>       // T: of u, y and out; AGGREGATE: the first of the two
+// kernels; else with nseg > 1 the second, with nseg 1 the only one
 __global__ void __launch_bounds__(THREADS) recurrence_kernel(const Rec p) {
     pdl_wait();
     const int c = blockIdx.x * THREADS + threadIdx.x;
@@ -65,9 +66,12 @@ __global__ void __launch_bounds__(THREADS) recurrence_kernel(const Rec p) {
     const int slot = p.slots[b];
     const int r0 = sg * p.seg, r1 = min(r0 + p.seg, n);
     if (r0 >= n) return;
+    const T* up = (const T*)p.u;
+    const T* yp = (const T*)p.y;
+    T* op = (T*)p.out;
     if (slot < 0) {
         if (!AGGREGATE)
-            for (int r = r0; r < r1; ++r) store_from_f(p.out, p.out_dt, (size_t)(row0 + r) * p.ldo + c, 0.f);
+            for (int r = r0; r < r1; ++r) op[(size_t)(row0 + r) * p.ldo + c] = from_f<T>(0.f);
         return;
     }
     const int blk = c / p.part;
@@ -84,7 +88,7 @@ __global__ void __launch_bounds__(THREADS) recurrence_kernel(const Rec p) {
 #pragma unroll 4
         for (int r = r0; r < r1; ++r) {
             float* z = p.z + (size_t)(row0 + r) * p.ldz + zc;
-            const float2 ab = gates(z[0], z[p.part], br, bi, decay, load_as_f(p.u, p.u_dt, (size_t)(row0 + r) * p.ldu + c));
+            const float2 ab = gates(z[0], z[p.part], br, bi, decay, to_f(up[(size_t)(row0 + r) * p.ldu + c]));
             z[0] = ab.x;
             z[p.part] = ab.y;
             all *= ab.x;
@@ -111,24 +115,24 @@ __global__ void __launch_bounds__(THREADS) recurrence_kernel(const Rec p) {
     const float yb = p.yb != nullptr ? load_as_f(p.yb, p.yb_dt, c) : 0.f;
     constexpr int AHEAD = 8;                                   // rows asked for together
     for (int r = r0; r < r1; r += AHEAD) {
-        float za[AHEAD], zb[AHEAD], yv[AHEAD], uv[AHEAD];
+        float za[AHEAD], zb[AHEAD];
+        T yv[AHEAD], uv[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-            if (r + i >= r1) continue;
-            const size_t row = (size_t)(row0 + r + i);
+            const size_t row = (size_t)(row0 + min(r + i, r1 - 1));
             za[i] = p.z[row * p.ldz + zc];
             zb[i] = p.z[row * p.ldz + zc + p.part];
-            if (p.y != nullptr) yv[i] = load_as_f(p.y, p.y_dt, row * p.ldy + c);
-            if (whole) uv[i] = load_as_f(p.u, p.u_dt, row * p.ldu + c);
+            if (yp != nullptr) yv[i] = yp[row * p.ldy + c];
+            if (whole) uv[i] = up[row * p.ldu + c];
         }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
             if (r + i >= r1) continue;
             float2 ab = make_float2(za[i], zb[i]);
-            if (whole) ab = gates(ab.x, ab.y, br, bi, decay, uv[i]);
+            if (whole) ab = gates(ab.x, ab.y, br, bi, decay, to_f(uv[i]));
             S = fmaf(ab.x, S, ab.y);
-            const float gate = p.y != nullptr ? gelu_tanh(yv[i] + yb) : 1.f;
-            store_from_f(p.out, p.out_dt, (size_t)(row0 + r + i) * p.ldo + c, p.scale * S * gate);
+            const float gate = yp == nullptr ? 1.f : (sizeof(T) == 2 ? activate_fast(to_f(yv[i]) + yb, QNN_ACT_GELU_TANH) : gelu_tanh(to_f(yv[i]) + yb));
+            op[(size_t)(row0 + r + i) * p.ldo + c] = from_f<T>(p.scale * S * gate);
         }
     }
     if (r1 == n) *state = S;
@@ -143,14 +147,14 @@ __global__ void __launch_bounds__(THREADS) recurrence_prefix_kernel(const Rec p)
     const int segs = (n + p.seg - 1) / p.seg;
     float* sc = p.scratch + (size_t)b * p.nseg * 3 * p.C + c;
     float S = sc[2 * (size_t)p.C];
-    constexpr int AHEAD = 8;
+    constexpr int AHEAD = 16;
     for (int k = 0; k < segs; k += AHEAD) {
         float all[AHEAD], reached[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-            if (k + i >= segs) continue;
-            all[i] = sc[(size_t)(k + i) * 3 * p.C];
-            reached[i] = sc[((size_t)(k + i) * 3 + 1) * p.C];
+            const int kk = min(k + i, segs - 1);
+            all[i] = sc[(size_t)kk * 3 * p.C];
+            reached[i] = sc[((size_t)kk * 3 + 1) * p.C];
         }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
@@ -173,18 +177,19 @@ QNN_API int qnn_linear_recurrence(float* z, long long ldz, const void* rb, const
                                   int C, int part, int seg, int nseg, float* scratch, int gates_done,
                                   cudaStream_t st) {
     if (n_seqs <= 0) return 0;
+    if (u_dt != out_dt || (y != nullptr && y_dt != u_dt)) return QNN_ERR_ARGUMENT;
     if (C <= 0 || part <= 0 || C % part || nseg < 1 || seg < 1 || n_seqs > 65535 || nseg > 65535 || ldz < 2LL * C ||
         ldu < C || ldo < C || (y != nullptr && ldy < C) || slot_stride < C || (nseg > 1 && (scratch == nullptr || seq_row0 == nullptr)))
         return QNN_ERR_ARGUMENT;
     Rec p;
     p.z = z; p.rb = rb; p.ib = ib; p.decay = decay; p.u = u; p.y = y; p.yb = yb; p.out = out; p.state = state;
     p.scratch = scratch; p.seq_row0 = seq_row0; p.seq_len = seq_len; p.slots = slots; p.ldz = ldz; p.ldu = ldu; p.ldy = ldy;
-    p.ldo = ldo; p.slot_stride = slot_stride; p.b_dt = b_dt; p.u_dt = u_dt; p.y_dt = y_dt; p.yb_dt = yb_dt; p.out_dt = out_dt;
+    p.ldo = ldo; p.slot_stride = slot_stride; p.b_dt = b_dt; p.yb_dt = yb_dt;
     p.C = C; p.part = part; p.seg = seg; p.nseg = nseg; p.scale = scale;
     p.prefixed = nseg > INLINE_PREFIX ? 1 : 0;
     const dim3 grid((C + THREADS - 1) / THREADS, nseg, n_seqs);
     if (nseg > 1 && !gates_done) {
-        launch_pdl(recurrence_kernel<true>, grid, dim3(THREADS), 0, st, p);
+        launch_pdl(u_dt == QNN_DT_BF16 ? recurrence_kernel<true, bf16> : recurrence_kernel<true, float>, grid, dim3(THREADS), 0, st, p);
         const cudaError_t e = cudaGetLastError();
         if (e != cudaSuccess) return (int)e;
     }
@@ -193,6 +198,6 @@ QNN_API int qnn_linear_recurrence(float* z, long long ldz, const void* rb, const
         const cudaError_t e = cudaGetLastError();
         if (e != cudaSuccess) return (int)e;
     }
-    launch_pdl(recurrence_kernel<false>, grid, dim3(THREADS), 0, st, p);
+    launch_pdl(u_dt == QNN_DT_BF16 ? recurrence_kernel<false, bf16> : recurrence_kernel<false, float>, grid, dim3(THREADS), 0, st, p);
     QNN_LAUNCH_CHECK();
 }

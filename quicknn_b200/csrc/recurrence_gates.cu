@@ -1,9 +1,9 @@
 // The gates of a real-gated linear recurrence for many rows, and the first pass over its segments, in one kernel (what this
 // leaves is described at the head of linear_recurrence.cu; the formulas are those of its `gates`).
 //
-// A CTA owns 128 rows (four segments of 32) of one sequence and 64 channels of one part.  The product is that of
-// block_linear.cu: u of the part against the r rows and the i rows of the channels, 128 x 128 outputs, mma.sync m16n8k16, a
-// cp.async ring of three stages of 64 inner elements, float32 sums.  The logits stay in shared memory; then a thread per
+// A CTA owns 64 rows (two segments of 32) of one sequence and 64 channels of one part.  The product is that of
+// block_linear.cu: u of the part against the r rows and the i rows of the channels, 64 x 128 outputs, mma.sync m16n8k16, a
+// cp.async ring of two stages of 64 inner elements, float32 sums.  The logits stay in shared memory; then a thread per
 // channel and segment forms (a, term) of its rows in order, writes them out and leaves the segment's product of a and the
 // state that it reaches.
 #include "common.cuh"
@@ -29,11 +29,25 @@ __device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4],
         : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-constexpr int BM = 128, CH = 64, BN = 2 * CH, BK = 64, STAGES = 3, THREADS = 256, ROWB = BK * 2;
+constexpr int BM = 64, CH = 64, BN = 2 * CH, BK = 64, STAGES = 2, THREADS = 128, ROWB = BK * 2;   // four CTAs per SM
 constexpr int SEG = 32, STAGE = (BM + BN) * ROWB, LDL = BN + 1;
 constexpr size_t SMEM = (size_t)STAGES * STAGE;
 static_assert((size_t)BM * LDL * 4 <= SMEM, "the logits take the ring's place");
 static_assert(THREADS == CH * (BM / SEG), "a thread per channel and segment");
+
+// 32-bit arithmetic on the fast exponential, quotient and square root (relative errors of about 1e-6; u and the product's
+// operands are bfloat16).
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+// 1 - e^t for t <= 0, with the digits kept where t is near 0 (there the Taylor sum, remainder below 3e-7 of it)
+__device__ __forceinline__ float one_minus_exp(float t) {
+    const float series = -t * fmaf(t * 0.5f, fmaf(t * (1.f / 3.f), fmaf(t * 0.25f, fmaf(t * 0.2f, fmaf(t, 1.f / 6.f, 1.f), 1.f), 1.f), 1.f), 1.f);
+    return t > -0.35f ? series : 1.f - __expf(t);
+}
+__device__ __forceinline__ float sqrt_fast(float x) {
+    float r;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
 
 struct Gates {
     const bf16* u;              // rows of pitch ldu
@@ -51,13 +65,13 @@ struct Gates {
     int C, part, nseg, tiles;   // tiles: channel tiles of a part
 };
 
-__global__ void __launch_bounds__(THREADS) recurrence_gates_kernel(const Gates p) {
+__global__ void __launch_bounds__(THREADS, 4) recurrence_gates_kernel(const Gates p) {
     extern __shared__ __align__(128) unsigned char smem[];
     float* logits = reinterpret_cast<float*>(smem);             // [BM][LDL], once the products are done
     const int blk = blockIdx.x / p.tiles, c0 = (blockIdx.x - blk * p.tiles) * CH;
     const int b = blockIdx.z, m0 = blockIdx.y * BM;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-    const int wm = warp >> 2, wn = warp & 3;
+    const int wm = warp >> 1, wn = warp & 1;                    // warp tiles of 32 x 64
     const int n = p.seq_len[b], slot = p.slots[b];              // from the host, before the step
     if (m0 >= n || slot < 0) return;
     const int row0 = p.seq_row0[b] + m0, rows = min(BM, n - m0);
@@ -94,11 +108,11 @@ __global__ void __launch_bounds__(THREADS) recurrence_gates_kernel(const Gates p
         if (s < nk) load_u(s);
         cp_async_commit();                                      // (the first group also holds the weights asked for above)
     }
-    float acc[4][4][4];
+    float acc[2][8][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
     for (int kb = 0; kb < nk; ++kb) {
@@ -112,21 +126,21 @@ __global__ void __launch_bounds__(THREADS) recurrence_gates_kernel(const Gates p
         const unsigned sa = base + (kb % STAGES) * STAGE, sb = sa + BM * ROWB;
 #pragma unroll
         for (int ks = 0; ks < BK / 16; ++ks) {
-            uint32_t af[4][4], bf[2][4];
+            uint32_t af[2][4], bf[4][4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int r = wm * 64 + i * 16 + (lane & 15), c = ks * 2 + (lane >> 4);
+            for (int i = 0; i < 2; ++i) {
+                const int r = wm * 32 + i * 16 + (lane & 15), c = ks * 2 + (lane >> 4);
                 ldmatrix_x4(af[i], sa + r * ROWB + ((c ^ (r & 7)) << 4));
             }
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int r = wn * 32 + j * 16 + (lane & 7) + ((lane >> 4) << 3), c = ks * 2 + ((lane >> 3) & 1);
+            for (int j = 0; j < 4; ++j) {
+                const int r = wn * 64 + j * 16 + (lane & 7) + ((lane >> 4) << 3), c = ks * 2 + ((lane >> 3) & 1);
                 ldmatrix_x4(bf[j], sb + r * ROWB + ((c ^ (r & 7)) << 4));
             }
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+            for (int i = 0; i < 2; ++i)
 #pragma unroll
-                for (int j = 0; j < 2; ++j) {
+                for (int j = 0; j < 4; ++j) {
                     mma_16816(acc[i][2 * j], af[i], bf[j][0], bf[j][1]);
                     mma_16816(acc[i][2 * j + 1], af[i], bf[j][2], bf[j][3]);
                 }
@@ -135,12 +149,12 @@ __global__ void __launch_bounds__(THREADS) recurrence_gates_kernel(const Gates p
     cp_async_wait<0>();
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
+        for (int j = 0; j < 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-                logits[(wm * 64 + i * 16 + g + (e >> 1) * 8) * LDL + wn * 32 + j * 8 + t4 * 2 + (e & 1)] = acc[i][j][e];
+                logits[(wm * 32 + i * 16 + g + (e >> 1) * 8) * LDL + wn * 64 + j * 8 + t4 * 2 + (e & 1)] = acc[i][j][e];
     __syncthreads();
     const int cl = tid & (CH - 1), seg = tid / CH, k = c0 + cl;
     const int r0 = seg * SEG, r1 = min(r0 + SEG, rows);
@@ -153,24 +167,32 @@ __global__ void __launch_bounds__(THREADS) recurrence_gates_kernel(const Gates p
         S = p.state[(size_t)slot * p.slot_stride + ch];
         sc[2 * (size_t)p.C] = S;
     }
-    const bf16* uc = ub + k;
-    float* zc = p.z + (size_t)row0 * p.ldz + (size_t)blk * 2 * p.part + k;
-    constexpr int AHEAD = 8;
-    for (int r = r0; r < r1; r += AHEAD) {
-        float u[AHEAD];
+    const bf16* uc = ub + (size_t)r0 * p.ldu + k;
+    float* zc = p.z + (size_t)(row0 + r0) * p.ldz + (size_t)blk * 2 * p.part + k;
+    const float* lg = logits + r0 * LDL + cl;
+    auto row = [&](float u, int i) {                            // row r0 + i of the segment
+        const float la = -decay * sigmoid_fast(lg[i * LDL] + br);
+        const float a = __expf(la), term = sqrt_fast(one_minus_exp(2.f * la)) * sigmoid_fast(lg[i * LDL + CH] + bi) * u;
+        zc[0] = a;
+        zc[p.part] = term;
+        zc += p.ldz;
+        all *= a;
+        S = fmaf(a, S, term);
+    };
+    if (r1 - r0 == SEG) {
+        constexpr int AHEAD = 16;                               // rows of u asked for together
+#pragma unroll 1
+        for (int r = 0; r < SEG; r += AHEAD) {
+            bf16 u[AHEAD];
 #pragma unroll
-        for (int i = 0; i < AHEAD; ++i) u[i] = r + i < r1 ? __bfloat162float(uc[(size_t)(r + i) * p.ldu]) : 0.f;
+            for (int i = 0; i < AHEAD; ++i) u[i] = uc[(size_t)i * p.ldu];
+            uc += (size_t)AHEAD * p.ldu;
 #pragma unroll
-        for (int i = 0; i < AHEAD; ++i) {
-            if (r + i >= r1) continue;
-            const float la = -decay * (1.f / (1.f + expf(-(logits[(r + i) * LDL + cl] + br))));
-            const float gi = 1.f / (1.f + expf(-(logits[(r + i) * LDL + CH + cl] + bi)));
-            const float a = expf(la), term = sqrtf(-expm1f(2.f * la)) * gi * u[i];
-            zc[(size_t)(r + i) * p.ldz] = a;
-            zc[(size_t)(r + i) * p.ldz + p.part] = term;
-            all *= a;
-            S = fmaf(a, S, term);
+            for (int i = 0; i < AHEAD; ++i) row(__bfloat162float(u[i]), i);
+            lg += AHEAD * LDL;
         }
+    } else {
+        for (int r = 0; r < r1 - r0; ++r) row(__bfloat162float(uc[(size_t)r * p.ldu]), r);
     }
     sc[0] = all;
     sc[p.C] = S;

@@ -24,19 +24,45 @@ __device__ __forceinline__ void load_v(const void* p, int dt, size_t i, float* o
     if (VEC == 8) load8_as_f(p, dt, i, o);
     else o[0] = load_as_f(p, dt, i);
 }
-template <int VEC>
-__device__ __forceinline__ void store_v(void* p, int dt, size_t i, const float* v) {
-    if (VEC == 8) store8_from_f(p, dt, i, v);
-    else store_from_f(p, dt, i, v[0]);
+// VEC consecutive elements as they lie in memory: loads that do not wait for one another
+template <typename T, int VEC> struct Raw {
+    static constexpr int PIECES = VEC == 8 ? 8 / Vec16<T>::N : 1;
+    Vec16<T> v[PIECES];
+    T one;
+    __device__ __forceinline__ void load(const T* p) {
+        if (VEC == 8) {
+#pragma unroll
+            for (int i = 0; i < PIECES; ++i) v[i].load(p + i * Vec16<T>::N);
+        } else {
+            one = *p;
+        }
+    }
+    __device__ __forceinline__ void unpack(float* o) const {
+        if (VEC == 8) {
+#pragma unroll
+            for (int i = 0; i < PIECES; ++i) v[i].unpack(o + i * Vec16<T>::N);
+        } else {
+            o[0] = to_f(one);
+        }
+    }
+};
+template <typename T, int VEC>
+__device__ __forceinline__ void store_v(T* p, const float* v) {
+    if (VEC == 8) {
+#pragma unroll
+        for (int i = 0; i < 8 / Vec16<T>::N; ++i) Vec16<T>::store(p + i * Vec16<T>::N, v + i * Vec16<T>::N);
+    } else {
+        p[0] = from_f<T>(v[0]);
+    }
 }
 
 // TAPS > 0: the number of taps and of rows per tile (ROWS) is known here, and the filter and the tile's inputs stay in
 // registers; 0: any numbers, inputs are read again for every tap.
-template <int VEC, int TAPS, int ROWS>
+template <typename T, int VEC, int TAPS, int ROWS>
 __global__ void __launch_bounds__(THREADS)
-causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const void* __restrict__ x_bias, int xb_dt,
+causal_conv_kernel(const T* __restrict__ x, long long ldx, const void* __restrict__ x_bias, int xb_dt,
                    const void* __restrict__ w, int w_dt, const void* __restrict__ out_bias, int ob_dt, int add_input,
-                   void* __restrict__ out, int out_dt, long long ldo, float* state, long long slot_stride, int C, int taps_,
+                   T* __restrict__ out, long long ldo, float* state, long long slot_stride, int C, int taps_,
                    const int* __restrict__ seq_row0, const int* __restrict__ seq_len, const int* __restrict__ tok_pos,
                    const int* __restrict__ slots, int rows_) {
     const int taps = TAPS > 0 ? TAPS : taps_, rows = TAPS > 0 ? ROWS : rows_;
@@ -70,7 +96,7 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
         float z[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) z[e] = 0.f;
-        for (int r = r0; r < r1; ++r) store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, z);
+        for (int r = r0; r < r1; ++r) store_v<T, VEC>(out + (size_t)(row0 + r) * ldo + c0, z);
         return;
     }
     const int first = tok_pos[row0];                        // position of the sequence's first row of this step
@@ -78,7 +104,9 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
     // v of row r (may be negative: an earlier step's, or before the sequence)
     auto input = [&](int r, float* v) {
         if (r >= 0) {
-            load_v<VEC>(x, x_dt, (size_t)(row0 + r) * ldx + c0, v);
+            Raw<T, VEC> raw;
+            raw.load(x + (size_t)(row0 + r) * ldx + c0);
+            raw.unpack(v);
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v[e] += xb[e];
         } else if (first + r >= 0) {
@@ -92,10 +120,22 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
     };
     if constexpr (TAPS > 0) {
         float v[ROWS + TAPS - 1][VEC];
+        if (r0 >= TAPS - 1 && r0 + ROWS <= n) {             // a whole tile with its past among the step's rows: no branches
+            Raw<T, VEC> raw[ROWS + TAPS - 1];
 #pragma unroll
-        for (int i = 0; i < ROWS + TAPS - 1; ++i) {
-            const int r = r0 - TAPS + 1 + i;
-            if (r < r1) input(r, v[i]);
+            for (int i = 0; i < ROWS + TAPS - 1; ++i) raw[i].load(x + (size_t)(row0 + r0 - TAPS + 1 + i) * ldx + c0);
+#pragma unroll
+            for (int i = 0; i < ROWS + TAPS - 1; ++i) {
+                raw[i].unpack(v[i]);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[i][e] += xb[e];
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < ROWS + TAPS - 1; ++i) {
+                const int r = r0 - TAPS + 1 + i;
+                if (r < r1) input(r, v[i]);
+            }
         }
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
@@ -109,7 +149,7 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
                 acc[e] += ob[e];
                 if (add_input) acc[e] += v[i + TAPS - 1][e];
             }
-            store_v<VEC>(out, out_dt, (size_t)(row0 + r0 + i) * ldo + c0, acc);
+            store_v<T, VEC>(out + (size_t)(row0 + r0 + i) * ldo + c0, acc);
         }
     } else {
         for (int r = r0; r < r1; ++r) {
@@ -123,7 +163,7 @@ causal_conv_kernel(const void* __restrict__ x, int x_dt, long long ldx, const vo
             }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) acc[e] += ob[e] + (add_input ? v[e] : 0.f);
-            store_v<VEC>(out, out_dt, (size_t)(row0 + r) * ldo + c0, acc);
+            store_v<T, VEC>(out + (size_t)(row0 + r) * ldo + c0, acc);
         }
     }
     if (r0 == 0) {
@@ -148,7 +188,8 @@ QNN_API int qnn_causal_conv(const void* x, int x_dt, long long ldx, const void* 
                             const int* tok_pos, const int* slots, int n_seqs, int longest, cudaStream_t st) {
     if (n_seqs <= 0 || longest <= 0) return 0;
     if (C <= 0 || taps < 1 || n_seqs > 65535 || ldx < C || ldo < C || slot_stride < (long long)taps * C) return QNN_ERR_ARGUMENT;
-    const int xs = x_dt == QNN_DT_BF16 ? 2 : 4, os = out_dt == QNN_DT_BF16 ? 2 : 4;
+    if (x_dt != out_dt) return QNN_ERR_ARGUMENT;
+    const int xs = x_dt == QNN_DT_BF16 ? 2 : 4, os = xs;
     const bool vec = C % 8 == 0 && (ldx * xs) % 16 == 0 && (ldo * os) % 16 == 0 &&
                      (((uintptr_t)x | (uintptr_t)out | (uintptr_t)x_bias | (uintptr_t)out_bias | (uintptr_t)w) & 15) == 0;
     const bool known = vec && taps >= 2 && taps <= 4;
@@ -157,9 +198,14 @@ QNN_API int qnn_causal_conv(const void* x, int x_dt, long long ldx, const void* 
     const long long work = (long long)((longest + rows - 1) / rows) * ((C + (vec ? 7 : 0)) / (vec ? 8 : 1));
     if (work + THREADS > 0xffffffffLL) return QNN_ERR_UNSUPPORTED;
     const dim3 grid((unsigned)((work + THREADS - 1) / THREADS), n_seqs);
-#define QNN_CONV(V, TP, R)                                                                                             \
-    launch_pdl(causal_conv_kernel<V, TP, R>, grid, dim3(THREADS), 0, st, x, x_dt, ldx, x_bias, xb_dt, w, w_dt, out_bias, \
-               ob_dt, add_input, out, out_dt, ldo, state, slot_stride, C, taps, seq_row0, seq_len, tok_pos, slots, rows)
+#define QNN_CONV_AS(T, V, TP, R)                                                                                       \
+    launch_pdl(causal_conv_kernel<T, V, TP, R>, grid, dim3(THREADS), 0, st, (const T*)x, ldx, x_bias, xb_dt, w, w_dt,   \
+               out_bias, ob_dt, add_input, (T*)out, ldo, state, slot_stride, C, taps, seq_row0, seq_len, tok_pos, slots, rows)
+#define QNN_CONV(V, TP, R)                                        \
+    do {                                                          \
+        if (x_dt == QNN_DT_BF16) QNN_CONV_AS(bf16, V, TP, R);     \
+        else QNN_CONV_AS(float, V, TP, R);                        \
+    } while (0)
 #define QNN_CONV_TAPS(R)               \
     if (taps == 4) QNN_CONV(8, 4, R);  \
     else if (taps == 3) QNN_CONV(8, 3, R); \
@@ -170,5 +216,6 @@ QNN_API int qnn_causal_conv(const void* x, int x_dt, long long ldx, const void* 
     else QNN_CONV(1, 0, 1);
 #undef QNN_CONV_TAPS
 #undef QNN_CONV
+#undef QNN_CONV_AS
     QNN_LAUNCH_CHECK();
 }

@@ -35,6 +35,25 @@ struct Update {
     float mult, eps_post, off_post, eps_next, off_next;
 };
 
+// Eight consecutive values of either element type as they lie in memory: a load that nothing waits for until it is unpacked.
+struct Raw8 {
+    uint4 a, b;
+    __device__ __forceinline__ void load(const void* p, int dt, size_t i) {
+        if (dt == QNN_DT_BF16) {
+            a = *reinterpret_cast<const uint4*>((const bf16*)p + i);
+        } else {
+            a = *reinterpret_cast<const uint4*>((const float*)p + i);
+            b = *reinterpret_cast<const uint4*>((const float*)p + i + 4);
+        }
+    }
+    __device__ __forceinline__ void unpack(int dt, float* o) const {
+        const uint32_t w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+            o[e] = dt == QNN_DT_BF16 ? __uint_as_float((e & 1) ? (w[e >> 1] & 0xffff0000u) : (w[e >> 1] << 16)) : __uint_as_float(w[e]);
+    }
+};
+
 // TAPS > 0: h = n + conv(n), that many taps, of the normed row n (rounded as it is stored), a row per sequence; the row's n joins the ring.
 // What waits for no sum (weights before the wait for the kernel in front; the ring's earlier rows; the earlier layers' rows,
 // summed in the order of the layers) is asked for before the first sum.
@@ -46,18 +65,16 @@ __global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kerne
     __shared__ float red[32];
     const size_t base = (size_t)blockIdx.x * u.H;
     const int nchunks = u.H >> 3;
-    float g1[CH][8], g2[CH][8], v[CH][8], r[CH][8], z[CH][8];
-    float wv[CONV ? TAPS * 8 : 1], prev[TAPS > 1 ? TAPS - 1 : 1][8];
+    float v[CH][8], r[CH][8], z[CH][8];
+    Raw8 g1[CH], g2[CH], wr[CONV ? TAPS : 1];
+    float prev[TAPS > 1 ? TAPS - 1 : 1][8];
     const bool in0 = (int)threadIdx.x < nchunks;
 #pragma unroll
     for (int i = 0; i < CH; ++i) {                       // weights are written by no kernel of the step
         const int c = threadIdx.x + i * blockDim.x;
         if (c < nchunks) {
-            load8_as_f(u.w_post, u.wp_dt, (size_t)c * 8, g1[i]);
-            if (u.out_next != nullptr) load8_as_f(u.w_next, u.wn_dt, (size_t)c * 8, g2[i]);
-        } else {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) g1[i][e] = g2[i][e] = 0.f;
+            g1[i].load(u.w_post, u.wp_dt, (size_t)c * 8);
+            if (u.out_next != nullptr) g2[i].load(u.w_next, u.wn_dt, (size_t)c * 8);
         }
     }
     int slot = -1, pos = 0;
@@ -68,7 +85,7 @@ __global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kerne
         ring = u.ring + (size_t)(slot < 0 ? 0 : slot) * u.slot_stride + threadIdx.x * 8;
         if (in0)
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) load8_as_f(u.conv, u.conv_dt, (size_t)threadIdx.x * 8 * TAPS + j * 8, wv + j * 8);
+            for (int j = 0; j < TAPS; ++j) wr[j].load(u.conv, u.conv_dt, (size_t)threadIdx.x * 8 * TAPS + j * 8);
     }
     const float a_last = u.hist != nullptr ? load_as_f(u.numbers, u.num_dt, u.n_hist) : 1.f;
     pdl_wait();
@@ -80,11 +97,15 @@ __global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kerne
         for (int e = 0; e < 8; ++e) v[i][e] = r[i][e] = z[i][e] = 0.f;
         if (c < nchunks) {
             const size_t yat = (size_t)blockIdx.x * u.terms * u.H + (size_t)c * 8, at = base + (size_t)c * 8;
-            load8_as_f(u.y, u.y_dt, yat, v[i]);
+            Raw8 y0, y1;
+            y0.load(u.y, u.y_dt, yat);
+            if (u.terms > 1) y1.load(u.y, u.y_dt, yat + u.H);
             load8_as_f(u.resid, QNN_DT_F32, at, r[i]);
+            y0.unpack(u.y_dt, v[i]);
             for (int k = 1; k < u.terms; ++k) {
                 float t[8];
-                load8_as_f(u.y, u.y_dt, yat + (size_t)k * u.H, t);
+                y1.unpack(u.y_dt, t);
+                if (k + 1 < u.terms) y1.load(u.y, u.y_dt, yat + (size_t)(k + 1) * u.H);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[i][e] += t[e];
             }
@@ -119,8 +140,10 @@ __global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kerne
         const int c = threadIdx.x + i * blockDim.x;
         if (c >= nchunks) continue;
         const size_t at = base + (size_t)c * 8;
+        float w1[8];
+        g1[i].unpack(u.wp_dt, w1);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) r[i][e] += u.mult * (v[i][e] * inv * (g1[i][e] + u.off_post));
+        for (int e = 0; e < 8; ++e) r[i][e] += u.mult * (v[i][e] * inv * (w1[e] + u.off_post));
         store8_from_f(u.resid_out, QNN_DT_F32, at, r[i]);
         if (u.hist != nullptr) {
 #pragma unroll
@@ -137,16 +160,19 @@ __global__ void __launch_bounds__(TAPS > 0 ? 512 : 1024) stream_update_vec_kerne
     for (int i = 0; i < CH; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
         if (c >= nchunks) continue;
-        float o[8];
+        float o[8], w2[8];
+        g2[i].unpack(u.wn_dt, w2);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (g2[i][e] + u.off_next);
+        for (int e = 0; e < 8; ++e) o[e] = r[i][e] * inv2 * (w2[e] + u.off_next);
         if constexpr (CONV) {
             if (slot >= 0) {
                 if (u.out_dt == QNN_DT_BF16)
 #pragma unroll
                     for (int e = 0; e < 8; ++e) o[e] = __bfloat162float(__float2bfloat16_rn(o[e]));
                 store8_from_f(ring + (size_t)(pos % TAPS) * u.H, QNN_DT_F32, 0, o);
-                float acc[8];
+                float acc[8], wv[TAPS * 8];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) wr[j].unpack(u.conv_dt, wv + j * 8);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) acc[e] = 0.f;
 #pragma unroll

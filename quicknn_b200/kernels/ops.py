@@ -1911,7 +1911,7 @@ def linear_recurrence(u: torch.Tensor, w_gates: torch.Tensor, r_bias: torch.Tens
         _p(y_bias), dt_code(y_bias) if y_bias is not None else 0, float(scale), _col_ptr(out, out_col0), dt_code(out),
         out.shape[1], state_ptr, state.stride(0), _p(seq_row0), _p(seq_len), _p(slots), n_seqs, C, part, seg if nseg > 1 else longest,
         nseg, _p(scratch), int(done), _stream()), "linear_recurrence",
-        1 + (1 if nseg > 1 and not done else 0) + (1 if nseg > 64 else 0))
+        1 + (1 if nseg > 1 and not done else 0) + (1 if nseg > 8 else 0))
     return out
 
 

@@ -562,7 +562,7 @@ def test_the_recurrent_block_alone_and_a_lost_state_would_show(dtype, width, blo
 @pytest.mark.parametrize("dtype", BOTH)
 @pytest.mark.parametrize("width,blocks", [(96, 2), (40, 5)])
 def test_long_prompts_walk_the_recurrence_in_segments(dtype, width, blocks):
-    """2500 rows (more segments than are chained inside the last kernel), 33, 32 and 5 rows beside one another; then 600 and 40
+    """2500 rows (segments chained by a kernel of their own), 33, 32 and 5 rows beside one another; then 600 and 40
     rows onto states that are not empty; the plain walk, and for bfloat16 rows also the gates formed by kernels of their own."""
     from quicknn_b200.cache import KVCache
     from quicknn_b200.kernels import ops
