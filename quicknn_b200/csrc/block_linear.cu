@@ -124,13 +124,36 @@ block_linear_mma_kernel(const Args a) {
         for (int h = 0; h < 2; ++h) {
             const int t = m0 + wm * TM + i * 16 + g + h * 8;
             if (t >= a.T) continue;
+            float z[NT][2];
+            if (a.gate != nullptr) {                  // the row's gates are asked for together
+                const size_t at = (size_t)t * a.ldg + (size_t)b * a.N;
+                if (a.gate_dt == QNN_DT_BF16) {
+                    bf16 raw[NT][2];
+#pragma unroll
+                    for (int j = 0; j < NT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) raw[j][e] = ((const bf16*)a.gate)[at + min(n0 + wn * TN + j * 8 + t4 * 2 + e, a.N - 1)];
+#pragma unroll
+                    for (int j = 0; j < NT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) z[j][e] = __bfloat162float(raw[j][e]);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < NT; ++j)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) z[j][e] = ((const float*)a.gate)[at + min(n0 + wn * TN + j * 8 + t4 * 2 + e, a.N - 1)];
+                }
+            }
 #pragma unroll
             for (int j = 0; j < NT; ++j) {
                 const int n = n0 + wn * TN + j * 8 + t4 * 2;
                 if (n >= a.N) continue;
                 const size_t col = (size_t)b * a.N + n;
-                const float v0 = gated(a, t, col, acc[i][j][2 * h]);
-                const float v1 = n + 1 < a.N ? gated(a, t, col + 1, acc[i][j][2 * h + 1]) : 0.f;
+                float v0 = acc[i][j][2 * h], v1 = acc[i][j][2 * h + 1];
+                if (a.gate != nullptr) {
+                    v0 *= __fdividef(1.f, 1.f + __expf(-z[j][0]));
+                    v1 *= __fdividef(1.f, 1.f + __expf(-z[j][1]));
+                }
                 const size_t at = (size_t)t * a.ldo + col;
                 if (pair) {
                     if (a.out_dt == QNN_DT_BF16) *reinterpret_cast<__nv_bfloat162*>((bf16*)a.out + at) = __floats2bfloat162_rn(v0, v1);
@@ -208,7 +231,7 @@ QNN_API int qnn_block_linear(const void* x, int x_dt, long long ldx, long long x
     if (tensor) {
         if (T <= 32) return launch_mma<16, 64, 1, 4, 3>(a, blocks, st);
         const long long big = (long long)((T + 127) / 128) * ((N + 127) / 128) * blocks;
-        if (N > 64 && big >= 96) return launch_mma<128, 128, 2, 4, 3>(a, blocks, st);
+        if (N > 64 && big >= 448) return launch_mma<128, 128, 2, 4, 3>(a, blocks, st);
         return launch_mma<64, 64, 2, 2, 3>(a, blocks, st);
     }
     launch_pdl(block_linear_kernel, dim3((N + 31) / 32, (T + 31) / 32, blocks), dim3(256), 0, st, a);

@@ -140,7 +140,7 @@ int launch(const void* a, long long lda, int c_col, int r_col, const void* w, in
     const size_t smem = (((size_t)hd * sizeof(T) + 15) & ~(size_t)15) + (size_t)(rot / 2) * sizeof(float2);
     if (smem > 48 * 1024) return QNN_ERR_UNSUPPORTED;
     const int work = H * hd / V;
-    const int threads = work >= 256 ? 256 : 128;
+    const int threads = work >= 256 && T_rows <= 1024 ? 256 : 128;      // many rows: more of them on an SM at once
 #define QNN_LP(VV)                                                                                                       \
     launch_pdl(latent_prep_kernel<T, VV>, dim3(T_rows), dim3(threads), smem, st, (const T*)a, lda, c_col, r_col, w, w_dt, \
                eps, rank, rot, inv_freq, (const T*)q, ldq, (T*)q_out, ldo, H, hd, k_col, tok_pos, tok_slot, (T*)pool,     \

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 import dataclasses
-from typing import Any, Dict, List, Mapping, Optional
+from typing import Any, Dict, List, Mapping, Optional, Tuple
 
 import torch
 
@@ -32,7 +32,8 @@ class DepthHistory:
 
     results: torch.Tensor           # [layers + 1, T, width] float32: the embedded rows, then every layer's result
     stream: torch.Tensor            # [T, width] float32: the average that goes on
-    index: int = 0                  # the executed layer that runs: its result is results[index + 1]
+    rows: Tuple[torch.Tensor, ...]  # the same one by one: rows[j] is results[j]
+    index: int = 0                  # the executed layer that runs: its result is rows[index + 1]
 
 
 @dataclasses.dataclass

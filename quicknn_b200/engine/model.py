@@ -174,7 +174,9 @@ class Model:
         output head first and may return its result without the logits ever being written."""
         spec = self.spec
         sched = spec.schedule
-        first = self.blocks[sched[0].layer].entry(step, cache.line(sched[0].cache, writes=sched[0].writes_cache)) if sched else None
+        line_of = lambda e: cache.line(e.cache, writes=e.writes_cache)  # noqa: E731
+        line = line_of(sched[0]) if sched else None
+        first = self.blocks[sched[0].layer].entry(step, line) if sched else None
         if self.positions is not None and self.embedding_norm is None:
             # a learned vector per position joins the looked-up row; the first layer's norm in the same kernel
             if hasattr(first, "of_embedding_rows"):
@@ -190,11 +192,12 @@ class Model:
             # the embedded rows are the first of the results that later layers average over
             T, W = step.tokens.numel(), spec.hidden_size
             results = torch.empty((len(sched) + 1, T, W), dtype=torch.float32, device=step.tokens.device)
-            step.depth = DepthHistory(results, torch.empty((T, W), dtype=torch.float32, device=results.device))
+            step.depth = DepthHistory(results, torch.empty((T, W), dtype=torch.float32, device=results.device),
+                                      results.unbind(0))
             if hasattr(first, "of_embedding"):
-                x, normed = first.of_embedding(step.tokens, self.embedding, spec.embedding.scale, step.act_dtype, out=results[0])
+                x, normed = first.of_embedding(step.tokens, self.embedding, spec.embedding.scale, step.act_dtype, out=step.depth.rows[0])
             else:
-                x, normed = ops.embed(step.tokens, self.embedding, spec.embedding.scale, out=results[0]), None
+                x, normed = ops.embed(step.tokens, self.embedding, spec.embedding.scale, out=step.depth.rows[0]), None
         elif hasattr(first, "of_embedding"):
             # the first layer's first norm in the embedding's kernel; the layer is handed its input normed
             x, normed = first.of_embedding(step.tokens, self.embedding, spec.embedding.scale, step.act_dtype)
@@ -204,7 +207,6 @@ class Model:
         # the embedded rows once more, for the schedule entries before which they join the stream again
         x0 = ops.embed(step.tokens, self.embedding, spec.embedding.scale) if any(e.add_embedding for e in sched) else None
         for i, e in enumerate(sched):
-            line = cache.line(e.cache, writes=e.writes_cache)
             if line is not None:
                 line.has_readers = e.cache in self._lines_read
             if step.depth is not None:
@@ -216,14 +218,17 @@ class Model:
                 else:
                     ops.add_(x, x0)
                     normed = None
-            # the first norm of the layer that runs next is applied by this one, in the kernel
+            # what the layer that runs next does first (its first norm) is applied by this one, in the kernel
             # that adds this layer's last sublayer to the residual stream (not where the embedded rows come between)
-            nxt = None
-            if i + 1 < len(sched) and not sched[i + 1].add_embedding:
+            nxt, line_after = None, None
+            if i + 1 < len(sched):
                 after = sched[i + 1]
-                nxt = self.blocks[after.layer].entry(step, cache.line(after.cache, writes=after.writes_cache))
+                line_after = line_of(after)
+                if not after.add_embedding:
+                    nxt = self.blocks[after.layer].entry(step, line_after)
             out = self.blocks[e.layer].forward(x, step, line, normed=normed, next_norm=nxt)
             x, normed = out if nxt is not None else (out, None)
+            line = line_after
         for call in step.after_layers:         # appends that waited for the readers of their cache line
             call()
         step.after_layers.clear()

@@ -1800,6 +1800,10 @@ def sigmoid_attention(qkv: torch.Tensor, n_heads: int, n_kv: int, head_dim: int,
 
 # ---- short convolutions, block-diagonal products, the gated linear recurrence, rows of latent attention, averages over depth ----
 
+def _per_slot(state: torch.Tensor) -> int:
+    return state.numel() // state.shape[0]
+
+
 def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_row0: Optional[torch.Tensor],
                 seq_len: Optional[torch.Tensor], tok_pos: torch.Tensor, slots: torch.Tensor, n_seqs: int, longest: int = 1, *,
                 col0: int = 0, x_bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None,
@@ -1813,7 +1817,7 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_
     _req(state, "state", torch.float32)
     C, taps = weight.shape
     T = x.shape[0]
-    if col0 + C > x.shape[1] or state[0].numel() < taps * C or slots.numel() < n_seqs:
+    if col0 + C > x.shape[1] or _per_slot(state) < taps * C or slots.numel() < n_seqs:
         raise ValueError("causal_conv: shapes do not agree")
     for b in (x_bias, out_bias):
         if b is not None and b.numel() != C:
@@ -1877,7 +1881,7 @@ def linear_recurrence(u: torch.Tensor, w_gates: torch.Tensor, r_bias: torch.Tens
     B, _, part = w_gates.shape
     if B * part != C or w_gates.shape[1] != 2 * part or decay.numel() != C or r_bias.numel() != C or i_bias.numel() != C:
         raise ValueError("linear_recurrence: shapes do not agree")
-    if state[0].numel() < state_col0 + C or slots.numel() < n_seqs or (seq_row0 is None and T < n_seqs):
+    if _per_slot(state) < state_col0 + C or slots.numel() < n_seqs or (seq_row0 is None and T < n_seqs):
         raise ValueError("linear_recurrence: the state does not fit, or fewer rows than sequences")
     if y is not None and (y.shape[0] != T or y_col0 + C > y.shape[1]):
         raise ValueError("linear_recurrence: the output gate's rows do not fit")
@@ -1969,7 +1973,7 @@ def recurrent_step(p: torch.Tensor, y_col0: int, x_col0: int, x_bias: torch.Tens
             or any(v.dtype != conv.dtype for v in vecs):
         return False
     if (p.shape[0] != B or w_gates.shape[0] * part != C or w_gates.shape[1] != 2 * part or out.shape[0] != B
-            or out_col0 + C > out.shape[1] or max(y_col0, x_col0) + C > p.shape[1] or state[0].numel() < (taps + 1) * C):
+            or out_col0 + C > out.shape[1] or max(y_col0, x_col0) + C > p.shape[1] or _per_slot(state) < (taps + 1) * C):
         raise ValueError("recurrent_step: shapes do not agree")
     code = _lib.load().qnn_recurrent_step(
         _p(p), p.shape[1], int(y_col0), int(x_col0), _p(x_bias), _p(y_bias), _p(conv), _p(conv_bias), dt_code(conv), _p(w_gates),
@@ -1983,12 +1987,12 @@ def recurrent_step(p: torch.Tensor, y_col0: int, x_col0: int, x_bias: torch.Tens
 
 def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: torch.Tensor, eps_post: float, unit_post: bool,
                   out: Optional[torch.Tensor] = None, *, terms: int = 1, hist: Optional[torch.Tensor] = None,
-                  numbers: Optional[torch.Tensor] = None, avg_out: Optional[torch.Tensor] = None,
+                  n_hist: Optional[int] = None, numbers: Optional[torch.Tensor] = None, avg_out: Optional[torch.Tensor] = None,
                   w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0, unit_next: bool = False,
                   out_dtype: Optional[torch.dtype] = None, conv: Optional[tuple] = None) -> Optional[torch.Tensor]:
     """X = resid + mult * rmsnorm(y, w_post), written to ``out`` (default: resid, in place).  ``terms``: y has that many rows
-    per row, which are summed first.  With ``hist`` ([n, rows, width] float32, contiguous layers) and ``numbers`` (n + 1):
-    avg_out = sum_j numbers[j] hist[j] + numbers[n] X.  Returns n = rmsnorm(the average, or X; w_next) when ``w_next`` is given;
+    per row, which are summed first.  With ``hist`` ([.., rows, width] float32, contiguous layers, of which the first n = ``n_hist``
+    (default: all) count) and ``numbers`` (n + 1): avg_out = sum_j numbers[j] hist[j] + numbers[n] X.  Returns n = rmsnorm(the average, or X; w_next) when ``w_next`` is given;
     with ``conv`` = (weight [width, taps], ring state, tok_pos, slots), a row per sequence, n + conv(n) (``causal_conv`` with
     ``add_input``).  One kernel, float32 sums."""
     _req(resid, "resid", torch.float32, 2)
@@ -2004,15 +2008,15 @@ def stream_update(resid: torch.Tensor, y: torch.Tensor, mult: float, w_post: tor
     if hist is not None:
         _req(hist, "hist", torch.float32, 3)
         _req(avg_out, "avg_out", torch.float32, 2)
-        n = hist.shape[0]
-        if n < 1 or tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
+        n = hist.shape[0] if n_hist is None else int(n_hist)
+        if not (1 <= n <= hist.shape[0]) or tuple(hist.shape[1:]) != (T, H) or tuple(avg_out.shape) != (T, H) or numbers is None or numbers.numel() != n + 1:
             raise ValueError("stream_update: an average takes a number per earlier layer's rows and one for these")
     normed = torch.empty((T, H), dtype=out_dtype, device=resid.device) if w_next is not None else None
     cw = state = pos = slots = None
     if conv is not None:
         cw, state, pos, slots = conv
         _req(state, "state", torch.float32)
-        if w_next is None or cw.shape[0] != H or state[0].numel() < cw.numel() or slots.numel() != T:
+        if w_next is None or cw.shape[0] != H or _per_slot(state) < cw.numel() or slots.numel() != T:
             raise ValueError("stream_update: a convolution follows a norm, a filter per column, a row per sequence")
 
     def call(with_conv: bool) -> int:

@@ -171,7 +171,7 @@ class SandwichBlock(_LayerParts):
             if step.mode == "decode":
                 kw["conv"] = (conv.weight, conv.state, step.tok_pos, step.slots)
         if closes and self.depth is not None:
-            kw.update(hist=d.results[:d.index + 1], numbers=self.depth, avg_out=d.stream)
+            kw.update(hist=d.results, n_hist=d.index + 1, numbers=self.depth, avg_out=d.stream)
         if isinstance(then, RMSNorm):
             kw.update(w_next=then.weight, eps_next=then.eps, unit_next=then.unit_offset, out_dtype=step.act_dtype)
         n = ops.stream_update(resid, y, self.mult, p.weight, p.eps, p.unit_offset, out, **kw)
@@ -180,7 +180,7 @@ class SandwichBlock(_LayerParts):
     def _forward_general(self, resid: torch.Tensor, step, line, n, next_norm):
         y = self.mixer.forward(n, step, line)
         # with an average over depth the layer's result has a place of its own; the stream that came in is not touched
-        out = resid if self.depth is None else step.depth.results[step.depth.index + 1]
+        out = resid if self.depth is None else step.depth.rows[step.depth.index + 1]
         if self.ff is None:
             n = self._update(resid, y, "post_mixer", next_norm, step, out, True)
         else:

@@ -242,7 +242,7 @@ def test_causal_convolution_over_prompts_portions_and_single_tokens(dtype, C, ta
 
 @pytest.mark.parametrize("dtype", BOTH)
 @pytest.mark.parametrize("T,B,N,K", [(5, 3, 40, 24), (70, 2, 64, 64), (300, 4, 130, 72), (33, 1, 24, 200), (17, 5, 12, 12),
-                                     (40, 2, 7, 9), (16, 6, 96, 320), (1000, 8, 192, 96)])
+                                     (40, 2, 7, 9), (16, 6, 96, 320), (1000, 8, 192, 96), (3600, 8, 256, 64)])
 def test_block_diagonal_products(dtype, T, B, N, K):
     """Parts of rows times matrices of their own: float32 and rounded results, a gate per output, parts that lie further apart
     than they are wide."""
