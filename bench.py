@@ -261,6 +261,9 @@ def timed_tiny(torch):
 
 # ---- another design beside its closest model at equal size (--design) ------------------------------------
 
+HOST_LEAD_CYCLES = 40_000_000      # about 20 ms of device time: longer than the host needs to launch a step eagerly
+
+
 def design_sizes(name, design="fuposun"):
     """The configurations that ``--design`` times side by side, the design first: all have the same width, depth,
     vocabulary, window and dense feed-forward width.  ``2b``: the 2B layer sizes; ``1b``: about half of them.
@@ -385,7 +388,10 @@ def design_run(args, torch, pk):
                               "launches_per_step": dec["launches"] // max(1, min(args.steps, 128))}}
             # by kernel wrapper: one prompt, then eager decode steps at the context
             slot = eng.new_sequence()
+            # (the device is kept busy for a while first, so that it runs behind the host and the events bracket kernels,
+            # not the host's time between launches)
             with OpTimer(eng, pk["hbm_gbs"], pk["bf16_tflops"]) as t:
+                torch.cuda._sleep(HOST_LEAD_CYCLES)
                 eng.step([(slot, ids)], "last")
             rec["prefill_ops"] = t.rows()
             eng.release(slot)
@@ -395,6 +401,7 @@ def design_run(args, torch, pk):
             eng.decode(slots, toks, use_graph=False)
             with OpTimer(eng, pk["hbm_gbs"], pk["bf16_tflops"], context=args.context - 6) as t:
                 for _ in range(4):
+                    torch.cuda._sleep(HOST_LEAD_CYCLES)
                     eng.decode(slots, toks, use_graph=False)
             rows = t.rows()
             for r in rows:

@@ -283,9 +283,11 @@ class OpTimer:
             byts = float(q.shape[0] * row * q.element_size() + (_nbytes(q) + _nbytes(packed) if packed is not None else 2 * turned))
         elif name == "stream_update":
             resid, y = a[0], a[1]
-            byts = float(2 * _nbytes(resid) + _nbytes(y) + _nbytes(kw.get("hist")) + _nbytes(kw.get("avg_out")) + _nbytes(out))
+            hist, n = kw.get("hist"), kw.get("n_hist")
+            earlier = _nbytes(hist) if n is None or hist is None else n * _nbytes(resid)
+            byts = float(2 * _nbytes(resid) + _nbytes(y) + earlier + _nbytes(kw.get("avg_out")) + _nbytes(out))
         elif name == "gate_heads":
-            byts = float(2 * _nbytes(a[0]) + _nbytes(a[1]) + _nbytes(a[2]))
+            byts = float(2 * _nbytes(a[0]) + (_nbytes(a[1]) + _nbytes(a[2]) if a[2] is not None else a[0].shape[0] * a[3] * a[1].element_size()))
         elif name in ("rope_cache_write",):
             byts = float(2 * _nbytes(a[0]))
         elif name.startswith("embed"):               # the rows that are looked up, not the table
