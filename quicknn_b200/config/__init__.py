@@ -7,9 +7,11 @@ from .tumudra import TUMUDRA, TumudraConfig, tumudra_spec
 from .mubasun import MUBASUN, MubasunConfig, mubasun_spec
 from .gunirax import GUNIRAX, GuniraxConfig, gunirax_spec
 from .linedra import LINEDRA, LinedraConfig, linedra_spec
+from .vonulorn import VONULORN, VonulornConfig, vonulorn_spec
 
 __all__ = ["Architecture", "ConfigError", "ModelConfig", "find_architecture", "load_config",
            "register_architecture", "registered_architectures", "unregister_architecture",
            "GEMMA2", "Gemma2Config", "gemma2_spec", "FUPOSUN", "FuposunConfig", "fuposun_spec",
            "TUMUDRA", "TumudraConfig", "tumudra_spec", "MUBASUN", "MubasunConfig", "mubasun_spec",
-           "GUNIRAX", "GuniraxConfig", "gunirax_spec", "LINEDRA", "LinedraConfig", "linedra_spec"]
+           "GUNIRAX", "GuniraxConfig", "gunirax_spec", "LINEDRA", "LinedraConfig", "linedra_spec",
+           "VONULORN", "VonulornConfig", "vonulorn_spec"]

@@ -69,7 +69,7 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_scale_heads": [c_vp, c_int, c_vp, c_int, c_int, c_int, c_vp],
     "qnn_gate_heads": [c_vp, c_int, c_ll, c_vp, c_int, c_int, c_vp, c_int, c_vp, c_ll, c_float, c_int, c_int, c_int, c_vp],
     "qnn_causal_conv": [c_vp, c_int, c_ll, c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_int, c_ll, c_vp, c_ll, c_int,
-                        c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_vp],
+                        c_int, c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_int, c_int, c_float, c_vp],
     "qnn_stream_update": [c_vp, c_vp, c_int, c_int, c_float, c_vp, c_int, c_float, c_int, c_vp, c_vp, c_ll, c_int, c_vp, c_int,
                           c_vp, c_vp, c_int, c_float, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_ll, c_vp, c_vp, c_int,
                           c_int, c_vp],
@@ -133,6 +133,15 @@ _SIGNATURES: Dict[str, list] = {
     "qnn_sigattn_prefill_mma": [c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_int, c_int, c_float, c_vp, c_vp, c_vp, c_int, c_ll,
                                 c_vp, c_ll, c_int, c_int, c_int, c_vp, c_int, c_vp],
     "qnn_sigattn_prefill_ranges": [c_int, c_int, c_int, c_int, c_int, c_int, c_vp],
+    "qnn_delta_chunks": [c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_vp, c_int, c_vp, c_vp, c_float, c_vp, c_vp, c_vp, c_int, c_int,
+                         c_int, c_int, c_int, c_vp],
+    "qnn_delta_scan": [c_vp, c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_float, c_vp, c_vp, c_vp, c_vp, c_vp, c_ll, c_vp, c_ll, c_int,
+                       c_int, c_int, c_int, c_int, c_int, c_vp],
+    "qnn_delta_step": [c_vp, c_int, c_ll, c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_vp, c_vp, c_int, c_float, c_float,
+                       c_float, c_vp, c_ll, c_ll, c_vp, c_vp, c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_vp],
+    "qnn_map_prep": [c_vp, c_int, c_ll, c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_vp, c_vp,
+                     c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_int, c_int, c_vp],
+    "qnn_map_difference": [c_vp, c_ll, c_int, c_vp, c_ll, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_vp],
     "qnn_head_norm_gate": [c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_int, c_int, c_float, c_vp, c_ll, c_int, c_vp, c_ll,
                            c_int, c_int, c_int, c_int, c_vp],
 }

@@ -441,6 +441,14 @@ def _takes_skinny_tcgen05(M: int, N: int, K: int) -> bool:
 _SM_COUNT: dict = {}
 
 
+def _sm_count(device) -> int:
+    key = str(device)
+    if key not in _SM_COUNT:
+        dev = torch.device(device)
+        _SM_COUNT[key] = torch.cuda.get_device_properties(dev).multi_processor_count if dev.type == "cuda" else 148
+    return _SM_COUNT[key]
+
+
 def _rows_for_the_small_kernel(M: int, n_out: int, K: int, epilogue: int, device) -> int:
     """How many of the last rows of a whole-prompt product go to the kernel for few rows instead (0: none).
 
@@ -457,10 +465,7 @@ def _rows_for_the_small_kernel(M: int, n_out: int, K: int, epilogue: int, device
     tail = M % 256
     if tail == 0 or tail > 64:
         return 0
-    key = str(device)
-    if key not in _SM_COUNT:
-        _SM_COUNT[key] = torch.cuda.get_device_properties(device).multi_processor_count if device.type == "cuda" else 148
-    pairs = max(1, _SM_COUNT[key] // 2)
+    pairs = max(1, _sm_count(device) // 2)
     per_row_tile = -(-n_out // (128 if epilogue == EPI_GATED else 256))
     rounds = lambda m_tiles: -(-m_tiles * per_row_tile // pairs)          # noqa: E731
     if rounds(-(-M // 256)) == rounds(M // 256):
@@ -1433,11 +1438,7 @@ def _segment_rows(longest: int, blocks_per_segment: int, device) -> int:
     least 128 rows each, whole chunks of 16 rows); where not even two fit, the standing 256 rows.  Measured at 9 heads
     of 128 x 257, one prompt of 2048 rows: 8 segments of 256 are 360 blocks, a second round for 64 of them, 0.41 ms;
     6 segments of 352 are 270 blocks in one round."""
-    key = str(device)
-    if key not in _SM_COUNT:
-        dev = torch.device(device)
-        _SM_COUNT[key] = torch.cuda.get_device_properties(dev).multi_processor_count if dev.type == "cuda" else 148
-    fit = (2 * _SM_COUNT[key]) // max(1, blocks_per_segment)
+    fit = (2 * _sm_count(device)) // max(1, blocks_per_segment)
     if fit < 2:
         return GLA_SEGMENT
     nseg = max(1, min(fit, longest // 128))
@@ -1807,11 +1808,13 @@ def _per_slot(state: torch.Tensor) -> int:
 def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_row0: Optional[torch.Tensor],
                 seq_len: Optional[torch.Tensor], tok_pos: torch.Tensor, slots: torch.Tensor, n_seqs: int, longest: int = 1, *,
                 col0: int = 0, x_bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None,
-                add_input: bool = False) -> torch.Tensor:
+                add_input: bool = False, activation: Optional[str] = None, unit_heads: Optional[tuple] = None):
     """A causal convolution over time per channel: with v = x[:, col0 : col0 + C] + x_bias,
     out_t = sum_j weight[:, j] v_(t - taps + 1 + j) + out_bias (+ v_t with ``add_input``), zeros before a sequence's first
     position.  weight: [C, taps].  ``state``: float32 [slots, >= taps * C], whose first taps * C numbers per slot are a ring
-    of the last inputs (position p in row p mod taps).  ``seq_row0`` / ``seq_len`` None: a row per sequence (decode)."""
+    of the last inputs (position p in row p mod taps).  ``seq_row0`` / ``seq_len`` None: a row per sequence (decode).
+    ``activation`` "silu": applied to out_t.  ``unit_heads`` = (heads, size, eps): the first heads * size channels are heads, and
+    the result is the pair (out, float32 [rows, heads] with 1 / sqrt(sum of a head's squares + eps))"""
     _req(x, "x", None, 2)
     _req(weight, "weight", None, 2)
     _req(state, "state", torch.float32)
@@ -1824,12 +1827,135 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_
             raise ValueError("causal_conv: a bias per channel")
     if (seq_row0 is None) != (seq_len is None) or (seq_row0 is None and T < n_seqs):
         raise ValueError("causal_conv: first rows and row counts come together, or a row per sequence")
+    if activation not in (None, "silu"):
+        raise ValueError(f"causal_conv: {activation!r} is not an activation of this kernel")
     out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    heads, size, unit_eps = unit_heads if unit_heads is not None else (0, 0, 0.0)
+    inv = torch.empty((T, heads), dtype=torch.float32, device=x.device) if unit_heads is not None else None
     _lib.check(_lib.load().qnn_causal_conv(
         _col_ptr(x, col0), dt_code(x), x.shape[1], _p(x_bias), dt_code(x_bias) if x_bias is not None else 0, _p(weight),
         dt_code(weight), _p(out_bias), dt_code(out_bias) if out_bias is not None else 0, int(add_input), _p(out), dt_code(out),
         C, _p(state), state.stride(0), C, taps, _p(seq_row0), _p(seq_len), _p(tok_pos), _p(slots), n_seqs,
-        int(longest) if seq_row0 is not None else 1, _stream()), "causal_conv")
+        int(longest) if seq_row0 is not None else 1, int(activation is not None), _p(inv), int(size), int(heads), float(unit_eps),
+        _stream()), "causal_conv")
+    return out if inv is None else (out, inv)
+
+
+DELTA_CHUNK = 16             # rows of a chunk of the delta rule's scan
+DELTA_RECORD = 2 * DELTA_CHUNK * DELTA_CHUNK + 2 * DELTA_CHUNK
+
+
+def delta_scan(rows: torch.Tensor, inv: torch.Tensor, pre: torch.Tensor, rate: torch.Tensor, bias: torch.Tensor, q_scale: float,
+               state: torch.Tensor, state_col0: int, seq_row0: Optional[torch.Tensor], seq_len: Optional[torch.Tensor],
+               slots: torch.Tensor, n_seqs: int, longest: int, n_heads: int, n_kv: int, dim: int, vdim: int) -> torch.Tensor:
+    """The gated delta rule over the rows of every sequence in order, from the state of the sequence's slot and back into it:
+    S = g S, u = beta (v - S^T k), S = S + k u^T, o = S^T q, with beta and g one float32 number each per (row, value head).
+
+    ``rows``: q | k (``n_kv`` heads of ``dim``) | v (``n_heads`` of ``vdim``); ``inv``: float32 [rows, 2 n_kv], what q's and k's heads
+    are multiplied by (q also by ``q_scale``).  ``pre``: float32 [rows, 2 n_heads], z_b | z_a: beta = sigmoid(z_b),
+    g = exp(-rate softplus(z_a + bias)).  ``state``: float32 [slots, n], a slot's [n_heads, dim, vdim] from column ``state_col0``
+    on.  Returns o, float32 [rows, n_heads * vdim].  Rows are taken 16 at a time; how a sequence is cut into steps moves results
+    by rounding only."""
+    _req(rows, "rows", None, 2)
+    _req(inv, "inv", torch.float32, 2)
+    _req(pre, "pre", torch.float32, 2)
+    _req(rate, "rate", torch.float32, 1)
+    _req(bias, "bias", torch.float32, 1)
+    _req(state, "state", torch.float32)
+    T = rows.shape[0]
+    C = 2 * n_kv * dim + n_heads * vdim
+    if (rows.shape[1] < C or tuple(inv.shape) != (T, 2 * n_kv) or tuple(pre.shape) != (T, 2 * n_heads) or rate.numel() != n_heads
+            or bias.numel() != n_heads or slots.numel() < n_seqs or _per_slot(state) < state_col0 + n_heads * dim * vdim):
+        raise ValueError("delta_scan: shapes do not agree")
+    if (seq_row0 is None) != (seq_len is None) or (seq_row0 is None and T < n_seqs):
+        raise ValueError("delta_scan: first rows and row counts come together, or a row per sequence")
+    longest = int(longest) if seq_row0 is not None else 1
+    rec = torch.empty((T // DELTA_CHUNK + n_seqs) * n_heads * DELTA_RECORD, dtype=torch.float32, device=rows.device)
+    out = torch.empty((T, n_heads * vdim), dtype=torch.float32, device=rows.device)
+    L = _lib.load()
+    k0, v0 = n_kv * dim, 2 * n_kv * dim
+    _lib.check(L.qnn_delta_chunks(_p(rows), _col_ptr(rows, k0), rows.shape[1], dt_code(rows), _p(inv), inv.shape[1], _p(pre),
+                                  pre.shape[1], _p(rate), _p(bias), float(q_scale), _p(seq_row0), _p(seq_len), _p(rec), n_seqs,
+                                  longest, n_heads, n_kv, dim, _stream()), "delta_chunks")
+    # 16 value columns per block until they fill the device twice over
+    wide = n_seqs * n_heads * -(-vdim // 16) > 2 * _sm_count(rows.device)
+    _lib.check(L.qnn_delta_scan(_p(rows), _col_ptr(rows, k0), _col_ptr(rows, v0), rows.shape[1], dt_code(rows), _p(inv), inv.shape[1],
+                                float(q_scale), _p(rec), _p(seq_row0), _p(seq_len), _p(slots),
+                                ctypes.c_void_p(state.data_ptr() + 4 * state_col0), state.stride(0), _p(out), out.shape[1], n_seqs,
+                                n_heads, n_kv, dim, vdim, 2 if wide else 1, _stream()), "delta_scan")
+    return out
+
+
+def delta_step(p: torch.Tensor, x: torch.Tensor, w_ba: torch.Tensor, conv: torch.Tensor, rate: torch.Tensor, bias: torch.Tensor,
+               norm: torch.Tensor, eps: float, unit_eps: float, q_scale: float, state: torch.Tensor, state_col0: int,
+               tok_pos: torch.Tensor, slots: torch.Tensor, n_heads: int, n_kv: int, dim: int, vdim: int) -> Optional[torch.Tensor]:
+    """One token per sequence through everything between the input and the output product of the gated delta rule, in one
+    kernel: the convolutions with silu, the unit vectors, the gates' products (x w_ba^T, float32), ``delta_scan``, the RMS norm of
+    every head and the gate silu.  ``p``: rows q | k | v | gate; ``state``: float32 [slots, n], a slot's ring of last inputs
+    [taps, channels] and, from column ``state_col0`` on, [n_heads, dim, vdim].  The state is asked for before the kernel in front of this one has ended:
+    that kernel must not be one that writes it.  None where the kernel does not take the sizes: nothing has run then."""
+    _req(p, "p", None, 2)
+    _req(x, "x", p.dtype, 2)
+    _req(w_ba, "w_ba", None, 2)
+    _req(conv, "conv", None, 2)
+    _req(rate, "rate", torch.float32, 1)
+    _req(bias, "bias", torch.float32, 1)
+    _req(norm, "norm", None, 1)
+    _req(state, "state", torch.float32)
+    B = slots.numel()
+    C, taps = conv.shape
+    if (C != 2 * n_kv * dim + n_heads * vdim or p.shape != (B, C + n_heads * vdim) or x.shape[0] != B
+            or tuple(w_ba.shape) != (2 * n_heads, x.shape[1]) or norm.numel() != vdim or rate.numel() != n_heads
+            or bias.numel() != n_heads or state_col0 < taps * C or _per_slot(state) < state_col0 + n_heads * dim * vdim):
+        raise ValueError("delta_step: shapes do not agree")
+    out = torch.empty((B, n_heads * vdim), dtype=p.dtype, device=p.device)
+    code = _lib.load().qnn_delta_step(
+        _p(p), dt_code(p), p.shape[1], _p(x), x.shape[1], _p(w_ba), dt_code(w_ba), _p(conv), dt_code(conv), taps, _p(rate), _p(bias),
+        _p(norm), dt_code(norm), float(eps), float(unit_eps), float(q_scale), _p(state), state.stride(0), int(state_col0), _p(tok_pos), _p(slots),
+        _p(out), out.shape[1], B, n_heads, n_kv, dim, vdim, _stream())
+    if code == _lib.ERR_UNSUPPORTED:
+        return None
+    _lib.check(code, "delta_step")
+    return out
+
+
+def map_prep(src: torch.Tensor, n_heads: int, n_kv: int, maps: int, dim: int, vdim: int, head_dim: int, tok_pos: torch.Tensor,
+             tok_slot: torch.Tensor, line, append: bool, with_kv: bool, coef: float = 0.0, every: float = 1.0) -> torch.Tensor:
+    """The rows of a stacked q | k | v product packed for the attention kernels: query head h's map m becomes query head
+    h * maps + m of ``head_dim`` columns, its ``dim`` numbers at column m * dim, zeros elsewhere; a key head's maps lie side by
+    side, zeros behind; values get zeros behind.  Queries are multiplied by 1 + coef ln(floor((position + 1) / every) + 1).
+    Returns [rows, (n_heads * maps + 2 n_kv) * head_dim], without ``with_kv`` the queries alone; ``append``: keys and values go to
+    the cache line."""
+    _req(src, "src", None, 2)
+    T = src.shape[0]
+    if src.shape[1] != (n_heads + n_kv) * maps * dim + n_kv * vdim or head_dim < max(maps * dim, vdim):
+        raise ValueError("map_prep: shapes do not agree")
+    dst = torch.empty((T, (n_heads * maps + (2 * n_kv if with_kv else 0)) * head_dim), dtype=src.dtype, device=src.device)
+    k_pool = v_pool = table = slot_len = None
+    max_pages = page_size = ring = 0
+    if append:
+        if line.k.dtype != src.dtype or tuple(line.k.shape[1:]) != (n_kv, line.page_size, head_dim):
+            raise ValueError("map_prep: the cache line has another shape")
+        k_pool, v_pool, table, slot_len = line.k, line.v, line.page_table, line.slot_len
+        max_pages, page_size, ring = line.page_table.shape[1], line.page_size, line.ring
+    _lib.check(_lib.load().qnn_map_prep(
+        _p(src), dt_code(src), src.shape[1], _p(dst), dst.shape[1], T, n_heads, n_kv, maps, dim, vdim, head_dim, float(coef),
+        float(every), _p(tok_pos), _p(tok_slot), _p(k_pool), _p(v_pool), _p(table), max_pages, page_size, ring, _p(slot_len),
+        int(append), int(with_kv), _stream()), "map_prep")
+    return dst
+
+
+def map_difference(a: torch.Tensor, n_heads: int, vdim: int, lam: float, eps: float, scale: float) -> torch.Tensor:
+    """Per head of ``a`` ([rows, n_heads * 2 * head_dim]: the outputs of two maps, whose first ``vdim`` columns count): o = a_1 -
+    lam a_2, then o / sqrt(mean(o^2) + eps) * scale.  Returns [rows, n_heads * vdim]."""
+    _req(a, "a", None, 2)
+    T = a.shape[0]
+    hd = a.shape[1] // (2 * n_heads)
+    if a.shape[1] != 2 * n_heads * hd or hd < vdim:
+        raise ValueError("map_difference: shapes do not agree")
+    out = torch.empty((T, n_heads * vdim), dtype=a.dtype, device=a.device)
+    _lib.check(_lib.load().qnn_map_difference(_p(a), a.shape[1], hd, _p(out), out.shape[1], T, n_heads, vdim, float(lam), float(eps),
+                                              float(scale), dt_code(a), _stream()), "map_difference")
     return out
 
 

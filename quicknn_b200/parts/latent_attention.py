@@ -22,11 +22,15 @@ Options:
 * ``position`` (a ``rotary`` part of head size rot_dim): a rotated key part of rot_dim columns, shared by the heads and not
   normed, that W_dkv gives beside the latent; queries have rot_dim columns more per head (behind the ``dim`` others in
   the checkpoint's order).  A key row is then [rotated part | latent], one row per position in the cache, and serves as the
-  value row too: the read-out's first rot_dim columns meet no weight.  Without it the mixer has no positions.
+  value row too: the read-out's first rot_dim columns meet no weight.  Without it the mixer has no positions.  An interleaved
+  layout (columns 2i and 2i + 1 turn together) is a half-split one of reordered columns: the rows of the matrices that give the
+  rotated parts are reordered when the model is loaded, queries and key alike, which no score notices.
 * ``sink``: a learned number per head in the softmax's denominator (see ``attention``).
 * ``gate`` = "element": the concatenated heads are multiplied element by element by sigmoid(W_g x).  That gate does not
   commute with W_uv, so the values are formed from the read-out per head (one block-diagonal product with the gate in its
   epilogue) and W_o stays a matrix of its own.  W_g is then part of the stacked input product.
+* ``gate`` = "none": no gate.  W_o and W_uv are folded into one matrix unless that makes it more than twice as large as
+  the two.
 
 Rows are carried at head sizes that the tensor-core attention kernels take (64, 128, 256) where rot_dim + kv_rank fits one,
 with zero columns behind, when any of these options is on.
@@ -70,13 +74,16 @@ class LatentAttentionMixer(AttentionMixer):
         pos: Optional[PartSpec] = p.get("position")
         self.rotation = None if pos is None else POSITIONS.get(pos.kind)(pos)
         self.rot_dim = 0 if pos is None else int(self.rotation.rotary_dim)
-        self.element_gate = str(p.get("gate", "head")) == "element"
+        self.gate = str(p.get("gate", "head"))
+        if self.gate not in ("head", "element", "none"):
+            raise ValueError(f"latent attention: gate {self.gate!r} is not one of head, element, none")
+        self.element_gate = self.gate == "element"
         sink = bool(p.get("sink", False))
         # the form with key rows [rotated part | latent] prepared by one kernel, and values formed per head
-        self.by_head = self.rotation is not None or self.element_gate or sink
+        self.by_head = self.rotation is not None or self.gate != "head" or sink
         if self.by_head:
-            if pos is not None and (self.rotation.layout != "half" or self.rot_dim != self.rotation.head_dim):
-                raise ValueError("latent attention: the shared key part turns as a whole, in halves")
+            if pos is not None and self.rot_dim != self.rotation.head_dim:
+                raise ValueError("latent attention: the shared key part turns as a whole")
             self.rank_pad = carried_size(self.kv_rank + self.rot_dim)
         inner = PartSpec("attention", {
             "hidden_size": self.hidden, "n_heads": self.n_heads, "n_kv_heads": 1, "head_dim": self.rank_pad,
@@ -102,7 +109,10 @@ class LatentAttentionMixer(AttentionMixer):
         rot = 0 if pos is None else int(pos.params["head_dim"])
         out = {"dq": ((rq, W), M), "dq_norm": ((rq,), N), "uq": ((H * (d + rot), rq), M),
                "dkv": ((rkv + rot, W), M), "dkv_norm": ((rkv,), N), "uk": ((H * d, rkv), M), "uv": ((H * vd, rkv), M),
-               "gate": ((H * vd if str(p.get("gate", "head")) == "element" else H, W), M), "o": ((W, H * vd), M)}
+               "o": ((W, H * vd), M)}
+        gate = str(p.get("gate", "head"))
+        if gate != "none":
+            out["gate"] = ((H * vd if gate == "element" else H, W), M)
         if p.get("sink", False):
             out["sink"] = ((H,), cls.PARAM_ROLE_NORM)
         return out
@@ -141,10 +151,14 @@ class LatentAttentionMixer(AttentionMixer):
 
     def _load_by_head(self, tensors, compute_dtype, device) -> None:
         H, d, vd, r, rot, rp = self.n_heads, self.dim, self.vdim, self.kv_rank, self.rot_dim, self.rank_pad
-        rows = [tensors["dq"], tensors["dkv"]]
+        # half-split order of the rotated columns, which is what the kernel turns
+        order = torch.arange(rot, device=tensors["dkv"].device)
+        if self.rotation is not None and self.rotation.layout == "interleaved":
+            order = torch.cat([order[0::2], order[1::2]])
+        rows = [tensors["dq"], tensors["dkv"][:r], tensors["dkv"][r:][order]]
         if self.element_gate:
             rows.append(tensors["gate"])                          # q_rank | latent | rotated part | gate
-        else:
+        elif self.gate == "head":
             self.w_gate = tensors["gate"].contiguous()
         self.w_in = stack_rows(rows)
         self.norm_q = tensors["dq_norm"].contiguous()
@@ -153,13 +167,19 @@ class LatentAttentionMixer(AttentionMixer):
         uq = tensors["uq"].to(wide).view(H, d + rot, self.q_rank)
         uk = tensors["uk"].to(wide).view(H, d, r)
         w_qk = torch.zeros((H, rp, self.q_rank), dtype=wide, device=uq.device)
-        w_qk[:, :rot] = uq[:, d:]
+        w_qk[:, :rot] = uq[:, d:][:, order]
         w_qk[:, rot:rot + r] = torch.einsum("hdr,hdq->hrq", uk, uq[:, :d])
         self.w_qk = w_qk.reshape(H * rp, self.q_rank).to(keep).contiguous()
-        w_uv = torch.zeros((H, vd, rp), dtype=tensors["uv"].dtype, device=uq.device)
-        w_uv[:, :, rot:rot + r] = tensors["uv"].view(H, vd, r)
-        self.w_uv = w_uv
-        self.w_o = tensors["o"].contiguous()
+        if self.gate == "none" and self.hidden * rp <= 2 * vd * (rp + self.hidden):
+            w_ov = torch.zeros((self.hidden, H, rp), dtype=wide, device=uq.device)
+            w_ov[:, :, rot:rot + r] = torch.einsum("whv,hvr->whr", tensors["o"].to(wide).view(self.hidden, H, vd),
+                                                   tensors["uv"].to(wide).view(H, vd, r))
+            self.w_ov = w_ov.reshape(self.hidden, H * rp).to(keep).contiguous()
+        else:
+            w_uv = torch.zeros((H, vd, rp), dtype=tensors["uv"].dtype, device=uq.device)
+            w_uv[:, :, rot:rot + r] = tensors["uv"].view(H, vd, r)
+            self.w_uv = w_uv
+            self.w_o = tensors["o"].contiguous()
         if self.rotation is not None:
             self.rotation.prepare(device)
         why = (ops.attention_refusal(compute_dtype, H, 1, rp) or ops.linear_refusal(self.w_in.dtype, self.hidden))
@@ -189,12 +209,15 @@ class LatentAttentionMixer(AttentionMixer):
         rows = ops.latent_prep(a, rq, rq + r, self.norm_kv, self.eps, rot, self.rotation.inv_freq if rot else None, q, H, rp,
                                step.tok_pos, step.tok_slot, line, bool(line.writes and step.mode != "extend"), packed)
         o = self.attend(rows, step, line)                          # [T, heads * carried row]
+        if self.w_ov is not None:
+            return project(o, self.w_ov)
         if self.element_gate:
             o = ops.block_linear(o if o.dtype == self.w_uv.dtype else ops.cast(o, self.w_uv.dtype), self.w_uv,
                                  out_dtype=x.dtype, gate=a, gate_col0=rq + r + rot)
         else:
             o = ops.block_linear(o if o.dtype == self.w_uv.dtype else ops.cast(o, self.w_uv.dtype), self.w_uv, out_dtype=x.dtype)
-            ops.gate_heads(o, x, self.w_gate, H)
+            if self.gate == "head":
+                ops.gate_heads(o, x, self.w_gate, H)
         return project(o, self.w_o)
 
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
