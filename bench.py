@@ -272,7 +272,8 @@ def design_sizes(name, design="fuposun"):
     attention on the keys and values of the attention layer before it (all with the dense feed-forward); Gunirax's:
     six layers of which the second and third run twice (chunked sigmoid attention beside a lightning memory, and HGRN2,
     with dense and routed feed-forwards in turn); Linedra's: windowed attention beside a linear recurrence as wide as the
-    model, latent attention in every fourth layer, routed experts everywhere."""
+    model, latent attention in every fourth layer, routed experts everywhere; Vonulorn's: two gated delta rules, differential
+    attention, latent attention (all with the dense feed-forward)."""
     W, ff, heads, hd, kvh, layers, vocab, window = {
         "2b": (2304, 9216, 8, 256, 4, 8, 32768, 4096), "1b": (1536, 6144, 8, 128, 4, 8, 32768, 2048)}[name]
     rank, qr, d = (256, 768, 128) if name == "2b" else (128, 512, 64)
@@ -291,7 +292,7 @@ def design_sizes(name, design="fuposun"):
                  query_pre_attn_scalar=hd)
     if design == "fuposun":
         return [("fuposun", fupo), ("gemma2", gemma)]
-    if design == "linedra":
+    if design in ("linedra", "vonulorn"):
         rot = d // 2
         par = ("parallel", {"left": {"heads": heads, "kv_heads": kvh, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window}},
                             "right": {"width": W, "blocks": 8, "conv": 4}, "left_scale": 1.25, "right_scale": 0.75})
@@ -302,6 +303,14 @@ def design_sizes(name, design="fuposun"):
         line = dict(architecture="Linedra", vocab=vocab, width=W, embedding={"scale": W ** 0.5}, norm={"eps": 1e-6},
                     canon={"taps": 4}, residual_mult=0.5, logit_softcap=50.0,
                     layers=[{"type": t, "mixer": m, "mlp": lmoe} for t, m in ((par, lat, par, par) * layers)[:layers]])
+    if design == "vonulorn":
+        # the delta rule has the sizes of Fuposun's linear attention, differential attention the projections of Gemma 2's
+        delta = ("delta", {"heads": gla["heads"], "kv_heads": gla["heads"], "dim": d, "vdim": 2 * d, "conv": 4})
+        att = ("attention", {"heads": heads, "kv_heads": kvh, "dim": hd // 2, "vdim": hd, "scale": (hd // 2) ** -0.5, "softcap": 50.0,
+                             "diff": 0.35, "q_temp": {"coef": 0.1, "every": 1024}})
+        vonu = dict(architecture="Vonulorn", vocab=vocab, width=W, norm={"eps": 1e-6}, residual_mult=0.5,
+                    layers=[{"type": t, "mixer": m, "mlp": dense} for t, m in ((delta, delta, att, lat) * layers)[:layers]])
+        return [("vonulorn", vonu), ("fuposun", fupo), ("linedra", line), ("gemma2", gemma)]
     if design == "gunirax":
         # eight executed layers from six: the second and third run twice over (the loop).  Chunked sigmoid attention
         # with the other models' heads beside a lightning memory, HGRN2 layers, dense and routed feed-forwards.
@@ -433,7 +442,7 @@ def main():
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--skip-baseline", action="store_true", help="do not time the plain PyTorch / NumPy baselines")
-    ap.add_argument("--design", default=None, choices=["fuposun", "tumudra", "mubasun", "gunirax", "linedra"],
+    ap.add_argument("--design", default=None, choices=["fuposun", "tumudra", "mubasun", "gunirax", "linedra", "vonulorn"],
                     help="instead of the record: this design beside the library's other models at equal size "
                          "(prefill, decode, kernels)")
     ap.add_argument("--design-sizes", default="1b,2b", help="with --design: which of 1b, 2b")

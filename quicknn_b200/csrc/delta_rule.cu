@@ -448,18 +448,35 @@ delta_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __r
         }
 }
 
+constexpr size_t ALONE_BYTES = 120 * 1024;
+
+int sm_count() {
+    static int n = 0;
+    if (n == 0) {
+        int dev = 0;
+        if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) n = 148;
+    }
+    return n;
+}
+
 template <typename T, int RPT, int CPT, bool VEC>
 int scan_as(const void* q, const void* k, const void* v, long long ld, const float* inv, int ldi, float q_scale, const float* rec,
             const int* seq_row0, const int* seq_len, const int* slots, float* state, long long slot_stride, float* out,
             long long ldo, int B, int H, int G, int dim, int vdim, cudaStream_t st) {
     using Buf = ScanBuf<RPT, CPT>;
-    const size_t smem = Buf::bytes(RPT <= 16 ? 2 : 1);
+    // A block walks its sequence alone, so the scan takes as long as the slowest block: two on one SM while others are idle (the
+    // kernel in front still fills them when blocks are handed out) would set the pace.  Blocks that all fit one by one ask for
+    // more than half of an SM's shared memory.
+    const dim3 grid((vdim + Buf::COLS - 1) / Buf::COLS, H, B);
+    const bool alone = (long long)grid.x * H * B <= sm_count();
+    const size_t need = Buf::bytes(RPT <= 16 ? 2 : 1), smem = alone && need < ALONE_BYTES ? ALONE_BYTES : need;
     static bool set = false;
-    if (smem > 48 * 1024 && !set) {
-        cudaFuncSetAttribute(delta_scan_kernel<T, RPT, CPT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (!set) {
+        cudaFuncSetAttribute(delta_scan_kernel<T, RPT, CPT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             (int)(need > ALONE_BYTES ? need : ALONE_BYTES));
         set = true;
     }
-    launch_pdl(delta_scan_kernel<T, RPT, CPT, VEC>, dim3((vdim + Buf::COLS - 1) / Buf::COLS, H, B), dim3(SCAN_THREADS), smem, st,
+    launch_pdl(delta_scan_kernel<T, RPT, CPT, VEC>, grid, dim3(SCAN_THREADS), smem, st,
                (const T*)q, (const T*)k, (const T*)v, ld, inv, ldi, q_scale, rec, seq_row0, seq_len, slots, state, slot_stride, out,
                ldo, H, G, dim, vdim);
     QNN_LAUNCH_CHECK();

@@ -261,7 +261,7 @@ class OpTimer:
             flops = 2.0 * T * top * rows * W
             byts = float(used * rows * W * wgu.element_size() + _nbytes(x) + _nbytes(out))
         elif name == "causal_conv":
-            byts = float(2 * _nbytes(out) + _nbytes(a[1]))
+            byts = float(2 * _nbytes(out[0] if isinstance(out, tuple) else out) + _nbytes(a[1]))
         elif name == "block_linear":
             x, w, gate = a[0], a[1], kw.get("gate")
             flops = 2.0 * x.shape[0] * w.numel()
@@ -276,6 +276,23 @@ class OpTimer:
             C, rows = conv.shape[0], p.shape[0]
             flops = 2.0 * rows * w.numel()
             byts = float(_nbytes(w) + rows * C * (3 * p.element_size() + 4 * (conv.shape[1] + 2)))
+        elif name == "delta_scan":
+            rows, pre, n_seqs, H, G, dim, vdim = a[0], a[2], a[11], a[13], a[14], a[15], a[16]
+            T = rows.shape[0]
+            flops = 6.0 * T * H * dim * vdim                 # S^T k, S^T q and the update
+            byts = float(T * (2 * G * dim + H * vdim) * rows.element_size() + _nbytes(a[1]) + _nbytes(pre) + T * H * vdim * 4
+                         + 2 * n_seqs * H * dim * vdim * 4)
+        elif name == "delta_step":
+            p, x, w_ba, conv, H, dim, vdim = a[0], a[1], a[2], a[3], a[14], a[16], a[17]
+            flops = 6.0 * p.shape[0] * H * dim * vdim
+            byts = float(_nbytes(p) + _nbytes(x) + _nbytes(w_ba) + _nbytes(conv) + _nbytes(out)
+                         + p.shape[0] * 4 * (2 * H * dim * vdim + (conv.shape[1] + 1) * conv.shape[0]))
+        elif name == "map_prep":
+            append, with_kv = a[10], a[11]
+            T, wide = a[0].shape[0], a[0].element_size() * 2 * a[2] * a[6]
+            byts = float(_nbytes(a[0]) + _nbytes(out) + (T * wide if append else 0))
+        elif name == "map_difference":
+            byts = float(a[0].shape[0] * a[1] * a[2] * a[0].element_size() * 3)
         elif name == "latent_prep":
             row = a[3].numel() + int(a[5])               # latent and rotated part
             q, packed = a[7], kw.get("packed", a[14] if len(a) > 14 else None)

@@ -80,9 +80,9 @@ class DifferentialAttention(AttentionMixer):
     def forward(self, x: torch.Tensor, step, line) -> torch.Tensor:
         decode = step.mode == "decode"
         p = project(x, self.w_qkv)
-        # a step that continues sequences appends after its attention (``attend``)
+        # packed with keys and values for every step but a decode step, whose attention reads the cache; a step that continues
+        # sequences appends after its attention (``attend``)
         rows = ops.map_prep(p, self.real_heads, self.n_kv, MAPS, self.dim, self.vdim, self.head_dim, step.tok_pos, step.tok_slot, line,
-                            append=bool(line.writes and step.mode != "extend"), with_kv=not decode, coef=self.temp[0],
-                            every=self.temp[1])
+                            bool(line.writes and step.mode != "extend"), not decode, self.temp[0], self.temp[1])
         a = self.attend(rows, step, line)                                 # [T, heads * 2 * carried size]
         return project(ops.map_difference(a, self.real_heads, self.vdim, self.lam, self.eps, 1.0 - self.diff), self.w_o)
