@@ -9,7 +9,8 @@
 // never rounded.  n_kv query/key heads serve n_heads value heads.
 //
 //   qnn_delta_chunks   per chunk of 16 rows and value head: what does not depend on the state
-//   qnn_delta_scan     walks the chunks of every sequence in order, from the slot's state and back into it
+//   qnn_delta_scan     walks the chunks of every sequence in order, from the slot's state and back into it; bfloat16 rows on the
+//                      tensor cores with every float32 matrix in three bfloat16 parts, others on the FMA pipes
 //   qnn_delta_step     one token per sequence, everything between the input product and the output product in one kernel
 //
 // Chunks (Yang et al., "Parallelizing Linear Transformers with the Delta Rule over Sequence Length").  With S the state before a
@@ -132,7 +133,440 @@ delta_chunks_kernel(const T* __restrict__ q, const T* __restrict__ k, long long 
     }
 }
 
-// ---- the scan ---------------------------------------------------------------------------------------------------
+// ---- bfloat16 rows: the same on the tensor cores ---------------------------------------------------------------------
+// Keys and queries are bfloat16 numbers times a float32 factor per row, so a float32 matrix meets them on the tensor cores
+// without loss when it is cut into three bfloat16 numbers per element (hi + mid + lo holds 24 bits) and the factors are applied
+// to the results: x = hi + mid + lo costs three products with one exact factor and six with another float32 matrix (the three
+// smallest of nine terms lie below float32's rounding).  Accumulation is float32.
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], unsigned addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], unsigned addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+__device__ __forceinline__ float low_of(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float high_of(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
+struct Split3 { uint32_t h[4], m[4], l[4]; };
+__device__ __forceinline__ void split(float a, float b, uint32_t& h, uint32_t& m, uint32_t& l) {
+    h = pack2(a, b);
+    a -= low_of(h);
+    b -= high_of(h);
+    m = pack2(a, b);
+    l = pack2(a - low_of(m), b - high_of(m));
+}
+// two accumulator tiles (16 x 8 each, side by side) as the A operand of a product over those 16 columns
+__device__ __forceinline__ void split_tiles(const float (&x)[4], const float (&y)[4], Split3& s) {
+    split(x[0], x[1], s.h[0], s.m[0], s.l[0]);
+    split(x[2], x[3], s.h[1], s.m[1], s.l[1]);
+    split(y[0], y[1], s.h[2], s.m[2], s.l[2]);
+    split(y[2], y[3], s.h[3], s.m[3], s.l[3]);
+}
+__device__ __forceinline__ void cp16(unsigned dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src) : "memory");
+}
+
+// What a chunk leaves for the scan, per value head: T and A in three bfloat16 matrices each ([3][16][16]: row t, column j),
+// then per row P_t / |k_t|, P_t q_scale / |q_t|, D_16,t / |k_t|, and P_16: 3280 bytes.
+constexpr int TC_T = 0, TC_A = 3 * CK * CK * 2, TC_F = 2 * TC_A, TC_RECORD = TC_F + (3 * CK + 4) * 4;
+
+// a warp per (chunk, query/key head)
+__global__ void __launch_bounds__(128)
+delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, long long ld, const float* __restrict__ inv, int ldi,
+                       const float* __restrict__ pre, int ldp, const float* __restrict__ rate, const float* __restrict__ bias,
+                       float q_scale, const int* __restrict__ seq_row0, const int* __restrict__ seq_len,
+                       unsigned char* __restrict__ rec, int H, int G, int dim) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, j = lane & (CK - 1), half = lane >> 4;
+    const int dpad = (dim + 15) & ~15, pitch = dpad * 2 + 16;
+    const int own = 2 * CK * pitch + 3 * CK * (CK + 1) * 4;
+    unsigned char* mine = smem + (size_t)warp * own;
+    float* kk = reinterpret_cast<float*>(mine + 2 * CK * pitch);
+    float* qk = kk + CK * (CK + 1);
+    float* L = qk + CK * (CK + 1);
+    const int c = blockIdx.x * 4 + warp, g = blockIdx.y, b = blockIdx.z;
+    pdl_wait();
+    const int n = seq_len != nullptr ? seq_len[b] : 1, row0 = seq_row0 != nullptr ? seq_row0[b] : b, t0 = c * CK;
+    if (t0 >= n) return;                                      // (nothing below waits for another warp)
+    const int nt = min(CK, n - t0);
+    const int pieces = dpad / 8;
+    for (int i = lane; i < CK * pieces; i += 32) {
+        const int t = i / pieces, d = (i - t * pieces) * 8;
+        uint4 kv = make_uint4(0, 0, 0, 0), qv = kv;
+        if (t < nt && d < dim) {
+            const size_t at = (size_t)(row0 + t0 + t) * ld + (size_t)g * dim + d;
+            kv = *reinterpret_cast<const uint4*>(k + at);
+            qv = *reinterpret_cast<const uint4*>(q + at);
+        }
+        *reinterpret_cast<uint4*>(mine + t * pitch + d * 2) = kv;
+        *reinterpret_cast<uint4*>(mine + (CK + t) * pitch + d * 2) = qv;
+    }
+    float iq = 0.f, ik = 0.f;                                 // of row j
+    if (j < nt) {
+        const size_t row = (size_t)(row0 + t0 + j);
+        iq = inv[row * ldi + g] * q_scale;
+        ik = inv[row * ldi + G + g];
+    }
+    __syncwarp();
+    const unsigned kb = (unsigned)__cvta_generic_to_shared(mine), qb = kb + CK * pitch;
+    const int mi = lane >> 3, mr = lane & 7;                  // matrix and row that this lane addresses for ldmatrix
+    float akk[2][4], aqk[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) akk[i][e] = aqk[i][e] = 0.f;
+    for (int d = 0; d < dpad; d += 16) {
+        uint32_t ka[4], qa[4], kn[4];
+        ldsm4(ka, kb + ((mi & 1) * 8 + mr) * pitch + (d + (mi >> 1) * 8) * 2);      // rows as A
+        ldsm4(qa, qb + ((mi & 1) * 8 + mr) * pitch + (d + (mi >> 1) * 8) * 2);
+        ldsm4(kn, kb + ((mi >> 1) * 8 + mr) * pitch + (d + (mi & 1) * 8) * 2);      // rows as B
+        mma(akk[0], ka, kn[0], kn[1]);
+        mma(akk[1], ka, kn[2], kn[3]);
+        mma(aqk[0], qa, kn[0], kn[1]);
+        mma(aqk[1], qa, kn[2], kn[3]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int t = (lane >> 2) + (e >> 1) * 8, col = i * 8 + (lane & 3) * 2 + (e & 1);
+            const float kt = __shfl_sync(0xffffffffu, ik, t), qt = __shfl_sync(0xffffffffu, iq, t), kj = __shfl_sync(0xffffffffu, ik, col);
+            kk[t * (CK + 1) + col] = akk[i][e] * (kt * kj);
+            qk[t * (CK + 1) + col] = aqk[i][e] * (qt * kj);
+        }
+    __syncwarp();
+    const int per = H / G;
+    for (int s = 0; s < per; ++s) {
+        const int h = g * per + s;
+        unsigned char* out = rec + (record_of(row0, b, c) * H + h) * TC_RECORD;
+        bf16* oT = reinterpret_cast<bf16*>(out + TC_T);
+        bf16* oA = reinterpret_cast<bf16*>(out + TC_A);
+        float* oF = reinterpret_cast<float*>(out + TC_F);
+        float be = 0.f, ga = 1.f;
+        if (j < nt) {
+            const float* pr = pre + (size_t)(row0 + t0 + j) * ldp;
+            be = beta_of(pr[h]);
+            ga = decay_of(pr[H + h], rate[h], bias[h]);
+        }
+        auto put = [&](bf16* m, int t, float v) {
+            const bf16 hi = __float2bfloat16_rn(v);
+            const float r = v - __bfloat162float(hi);
+            const bf16 mid = __float2bfloat16_rn(r);
+            m[t * CK + j] = hi;
+            m[CK * CK + t * CK + j] = mid;
+            m[2 * CK * CK + t * CK + j] = __float2bfloat16_rn(r - __bfloat162float(mid));
+        };
+        float d = 1.f, p = 1.f, mine_p = 1.f;
+#pragma unroll
+        for (int t = 0; t < CK; ++t) {
+            const float gt = __shfl_sync(0xffffffffu, ga, t), bt = __shfl_sync(0xffffffffu, be, t);
+            if (t > j) d *= gt;
+            p *= gt;
+            if (t == j) mine_p = p;
+            if (half == 0) L[t * (CK + 1) + j] = t > j ? bt * d * kk[t * (CK + 1) + j] : 0.f;
+            else put(oA, t, t >= j ? d * qk[t * (CK + 1) + j] : 0.f);
+        }
+        if (half == 0) {
+            oF[j] = mine_p * ik;
+            oF[CK + j] = mine_p * iq;
+            oF[2 * CK + j] = d * ik;
+            if (j < 4) oF[3 * CK + j] = p;
+        }
+        __syncwarp();
+        if (half == 0) {
+            float x[CK];
+#pragma unroll
+            for (int t = 0; t < CK; ++t) {
+                float s0 = t == j ? 1.f : 0.f;
+#pragma unroll
+                for (int i = 0; i < t; ++i) s0 -= L[t * (CK + 1) + i] * x[i];
+                x[t] = s0;
+                put(oT, t, s0 * be);
+            }
+        }
+        __syncwarp();
+    }
+}
+
+// The scan.  A block owns 16 value columns of one (sequence, head) as S^T, 16 columns x key channels.  Four warps have a quarter
+// of the key channels each (KS times 16) as accumulator tiles, which serve as the A operand of the products with keys and queries
+// when they are split; their partial K S meet in shared memory (one barrier per chunk), and each of the four then forms X, U = T X
+// and its quarter of the update by itself, all in registers.  Q S is formed in the shadow of that; a fifth warp turns it into the
+// outputs a chunk later, a sixth fetches the chunks two ahead.
+constexpr int TC_WORKERS = 4, TC_THREADS = 32 * (TC_WORKERS + 2), TC_STAGES = 4;
+
+template <int KS>
+struct TcStage {
+    static constexpr int PITCH = KS * 128 + 16, VPITCH = 48;   // bytes: rows four banks apart
+    static constexpr int K = 0, Q = CK * PITCH, V = 2 * CK * PITCH, R = V + CK * VPITCH, BYTES = R + TC_RECORD;
+    static constexpr int RED = TC_STAGES * BYTES;              // [2][k, q][workers][2 tiles][32 lanes] float4
+    static constexpr int TOTAL = RED + 2 * 2 * TC_WORKERS * 2 * 32 * 16;
+    static_assert(BYTES % 16 == 0, "stages on 16 bytes");
+};
+
+template <int KS>
+__global__ void __launch_bounds__(TC_THREADS)
+delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v, long long ld,
+                     const unsigned char* __restrict__ rec, const int* __restrict__ seq_row0, const int* __restrict__ seq_len,
+                     const int* __restrict__ slots, float* __restrict__ state, long long slot_stride, float* __restrict__ out,
+                     long long ldo, int H, int G, int dim, int vdim) {
+    using St = TcStage<KS>;
+    extern __shared__ __align__(16) unsigned char smem[];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, t4 = lane & 3, gr = lane >> 2, mi = lane >> 3, mr = lane & 7;
+    const int h = blockIdx.y, c0 = blockIdx.x * 16, b = blockIdx.z;
+    for (int i = tid; i < St::RED / 16; i += TC_THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    const int n = seq_len != nullptr ? seq_len[b] : 1, row0 = seq_row0 != nullptr ? seq_row0[b] : b, slot = slots[b];
+    if (n <= 0) return;
+    if (slot < 0) {                                           // rows of no sequence
+        const int live = min(16, vdim - c0);
+        for (int i = tid; i < n * live; i += TC_THREADS)
+            out[(size_t)(row0 + i / live) * ldo + (size_t)h * vdim + c0 + i % live] = 0.f;
+        return;
+    }
+    const int chunks = (n + CK - 1) / CK, g = h / (H / G);
+    const unsigned base = (unsigned)__cvta_generic_to_shared(smem);
+    float4* red = reinterpret_cast<float4*>(smem + St::RED);
+    auto red_at = [&](int parity, int which, int w, int tile) { return red + (((parity * 2 + which) * TC_WORKERS + w) * 2 + tile) * 32 + lane; };
+    __syncthreads();                                          // the stages are zero: rows and columns that nothing fills stay so
+    if (warp == TC_WORKERS + 1) {
+        // ---- the loader.  Rows beyond the sequence keep what an earlier chunk left (or zeros): finite numbers whose factors are 0
+        const int pieces = dim / 8, vp = min(2, (vdim - c0) / 8);
+        auto load = [&](int c) {
+            if (c < chunks) {
+                const unsigned st = base + (c % TC_STAGES) * St::BYTES;
+                const int nt = min(CK, n - c * CK);
+                const size_t first = (size_t)(row0 + c * CK);
+                for (int i = lane; i < nt * pieces; i += 32) {
+                    const int t = i / pieces, d = i - t * pieces;
+                    const size_t at = (first + t) * ld + (size_t)g * dim + d * 8;
+                    cp16(st + St::K + t * St::PITCH + d * 16, k + at);
+                    cp16(st + St::Q + t * St::PITCH + d * 16, q + at);
+                }
+                {
+                    const int t = lane >> 1, p = lane & 1;
+                    if (t < nt && p < vp)
+                        cp16(st + St::V + t * St::VPITCH + p * 16, v + (first + t) * ld + (size_t)h * vdim + c0 + p * 8);
+                }
+                const unsigned char* r = rec + (record_of(row0, b, c) * H + h) * TC_RECORD;
+                for (int i = lane; i < TC_RECORD / 16; i += 32) cp16(st + St::R + i * 16, r + i * 16);
+            }
+            asm volatile("cp.async.commit_group;\n" ::: "memory");
+        };
+        load(0);
+        load(1);
+        asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        __syncthreads();
+        for (int c = 0; c < chunks; ++c) {
+            load(c + 2);                                      // (the stage of chunk c - 2: everybody is past its barrier c - 1)
+            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+            __syncthreads();
+        }
+        __syncthreads();
+        return;
+    }
+    // X^T = V^T - (P K S)^T of chunk c from the workers' partial sums, split for a product over the chunk's rows
+    auto form_x = [&](int c, Split3& x) {
+        const unsigned st = base + (c % TC_STAGES) * St::BYTES;
+        const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
+        uint32_t vr[4];
+        ldsm4t(vr, st + St::V + ((mi >> 1) * 8 + mr) * St::VPITCH + (mi & 1) * 16);
+        float xs[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            float4 m = *red_at(c & 1, 0, 0, i);
+#pragma unroll
+            for (int w = 1; w < TC_WORKERS; ++w) {
+                const float4 o = *red_at(c & 1, 0, w, i);
+                m.x += o.x; m.y += o.y; m.z += o.z; m.w += o.w;
+            }
+            const float2 pk = *reinterpret_cast<const float2*>(f + i * 8 + t4 * 2);
+            xs[i][0] = low_of(vr[2 * i]) - pk.x * m.x;
+            xs[i][1] = high_of(vr[2 * i]) - pk.y * m.y;
+            xs[i][2] = low_of(vr[2 * i + 1]) - pk.x * m.z;
+            xs[i][3] = high_of(vr[2 * i + 1]) - pk.y * m.w;
+        }
+        split_tiles(xs[0], xs[1], x);
+    };
+    // y += (x times the 16 x 16 matrix whose three parts are at `m`)^T, the small terms first
+    auto times = [&](const Split3& x, const uint32_t (&mh)[4], const uint32_t (&mm)[4], const uint32_t (&ml)[4], float (&y)[2][4]) {
+        float z[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) z[i][e] = 0.f;
+            mma(z[i], x.l, mh[2 * i], mh[2 * i + 1]);
+            mma(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
+            mma(z[i], x.h, ml[2 * i], ml[2 * i + 1]);
+            mma(y[i], x.h, mm[2 * i], mm[2 * i + 1]);
+            mma(z[i], x.m, mm[2 * i], mm[2 * i + 1]);
+            mma(y[i], x.h, mh[2 * i], mh[2 * i + 1]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[i][e] += z[i][e];
+    };
+    auto load_matrix = [&](int c, int at, uint32_t (&mh)[4], uint32_t (&mm)[4], uint32_t (&ml)[4]) {
+        const unsigned a = base + (c % TC_STAGES) * St::BYTES + St::R + at + ((mi >> 1) * 8 + mr) * (CK * 2) + (mi & 1) * 16;
+        ldsm4(mh, a);
+        ldsm4(mm, a + CK * CK * 2);
+        ldsm4(ml, a + 2 * CK * CK * 2);
+    };
+    if (warp == TC_WORKERS) {
+        // ---- the outputs: O = P Q S + A U, a chunk behind
+        Split3 us;
+        uint32_t ah[4], am[4], al[4];
+        float2 pq[2];
+        auto finish = [&](int c) {
+            float o[2][4];
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                float4 m = *red_at(c & 1, 1, 0, i);
+#pragma unroll
+                for (int w = 1; w < TC_WORKERS; ++w) {
+                    const float4 x = *red_at(c & 1, 1, w, i);
+                    m.x += x.x; m.y += x.y; m.z += x.z; m.w += x.w;
+                }
+                o[i][0] = pq[i].x * m.x;
+                o[i][1] = pq[i].y * m.y;
+                o[i][2] = pq[i].x * m.z;
+                o[i][3] = pq[i].y * m.w;
+            }
+            times(us, ah, am, al, o);
+            const int nt = min(CK, n - c * CK);
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = i * 8 + t4 * 2 + (e & 1), col = c0 + gr + (e >> 1) * 8;
+                    if (t < nt && col < vdim) out[(size_t)(row0 + c * CK + t) * ldo + (size_t)h * vdim + col] = o[i][e];
+                }
+        };
+        __syncthreads();
+        for (int c = 0; c < chunks; ++c) {
+            __syncthreads();
+            if (c > 0) finish(c - 1);
+            Split3 x;
+            form_x(c, x);
+            uint32_t th[4], tm[4], tl[4];
+            load_matrix(c, TC_T, th, tm, tl);
+            float u[2][4];
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) u[i][e] = 0.f;
+            times(x, th, tm, tl, u);
+            split_tiles(u[0], u[1], us);
+            load_matrix(c, TC_A, ah, am, al);                 // (the stage may be filled anew before the outputs are formed)
+            const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) pq[i] = *reinterpret_cast<const float2*>(f + CK + i * 8 + t4 * 2);
+        }
+        __syncthreads();
+        finish(chunks - 1);
+        return;
+    }
+    // ---- a worker: key channels d0 .. d0 + 16 KS of S^T
+    const int d0 = warp * KS * 16;
+    float* my_state = state + (size_t)slot * slot_stride + (size_t)h * dim * vdim + c0;
+    float S[2 * KS][4];
+#pragma unroll
+    for (int i = 0; i < 2 * KS; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = d0 + i * 8 + t4 * 2 + (e & 1), col = gr + (e >> 1) * 8;
+            S[i][e] = (d < dim && c0 + col < vdim) ? my_state[(size_t)d * vdim + col] : 0.f;
+        }
+    __syncthreads();
+    for (int c = 0; c < chunks; ++c) {
+        const unsigned st = base + (c % TC_STAGES) * St::BYTES;
+        const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
+        Split3 s[KS];
+        float m[2][4];
+        auto product = [&](unsigned rows) {                   // m = S^T times the chunk's rows, over this warp's channels
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) m[i][e] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) {
+                uint32_t r[4];
+                ldsm4(r, rows + ((mi >> 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi & 1) * 8) * 2);
+                mma(m[0], s[ks].l, r[0], r[1]);
+                mma(m[1], s[ks].l, r[2], r[3]);
+                mma(m[0], s[ks].m, r[0], r[1]);
+                mma(m[1], s[ks].m, r[2], r[3]);
+                mma(m[0], s[ks].h, r[0], r[1]);
+                mma(m[1], s[ks].h, r[2], r[3]);
+            }
+        };
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) split_tiles(S[2 * ks], S[2 * ks + 1], s[ks]);
+        product(st + St::K);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) *red_at(c & 1, 0, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
+        __syncthreads();
+        Split3 x;
+        form_x(c, x);
+        uint32_t th[4], tm[4], tl[4];
+        load_matrix(c, TC_T, th, tm, tl);
+        float u[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) u[i][e] = 0.f;
+        times(x, th, tm, tl, u);
+        product(st + St::Q);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) *red_at(c & 1, 1, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
+        const float pc = f[3 * CK];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const float2 dk = *reinterpret_cast<const float2*>(f + 2 * CK + i * 8 + t4 * 2);
+            u[i][0] *= dk.x;
+            u[i][1] *= dk.y;
+            u[i][2] *= dk.x;
+            u[i][3] *= dk.y;
+        }
+        Split3 y;
+        split_tiles(u[0], u[1], y);
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+            uint32_t r[4];
+            ldsm4t(r, st + St::K + ((mi & 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi >> 1) * 8) * 2);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) S[2 * ks + i][e] *= pc;
+                mma(S[2 * ks + i], y.l, r[2 * i], r[2 * i + 1]);
+                mma(S[2 * ks + i], y.m, r[2 * i], r[2 * i + 1]);
+                mma(S[2 * ks + i], y.h, r[2 * i], r[2 * i + 1]);
+            }
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2 * KS; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int d = d0 + i * 8 + t4 * 2 + (e & 1), col = gr + (e >> 1) * 8;
+            if (d < dim && c0 + col < vdim) my_state[(size_t)d * vdim + col] = S[i][e];
+        }
+}
+
+// ---- the scan on the FMA pipes (float32 rows, odd sizes) ----------------------------------------------------------------
 // A block owns 16 * CPT value columns of one (sequence, head).  Eight lanes share a group of CPT columns, each with an eighth
 // of the key channels of the state in registers (RPT of them); a warp has four groups, and everything of a chunk but the
 // staging happens inside a warp: the products of the state with the chunk's keys and queries (partial sums of four rows and
@@ -448,7 +882,7 @@ delta_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __r
         }
 }
 
-constexpr size_t ALONE_BYTES = 120 * 1024;
+constexpr int MAX_SMEM = 227 * 1024;
 
 int sm_count() {
     static int n = 0;
@@ -459,21 +893,42 @@ int sm_count() {
     return n;
 }
 
+// Shared memory that a scan's blocks ask for.  A block walks its sequence by itself, so a scan takes as long as its slowest block:
+// several on one SM while others are idle (the kernel in front still fills them when blocks are handed out) would set the pace.
+// Up to four rounds of blocks ask for so much that no SM takes more than its share.
+size_t spread(long long blocks, size_t need) {
+    const long long share = (blocks + sm_count() - 1) / sm_count();
+    if (share > 4) return need;
+    const size_t least = (size_t)(228 * 1024) / (size_t)(share + 1);
+    return need > least ? need : least;
+}
+
+template <int KS>
+int scan_tc(const void* q, const void* k, const void* v, long long ld, const void* rec, const int* seq_row0, const int* seq_len,
+            const int* slots, float* state, long long slot_stride, float* out, long long ldo, int B, int H, int G, int dim, int vdim,
+            cudaStream_t st) {
+    const dim3 grid((vdim + 15) / 16, H, B);
+    const size_t smem = spread((long long)grid.x * H * B, TcStage<KS>::TOTAL);
+    static bool set = false;
+    if (!set) {
+        cudaFuncSetAttribute(delta_scan_tc_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
+        set = true;
+    }
+    launch_pdl(delta_scan_tc_kernel<KS>, grid, dim3(TC_THREADS), smem, st, (const bf16*)q, (const bf16*)k, (const bf16*)v, ld,
+               (const unsigned char*)rec, seq_row0, seq_len, slots, state, slot_stride, out, ldo, H, G, dim, vdim);
+    QNN_LAUNCH_CHECK();
+}
+
 template <typename T, int RPT, int CPT, bool VEC>
 int scan_as(const void* q, const void* k, const void* v, long long ld, const float* inv, int ldi, float q_scale, const float* rec,
             const int* seq_row0, const int* seq_len, const int* slots, float* state, long long slot_stride, float* out,
             long long ldo, int B, int H, int G, int dim, int vdim, cudaStream_t st) {
     using Buf = ScanBuf<RPT, CPT>;
-    // A block walks its sequence alone, so the scan takes as long as the slowest block: two on one SM while others are idle (the
-    // kernel in front still fills them when blocks are handed out) would set the pace.  Blocks that all fit one by one ask for
-    // more than half of an SM's shared memory.
     const dim3 grid((vdim + Buf::COLS - 1) / Buf::COLS, H, B);
-    const bool alone = (long long)grid.x * H * B <= sm_count();
-    const size_t need = Buf::bytes(RPT <= 16 ? 2 : 1), smem = alone && need < ALONE_BYTES ? ALONE_BYTES : need;
+    const size_t smem = spread((long long)grid.x * H * B, Buf::bytes(RPT <= 16 ? 2 : 1));
     static bool set = false;
     if (!set) {
-        cudaFuncSetAttribute(delta_scan_kernel<T, RPT, CPT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             (int)(need > ALONE_BYTES ? need : ALONE_BYTES));
+        cudaFuncSetAttribute(delta_scan_kernel<T, RPT, CPT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
         set = true;
     }
     launch_pdl(delta_scan_kernel<T, RPT, CPT, VEC>, grid, dim3(SCAN_THREADS), smem, st,
@@ -754,33 +1209,50 @@ int step_rows(const StepArgs& a, int splits, cudaStream_t st) {
 
 // q, k: [rows, G * dim], v: [rows, H * vdim] of `dtype`, one row pitch `ld`; inv: [rows, ldi] with 1 / length of the G query heads,
 // then of the G key heads; seq_row0, seq_len: first row and row count of the B sequences (both null: row b alone); pre: [rows, ldp] with b of the H heads, then a of the H heads; rate, bias: [H] float32 (rate =
-// exp(A)); rec: at least (T / 16 + B) * H records of 544 floats.  longest: the most rows of a sequence.  dim up to 256.
+// exp(A)); rec: at least (T / 16 + B) * H records of 3280 bytes (tensor_cores) or 544 floats.  longest: the most rows of a
+// sequence.  dim up to 256.  tensor_cores: bfloat16 rows, dim and vdim multiples of 8, everything on 16 bytes.
 QNN_API int qnn_delta_chunks(const void* q, const void* k, long long ld, int dtype, const float* inv, int ldi, const float* pre,
                              int ldp, const float* rate, const float* bias, float q_scale, const int* seq_row0, const int* seq_len,
-                             float* rec, int B, int longest, int H, int G, int dim, cudaStream_t st) {
+                             void* rec, int B, int longest, int H, int G, int dim, int tensor_cores, cudaStream_t st) {
     if (B <= 0 || longest <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > MAX_DIM || B > 65535 || G > 65535 || ldi < 2 * G || ldp < 2 * H)
         return QNN_ERR_ARGUMENT;
     if ((seq_row0 == nullptr) != (seq_len == nullptr)) return QNN_ERR_ARGUMENT;
+    if (tensor_cores) {
+        if (dtype != QNN_DT_BF16 || dim % 8 || ld % 8 || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)rec) & 15)) return QNN_ERR_ARGUMENT;
+        const int dpad = (dim + 15) & ~15;
+        const size_t smem = (size_t)4 * (2 * CK * (dpad * 2 + 16) + 3 * CK * (CK + 1) * 4);
+        static bool set = false;
+        if (!set) {
+            cudaFuncSetAttribute(delta_chunks_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
+            set = true;
+        }
+        launch_pdl(delta_chunks_tc_kernel, dim3((unsigned)((longest + 4 * CK - 1) / (4 * CK)), G, B), dim3(128), smem, st,
+                   (const bf16*)q, (const bf16*)k, ld, inv, ldi, pre, ldp, rate, bias, q_scale, seq_row0, seq_len,
+                   (unsigned char*)rec, H, G, dim);
+        QNN_LAUNCH_CHECK();
+    }
     const int pitch = ((dim + 3) & ~3) + 4;
     const size_t smem = ((size_t)2 * CK * pitch + 6 * CK * (CK + 1)) * sizeof(float);
     if (smem > 48 * 1024) return QNN_ERR_UNSUPPORTED;
     const dim3 grid((unsigned)((longest + CK - 1) / CK), G, B);
     if (dtype == QNN_DT_BF16)
         launch_pdl(delta_chunks_kernel<bf16>, grid, dim3(128), smem, st, (const bf16*)q, (const bf16*)k, ld, inv, ldi, pre, ldp,
-                   rate, bias, q_scale, seq_row0, seq_len, rec, H, G, dim);
+                   rate, bias, q_scale, seq_row0, seq_len, (float*)rec, H, G, dim);
     else
         launch_pdl(delta_chunks_kernel<float>, grid, dim3(128), smem, st, (const float*)q, (const float*)k, ld, inv, ldi, pre, ldp,
-                   rate, bias, q_scale, seq_row0, seq_len, rec, H, G, dim);
+                   rate, bias, q_scale, seq_row0, seq_len, (float*)rec, H, G, dim);
     QNN_LAUNCH_CHECK();
 }
 
 // The same rows; slots: the state slot of each sequence (negative: nothing is read or written); state: slot s's
 // [H, dim, vdim] floats at state + s * slot_stride; out: [rows, ldo] float32, H * vdim columns; cpt: 16 or 32 value columns per
-// block (1 or 2: many sequences fill the device with the wider ones, which read the rows half as often).
+// block (1 or 2: many sequences fill the device with the wider ones, which read the rows half as often).  tensor_cores: rec as
+// qnn_delta_chunks left it with the same; cpt, inv and q_scale are not read then.
 QNN_API int qnn_delta_scan(const void* q, const void* k, const void* v, long long ld, int dtype, const float* inv, int ldi,
-                           float q_scale, const float* rec, const int* seq_row0, const int* seq_len, const int* slots, float* state,
+                           float q_scale, const void* rec_, const int* seq_row0, const int* seq_len, const int* slots, float* state,
                            long long slot_stride, float* out, long long ldo, int B, int H, int G, int dim, int vdim, int cpt,
+                           int tensor_cores,
                            cudaStream_t st) {
     if (B <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > MAX_DIM || vdim <= 0 || B > 65535 || H > 65535 || ldi < 2 * G ||
@@ -788,6 +1260,13 @@ QNN_API int qnn_delta_scan(const void* q, const void* k, const void* v, long lon
         return QNN_ERR_ARGUMENT;
     const size_t es = dtype == QNN_DT_BF16 ? 2 : 4;
     const bool vec = dim % 8 == 0 && vdim % 8 == 0 && (ld * es) % 16 == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) == 0;
+    if (tensor_cores) {
+        if (dtype != QNN_DT_BF16 || !vec || ((uintptr_t)rec_ & 15)) return QNN_ERR_ARGUMENT;
+        if (dim <= 64) return scan_tc<1>(q, k, v, ld, rec_, seq_row0, seq_len, slots, state, slot_stride, out, ldo, B, H, G, dim, vdim, st);
+        if (dim <= 128) return scan_tc<2>(q, k, v, ld, rec_, seq_row0, seq_len, slots, state, slot_stride, out, ldo, B, H, G, dim, vdim, st);
+        return scan_tc<4>(q, k, v, ld, rec_, seq_row0, seq_len, slots, state, slot_stride, out, ldo, B, H, G, dim, vdim, st);
+    }
+    const float* rec = (const float*)rec_;
     const int rpt = (dim + SHARE - 1) / SHARE;
 #define QNN_DS(T, R, C, VV) \
     return scan_as<T, R, C, VV>(q, k, v, ld, inv, ldi, q_scale, rec, seq_row0, seq_len, slots, state, slot_stride, out, ldo, B, H, \

@@ -134,9 +134,9 @@ _SIGNATURES: Dict[str, list] = {
                                 c_vp, c_ll, c_int, c_int, c_int, c_vp, c_int, c_vp],
     "qnn_sigattn_prefill_ranges": [c_int, c_int, c_int, c_int, c_int, c_int, c_vp],
     "qnn_delta_chunks": [c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_vp, c_int, c_vp, c_vp, c_float, c_vp, c_vp, c_vp, c_int, c_int,
-                         c_int, c_int, c_int, c_vp],
+                         c_int, c_int, c_int, c_int, c_vp],
     "qnn_delta_scan": [c_vp, c_vp, c_vp, c_ll, c_int, c_vp, c_int, c_float, c_vp, c_vp, c_vp, c_vp, c_vp, c_ll, c_vp, c_ll, c_int,
-                       c_int, c_int, c_int, c_int, c_int, c_vp],
+                       c_int, c_int, c_int, c_int, c_int, c_int, c_vp],
     "qnn_delta_step": [c_vp, c_int, c_ll, c_vp, c_int, c_vp, c_int, c_vp, c_int, c_int, c_vp, c_vp, c_vp, c_int, c_float, c_float,
                        c_float, c_vp, c_ll, c_ll, c_vp, c_vp, c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_vp],
     "qnn_map_prep": [c_vp, c_int, c_ll, c_vp, c_ll, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_vp, c_vp,

@@ -1842,7 +1842,8 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_
 
 
 DELTA_CHUNK = 16             # rows of a chunk of the delta rule's scan
-DELTA_RECORD = 2 * DELTA_CHUNK * DELTA_CHUNK + 2 * DELTA_CHUNK
+DELTA_RECORD, DELTA_RECORD_TC = 4 * (2 * DELTA_CHUNK * DELTA_CHUNK + 2 * DELTA_CHUNK), 3280      # bytes per chunk and value head
+DELTA_TENSOR_CORES = True    # bfloat16 rows: the scan on the tensor cores (tests switch it off to compare)
 
 
 def delta_scan(rows: torch.Tensor, inv: torch.Tensor, pre: torch.Tensor, rate: torch.Tensor, bias: torch.Tensor, q_scale: float,
@@ -1870,19 +1871,21 @@ def delta_scan(rows: torch.Tensor, inv: torch.Tensor, pre: torch.Tensor, rate: t
     if (seq_row0 is None) != (seq_len is None) or (seq_row0 is None and T < n_seqs):
         raise ValueError("delta_scan: first rows and row counts come together, or a row per sequence")
     longest = int(longest) if seq_row0 is not None else 1
-    rec = torch.empty((T // DELTA_CHUNK + n_seqs) * n_heads * DELTA_RECORD, dtype=torch.float32, device=rows.device)
+    tc = DELTA_TENSOR_CORES and rows.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and rows.shape[1] % 8 == 0
+    rec = torch.empty((T // DELTA_CHUNK + n_seqs) * n_heads * (DELTA_RECORD_TC if tc else DELTA_RECORD), dtype=torch.uint8,
+                      device=rows.device)
     out = torch.empty((T, n_heads * vdim), dtype=torch.float32, device=rows.device)
     L = _lib.load()
     k0, v0 = n_kv * dim, 2 * n_kv * dim
     _lib.check(L.qnn_delta_chunks(_p(rows), _col_ptr(rows, k0), rows.shape[1], dt_code(rows), _p(inv), inv.shape[1], _p(pre),
                                   pre.shape[1], _p(rate), _p(bias), float(q_scale), _p(seq_row0), _p(seq_len), _p(rec), n_seqs,
-                                  longest, n_heads, n_kv, dim, _stream()), "delta_chunks")
+                                  longest, n_heads, n_kv, dim, int(tc), _stream()), "delta_chunks")
     # 16 value columns per block until they fill the device twice over
     wide = n_seqs * n_heads * -(-vdim // 16) > 2 * _sm_count(rows.device)
     _lib.check(L.qnn_delta_scan(_p(rows), _col_ptr(rows, k0), _col_ptr(rows, v0), rows.shape[1], dt_code(rows), _p(inv), inv.shape[1],
                                 float(q_scale), _p(rec), _p(seq_row0), _p(seq_len), _p(slots),
                                 ctypes.c_void_p(state.data_ptr() + 4 * state_col0), state.stride(0), _p(out), out.shape[1], n_seqs,
-                                n_heads, n_kv, dim, vdim, 2 if wide else 1, _stream()), "delta_scan")
+                                n_heads, n_kv, dim, vdim, 2 if wide else 1, int(tc), _stream()), "delta_scan")
     return out
 
 
