@@ -147,7 +147,7 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], unsigned addr) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile(
+    asm(
         "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
         : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
         : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -302,9 +302,9 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
 // The scan.  A block owns 16 value columns of one (sequence, head) as S^T, 16 columns x key channels.  Four warps have a quarter
 // of the key channels each (KS times 16) as accumulator tiles, which serve as the A operand of the products with keys and queries
 // when they are split; their partial K S meet in shared memory (one barrier per chunk), and each of the four then forms X, U = T X
-// and its quarter of the update by itself, all in registers.  Q S is formed in the shadow of that; a fifth warp turns it into the
-// outputs a chunk later, a sixth fetches the chunks two ahead.
-constexpr int TC_WORKERS = 4, TC_THREADS = 32 * (TC_WORKERS + 2), TC_STAGES = 4;
+// and its quarter of the update by itself, all in registers.  Q S is formed in the shadow of that; two more warps take alternate
+// chunks and turn it into the outputs a chunk later; the last warp fetches chunks ahead.
+constexpr int TC_WORKERS = 4, TC_READERS = 2, TC_THREADS = 32 * (TC_WORKERS + TC_READERS + 1), TC_STAGES = 6, TC_AHEAD = TC_STAGES - 2;
 
 template <int KS>
 struct TcStage {
@@ -340,19 +340,22 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
     float4* red = reinterpret_cast<float4*>(smem + St::RED);
     auto red_at = [&](int parity, int which, int w, int tile) { return red + (((parity * 2 + which) * TC_WORKERS + w) * 2 + tile) * 32 + lane; };
     __syncthreads();                                          // the stages are zero: rows and columns that nothing fills stay so
-    if (warp == TC_WORKERS + 1) {
+    if (warp == TC_WORKERS + TC_READERS) {
         // ---- the loader.  Rows beyond the sequence keep what an earlier chunk left (or zeros): finite numbers whose factors are 0
         const int pieces = dim / 8, vp = min(2, (vdim - c0) / 8);
+        const int at_once = 32 / pieces, tl = lane / pieces, dl = lane - tl * pieces;        // rows side by side; this lane's
         auto load = [&](int c) {
             if (c < chunks) {
                 const unsigned st = base + (c % TC_STAGES) * St::BYTES;
                 const int nt = min(CK, n - c * CK);
                 const size_t first = (size_t)(row0 + c * CK);
-                for (int i = lane; i < nt * pieces; i += 32) {
-                    const int t = i / pieces, d = i - t * pieces;
-                    const size_t at = (first + t) * ld + (size_t)g * dim + d * 8;
-                    cp16(st + St::K + t * St::PITCH + d * 16, k + at);
-                    cp16(st + St::Q + t * St::PITCH + d * 16, q + at);
+                if (tl < at_once) {
+                    size_t at = (first + tl) * ld + (size_t)g * dim + dl * 8;
+                    unsigned to = st + tl * St::PITCH + dl * 16;
+                    for (int t = tl; t < nt; t += at_once, at += at_once * ld, to += at_once * St::PITCH) {
+                        cp16(to + St::K, k + at);
+                        cp16(to + St::Q, q + at);
+                    }
                 }
                 {
                     const int t = lane >> 1, p = lane & 1;
@@ -364,13 +367,12 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
             }
             asm volatile("cp.async.commit_group;\n" ::: "memory");
         };
-        load(0);
-        load(1);
-        asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+        for (int c = 0; c < TC_AHEAD; ++c) load(c);
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(TC_AHEAD - 1) : "memory");
         __syncthreads();
         for (int c = 0; c < chunks; ++c) {
-            load(c + 2);                                      // (the stage of chunk c - 2: everybody is past its barrier c - 1)
-            asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+            load(c + TC_AHEAD);                               // (the stage of chunk c - 2: everybody is past its barrier c - 1)
+            asm volatile("cp.async.wait_group %0;\n" ::"n"(TC_AHEAD - 1) : "memory");
             __syncthreads();
         }
         __syncthreads();
@@ -401,18 +403,19 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
     };
     // y += (x times the 16 x 16 matrix whose three parts are at `m`)^T, the small terms first
     auto times = [&](const Split3& x, const uint32_t (&mh)[4], const uint32_t (&mm)[4], const uint32_t (&ml)[4], float (&y)[2][4]) {
-        float z[2][4];
+        float z[2][4] = {};
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
+        for (int i = 0; i < 2; ++i) mma(z[i], x.l, mh[2 * i], mh[2 * i + 1]);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) z[i][e] = 0.f;
-            mma(z[i], x.l, mh[2 * i], mh[2 * i + 1]);
-            mma(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
-            mma(z[i], x.h, ml[2 * i], ml[2 * i + 1]);
-            mma(y[i], x.h, mm[2 * i], mm[2 * i + 1]);
-            mma(z[i], x.m, mm[2 * i], mm[2 * i + 1]);
-            mma(y[i], x.h, mh[2 * i], mh[2 * i + 1]);
-        }
+        for (int i = 0; i < 2; ++i) mma(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) mma(z[i], x.h, ml[2 * i], ml[2 * i + 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) mma(y[i], x.h, mm[2 * i], mm[2 * i + 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) mma(z[i], x.m, mm[2 * i], mm[2 * i + 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) mma(y[i], x.h, mh[2 * i], mh[2 * i + 1]);
 #pragma unroll
         for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -424,7 +427,7 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         ldsm4(mm, a + CK * CK * 2);
         ldsm4(ml, a + 2 * CK * CK * 2);
     };
-    if (warp == TC_WORKERS) {
+    if (warp >= TC_WORKERS) {
         // ---- the outputs: O = P Q S + A U, a chunk behind
         Split3 us;
         uint32_t ah[4], am[4], al[4];
@@ -457,7 +460,10 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         __syncthreads();
         for (int c = 0; c < chunks; ++c) {
             __syncthreads();
-            if (c > 0) finish(c - 1);
+            if ((c & 1) != warp - TC_WORKERS) {               // the other reader forms U of this chunk
+                if (c > 0) finish(c - 1);
+                continue;
+            }
             Split3 x;
             form_x(c, x);
             uint32_t th[4], tm[4], tl[4];
@@ -475,7 +481,7 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
             for (int i = 0; i < 2; ++i) pq[i] = *reinterpret_cast<const float2*>(f + CK + i * 8 + t4 * 2);
         }
         __syncthreads();
-        finish(chunks - 1);
+        if (((chunks - 1) & 1) == warp - TC_WORKERS) finish(chunks - 1);
         return;
     }
     // ---- a worker: key channels d0 .. d0 + 16 KS of S^T
@@ -494,8 +500,10 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         const unsigned st = base + (c % TC_STAGES) * St::BYTES;
         const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
         Split3 s[KS];
-        float m[2][4];
-        auto product = [&](unsigned rows) {                   // m = S^T times the chunk's rows, over this warp's channels
+        // S^T times the chunk's rows, over this warp's channels; one accumulator per part, so that no product waits for
+        // the one before it
+        auto product = [&](unsigned rows, float (&m)[2][4]) {
+            float lo[2][4] = {}, mid[2][4] = {};
 #pragma unroll
             for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -504,33 +512,39 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
             for (int ks = 0; ks < KS; ++ks) {
                 uint32_t r[4];
                 ldsm4(r, rows + ((mi >> 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi & 1) * 8) * 2);
-                mma(m[0], s[ks].l, r[0], r[1]);
-                mma(m[1], s[ks].l, r[2], r[3]);
-                mma(m[0], s[ks].m, r[0], r[1]);
-                mma(m[1], s[ks].m, r[2], r[3]);
+                mma(lo[0], s[ks].l, r[0], r[1]);
+                mma(lo[1], s[ks].l, r[2], r[3]);
+                mma(mid[0], s[ks].m, r[0], r[1]);
+                mma(mid[1], s[ks].m, r[2], r[3]);
                 mma(m[0], s[ks].h, r[0], r[1]);
                 mma(m[1], s[ks].h, r[2], r[3]);
             }
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) m[i][e] += mid[i][e] + lo[i][e];
         };
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) split_tiles(S[2 * ks], S[2 * ks + 1], s[ks]);
-        product(st + St::K);
-#pragma unroll
-        for (int i = 0; i < 2; ++i) *red_at(c & 1, 0, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
-        __syncthreads();
-        Split3 x;
-        form_x(c, x);
         uint32_t th[4], tm[4], tl[4];
         load_matrix(c, TC_T, th, tm, tl);
+        {
+            float m[2][4];
+            product(st + St::K, m);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) *red_at(c & 1, 0, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
+        }
+        __syncthreads();
+        float qs[2][4];
+        product(st + St::Q, qs);                              // the tensor cores work on this while X is formed
+        Split3 x;
+        form_x(c, x);
         float u[2][4];
 #pragma unroll
         for (int i = 0; i < 2; ++i)
 #pragma unroll
             for (int e = 0; e < 4; ++e) u[i][e] = 0.f;
         times(x, th, tm, tl, u);
-        product(st + St::Q);
-#pragma unroll
-        for (int i = 0; i < 2; ++i) *red_at(c & 1, 1, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
         const float pc = f[3 * CK];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -543,18 +557,21 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         Split3 y;
         split_tiles(u[0], u[1], y);
 #pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
-            uint32_t r[4];
-            ldsm4t(r, st + St::K + ((mi & 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi >> 1) * 8) * 2);
+        for (int i = 0; i < 2 * KS; ++i)
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
+            for (int e = 0; e < 4; ++e) S[i][e] *= pc;
+        uint32_t r[KS][4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) S[2 * ks + i][e] *= pc;
-                mma(S[2 * ks + i], y.l, r[2 * i], r[2 * i + 1]);
-                mma(S[2 * ks + i], y.m, r[2 * i], r[2 * i + 1]);
-                mma(S[2 * ks + i], y.h, r[2 * i], r[2 * i + 1]);
-            }
-        }
+        for (int ks = 0; ks < KS; ++ks)
+            ldsm4t(r[ks], st + St::K + ((mi & 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi >> 1) * 8) * 2);
+#pragma unroll
+        for (int i = 0; i < 2 * KS; ++i) mma(S[i], y.l, r[i >> 1][2 * (i & 1)], r[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+        for (int i = 0; i < 2 * KS; ++i) mma(S[i], y.m, r[i >> 1][2 * (i & 1)], r[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+        for (int i = 0; i < 2 * KS; ++i) mma(S[i], y.h, r[i >> 1][2 * (i & 1)], r[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) *red_at(c & 1, 1, warp, i) = make_float4(qs[i][0], qs[i][1], qs[i][2], qs[i][3]);
     }
     __syncthreads();
 #pragma unroll
