@@ -8,8 +8,8 @@
 // recurrence is not rounded) and for values that every head forms from one latent.
 //
 // Kernels: bfloat16 with inner sizes and pitches in whole 16-byte pieces on the tensor cores (mma.sync m16n8k16, tiles of
-// 128 x 128, 64 x 64 or 16 x 64, a cp.async ring of two or three stages of 64 inner elements, 16-byte chunks XOR-ed with
-// the row number); everything else on a plain FMA kernel, 32 x 32 tiles.
+// 128 x 128, 64 x 64, 16 x 64 or 16 x 32, a cp.async ring of three to eight stages of 64 inner elements, 16-byte chunks XOR-ed
+// with the row number); everything else on a plain FMA kernel, 32 x 32 tiles.
 #include "common.cuh"
 
 using namespace qnn;
@@ -230,6 +230,9 @@ QNN_API int qnn_block_linear(const void* x, int x_dt, long long ldx, long long x
                         (((uintptr_t)x | (uintptr_t)w) & 15) == 0 && ((uintptr_t)out & 7) == 0;
     if (tensor) {
         if (T <= 32) return launch_mma<16, 64, 1, 4, 3>(a, blocks, st);
+        // a few outputs of a long inner size: blocks of 16 rows fill the device, with eight stages on their way
+        if (blocks == 1 && N <= 32) return launch_mma<16, 32, 1, 2, 8>(a, blocks, st);
+        if (blocks == 1 && N <= 64) return launch_mma<16, 64, 1, 4, 8>(a, blocks, st);
         const long long big = (long long)((T + 127) / 128) * ((N + 127) / 128) * blocks;
         if (N > 64 && big >= 448) return launch_mma<128, 128, 2, 4, 3>(a, blocks, st);
         return launch_mma<64, 64, 2, 2, 3>(a, blocks, st);

@@ -1013,6 +1013,35 @@ delta_step_kernel(const StepArgs a, int splits) {
     const bool live = slot >= 0;
     float* base = a.state + (size_t)(live ? slot : 0) * a.slot_stride;
     float* S0 = base + a.s_off + (size_t)h * D * VD + c0;
+    // Channels of the convolution that this CTA needs: q of its head, k of its head, its value columns, two or three per thread
+    // (dim <= 256).  The last three past inputs and their filter columns are asked for together, older ones one by one.
+    const int nch = 2 * D + ncol;
+    constexpr int PER = (2 * MAX_DIM + CG * V + STEP_THREADS - 1) / STEP_THREADS, NEAR = 3;
+    float past[PER], last[PER], near_x[PER][NEAR], near_w[PER][NEAR];
+    int chan[PER];
+    const int newest = pos % a.taps;                          // the ring's row of this token
+#pragma unroll
+    for (int e = 0; e < PER; ++e) {
+        const int i = tid + e * STEP_THREADS;
+        last[e] = 0.f;
+        chan[e] = -1;
+#pragma unroll
+        for (int j = 0; j < NEAR; ++j) near_x[e][j] = near_w[e][j] = 0.f;
+        if (i < nch) {
+            const int ch = i < D ? g * D + i : (i < 2 * D ? a.G * D + g * D + (i - D) : 2 * a.G * D + h * VD + c0 + (i - 2 * D));
+            const size_t f = (size_t)ch * a.taps + a.taps - 1;
+            chan[e] = ch;
+            last[e] = load_as_f(a.conv, a.c_dt, f);
+#pragma unroll
+            for (int j = 0; j < NEAR; ++j) {                  // j + 1 tokens ago
+                const int r = newest - 1 - j;
+                if (live && j + 1 < a.taps && pos - 1 - j >= 0) {
+                    near_w[e][j] = load_as_f(a.conv, a.c_dt, f - 1 - j);
+                    near_x[e][j] = base[(size_t)(r < 0 ? r + a.taps : r) * C + ch];
+                }
+            }
+        }
+    }
     // the state: rows rg, rg + RG, ..; columns cg * V ..
     float S[RPT][V];
 #pragma unroll
@@ -1029,40 +1058,51 @@ delta_step_kernel(const StepArgs a, int splits) {
             }
         }
     }
-    // channels of the convolution that this CTA needs: q of its head, k of its head, its value columns.  Two or three per thread
-    // at most (dim <= 256); a channel's past inputs and its filter are summed up to the newest tap here.
-    const int nch = 2 * D + ncol;
-    constexpr int PER = (2 * MAX_DIM + CG * V + STEP_THREADS - 1) / STEP_THREADS;
-    float past[PER], last[PER];
-    int chan[PER];
+    const float rate = a.rate[h], bias = a.bias[h];
+    const float wn = tid < ncol ? load_as_f(a.norm, a.n_dt, c0 + tid) : 0.f;
+    // the gates' weights: the first two pieces of eight per thread stay as they come until the input is there
+    const size_t wb = (size_t)h * a.W, wa = (size_t)(a.H + h) * a.W;
+    const bool early = sizeof(T) == 2 && a.w_dt == QNN_DT_BF16 && a.W % 8 == 0;
+    constexpr int EARLY = 2;
+    Vec16<bf16> eb[EARLY], ea[EARLY];
 #pragma unroll
-    for (int e = 0; e < PER; ++e) {
-        const int i = tid + e * STEP_THREADS;
-        past[e] = last[e] = 0.f;
-        chan[e] = -1;
-        if (i < nch) {
-            const int ch = i < D ? g * D + i : (i < 2 * D ? a.G * D + g * D + (i - D) : 2 * a.G * D + h * VD + c0 + (i - 2 * D));
-            chan[e] = ch;
-            last[e] = load_as_f(a.conv, a.c_dt, (size_t)ch * a.taps + a.taps - 1);
-            if (live)
-                for (int j = 0; j + 1 < a.taps; ++j) {
-                    const int at = pos - a.taps + 1 + j;
-                    if (at >= 0) past[e] = fmaf(load_as_f(a.conv, a.c_dt, (size_t)ch * a.taps + j), base[(size_t)(at % a.taps) * C + ch], past[e]);
-                }
+    for (int u = 0; u < EARLY; ++u) {
+        const int i = (tid + u * STEP_THREADS) * 8;
+        eb[u].zero();
+        ea[u].zero();
+        if (early && i < a.W) {
+            eb[u].load((const bf16*)a.w_ba + wb + i);
+            ea[u].load((const bf16*)a.w_ba + wa + i);
         }
     }
-    const float rate = a.rate[h], bias = a.bias[h];
     pdl_wait();
     const T* prow = (const T*)a.p + (size_t)b * a.ldp;
     const T* xrow = (const T*)a.x + (size_t)b * a.W;
     float raw[PER];
 #pragma unroll
     for (int e = 0; e < PER; ++e) raw[e] = chan[e] >= 0 ? to_f(prow[chan[e]]) : 0.f;
+    const float z = tid < ncol ? to_f(prow[C + h * VD + c0 + tid]) : 0.f;
     // the gates' products
     float db = 0.f, da = 0.f;
-    const size_t wb = (size_t)h * a.W, wa = (size_t)(a.H + h) * a.W;
+    if (early) {
+#pragma unroll
+        for (int u = 0; u < EARLY; ++u) {
+            const int i = (tid + u * STEP_THREADS) * 8;
+            if (i < a.W) {
+                float xf[8], f[8], e8[8];
+                load8_as_f(xrow, QNN_DT_BF16, i, xf);
+                eb[u].unpack(f);
+                ea[u].unpack(e8);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    db += xf[j] * f[j];
+                    da += xf[j] * e8[j];
+                }
+            }
+        }
+    }
     if (a.W % 8 == 0) {
-        for (int i = tid * 8; i < a.W; i += STEP_THREADS * 8) {
+        for (int i = (tid + (early ? EARLY * STEP_THREADS : 0)) * 8; i < a.W; i += STEP_THREADS * 8) {
             float xf[8], f[8], e8[8];
             load8_as_f(xrow, sizeof(T) == 2 ? QNN_DT_BF16 : QNN_DT_F32, i, xf);
             load8_as_f(a.w_ba, a.w_dt, wb + i, f);
@@ -1080,6 +1120,19 @@ delta_step_kernel(const StepArgs a, int splits) {
             da += xf * load_as_f(a.w_ba, a.w_dt, wa + i);
         }
     }
+    // the past inputs' part of the convolution, oldest first
+#pragma unroll
+    for (int e = 0; e < PER; ++e) {
+        past[e] = 0.f;
+        if (chan[e] >= 0 && live)
+            for (int j = min(a.taps - 1, pos); j > NEAR; --j) {
+                const int r = newest - j;
+                past[e] = fmaf(load_as_f(a.conv, a.c_dt, (size_t)chan[e] * a.taps + a.taps - 1 - j),
+                               base[(size_t)(r < 0 ? r + a.taps : r) * C + chan[e]], past[e]);
+            }
+#pragma unroll
+        for (int j = NEAR - 1; j >= 0; --j) past[e] = fmaf(near_w[e][j], near_x[e][j], past[e]);
+    }
     // convolution, silu (rounded as a prompt's rows are stored), the ring's newest row
     float ssq = 0.f, ssk = 0.f;
 #pragma unroll
@@ -1092,7 +1145,7 @@ delta_step_kernel(const StepArgs a, int splits) {
             else sv[i - 2 * D] = y;
             // q and k belong to all heads of the group and all CTAs of a cluster: one of them keeps them
             const bool keeper = i >= 2 * D || (split == 0 && h % (a.H / a.G) == 0);
-            if (live && keeper) base[(size_t)(pos % a.taps) * C + chan[e]] = raw[e];
+            if (live && keeper) base[(size_t)newest * C + chan[e]] = raw[e];
         }
     }
     {
@@ -1181,8 +1234,7 @@ delta_step_kernel(const StepArgs a, int splits) {
         for (int r = 0; r < splits; ++r) total += squares[r];
     }
     if (tid < ncol) {
-        const float y = o * rsqrtf(total / (float)VD + a.eps) * load_as_f(a.norm, a.n_dt, c0 + tid);
-        const float z = to_f(prow[C + h * VD + c0 + tid]);
+        const float y = o * rsqrtf(total / (float)VD + a.eps) * wn;
         ((T*)a.out)[(size_t)b * a.ldo + (size_t)h * VD + c0 + tid] = from_f<T>(live ? y * silu(z) : 0.f);
     }
 }
@@ -1296,8 +1348,8 @@ QNN_API int qnn_delta_scan(const void* q, const void* k, const void* v, long lon
     else if (rpt <= 8) { QNN_DS_COLS(T, 8, VV) }  \
     else if (rpt <= 16) { QNN_DS_COLS(T, 16, VV) } \
     else { QNN_DS_COLS(T, 32, VV) }
-    if (dtype == QNN_DT_BF16) {
-        if (vec) { QNN_DS_ROWS(bf16, true) } else { QNN_DS_ROWS(bf16, false) }
+    if (dtype == QNN_DT_BF16) {                               // (aligned bfloat16 rows have the tensor-core kernel)
+        QNN_DS_ROWS(bf16, false)
     } else {
         if (vec) { QNN_DS_ROWS(float, true) } else { QNN_DS_ROWS(float, false) }
     }

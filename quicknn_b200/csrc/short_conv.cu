@@ -58,6 +58,10 @@ __device__ __forceinline__ void store_v(T* p, const float* v) {
     }
 }
 
+// silu of a result that is stored as T: the fast functions where it is rounded to bfloat16
+template <typename T> __device__ __forceinline__ float silu_as(float v) { return silu(v); }
+template <> __device__ __forceinline__ float silu_as<bf16>(float v) { return activate_fast(v, QNN_ACT_SILU); }
+
 // TAPS > 0: the number of taps and of rows per tile (ROWS) is known here, and the filter and the tile's inputs stay in
 // registers; 0: any numbers, inputs are read again for every tap.
 template <typename T, int VEC, int TAPS, int ROWS>
@@ -162,7 +166,7 @@ causal_conv_kernel(const T* __restrict__ x, long long ldx, const void* __restric
                 for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], v[i + j][e], acc[e]);
                 acc[e] += ob[e];
                 if (add_input) acc[e] += v[i + TAPS - 1][e];
-                if (act) acc[e] = silu(acc[e]);
+                if (act) acc[e] = silu_as<T>(acc[e]);
             }
             if (!idle) store_v<T, VEC>(out + (size_t)(row0 + r0 + i) * ldo + c0, acc);
             if (inv != nullptr) {                           // (a warp's rows are one tile's: all its lanes are here)
@@ -190,7 +194,7 @@ causal_conv_kernel(const T* __restrict__ x, long long ldx, const void* __restric
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
                 acc[e] += ob[e] + (add_input ? v[e] : 0.f);
-                if (act) acc[e] = silu(acc[e]);
+                if (act) acc[e] = silu_as<T>(acc[e]);
             }
             store_v<T, VEC>(out + (size_t)(row0 + r) * ldo + c0, acc);
         }

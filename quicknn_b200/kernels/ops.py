@@ -1843,7 +1843,7 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, seq_
 
 DELTA_CHUNK = 16             # rows of a chunk of the delta rule's scan
 DELTA_RECORD, DELTA_RECORD_TC = 4 * (2 * DELTA_CHUNK * DELTA_CHUNK + 2 * DELTA_CHUNK), 3280      # bytes per chunk and value head
-DELTA_TENSOR_CORES = True    # bfloat16 rows: the scan on the tensor cores (tests switch it off to compare)
+DELTA_TENSOR_CORES = True    # bfloat16 rows: the scan on the tensor cores (False: on the FMA pipes, for comparisons)
 
 
 def delta_scan(rows: torch.Tensor, inv: torch.Tensor, pre: torch.Tensor, rate: torch.Tensor, bias: torch.Tensor, q_scale: float,
