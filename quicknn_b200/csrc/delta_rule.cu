@@ -177,8 +177,8 @@ __device__ __forceinline__ void cp16(unsigned dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src) : "memory");
 }
 
-// What a chunk leaves for the scan, per value head: T and A in three bfloat16 matrices each ([3][16][16]: row t, column j),
-// then per row P_t / |k_t|, P_t q_scale / |q_t|, D_16,t / |k_t|, and P_16: 3280 bytes.
+// What a chunk leaves for the scan, per value head: T and A in three bfloat16 matrices each ([3][2][16][8]: row t of the columns
+// j = 8 c .. 8 c + 7, c = 0, 1, so that the eight rows of an ldmatrix lie side by side), then per row P_t / |k_t|, P_t q_scale / |q_t|, D_16,t / |k_t|, and P_16: 3280 bytes.
 constexpr int TC_T = 0, TC_A = 3 * CK * CK * 2, TC_F = 2 * TC_A, TC_RECORD = TC_F + (3 * CK + 4) * 4;
 
 // a warp per (chunk, query/key head)
@@ -263,9 +263,10 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
             const bf16 hi = __float2bfloat16_rn(v);
             const float r = v - __bfloat162float(hi);
             const bf16 mid = __float2bfloat16_rn(r);
-            m[t * CK + j] = hi;
-            m[CK * CK + t * CK + j] = mid;
-            m[2 * CK * CK + t * CK + j] = __float2bfloat16_rn(r - __bfloat162float(mid));
+            const int at = (j >> 3) * (CK * 8) + t * 8 + (j & 7);
+            m[at] = hi;
+            m[CK * CK + at] = mid;
+            m[2 * CK * CK + at] = __float2bfloat16_rn(r - __bfloat162float(mid));
         };
         float d = 1.f, p = 1.f, mine_p = 1.f;
 #pragma unroll
@@ -422,7 +423,7 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
             for (int e = 0; e < 4; ++e) y[i][e] += z[i][e];
     };
     auto load_matrix = [&](int c, int at, uint32_t (&mh)[4], uint32_t (&mm)[4], uint32_t (&ml)[4]) {
-        const unsigned a = base + (c % TC_STAGES) * St::BYTES + St::R + at + ((mi >> 1) * 8 + mr) * (CK * 2) + (mi & 1) * 16;
+        const unsigned a = base + (c % TC_STAGES) * St::BYTES + St::R + at + (mi & 1) * (CK * 16) + ((mi >> 1) * 8 + mr) * 16;
         ldsm4(mh, a);
         ldsm4(mm, a + CK * CK * 2);
         ldsm4(ml, a + 2 * CK * CK * 2);
