@@ -11,7 +11,7 @@
 //   qnn_delta_chunks   per chunk of 16 rows and value head: what does not depend on the state
 //   qnn_delta_scan     walks the chunks of every sequence in order, from the slot's state and back into it; bfloat16 rows on the
 //                      tensor cores with every float32 matrix in three bfloat16 parts, others on the FMA pipes
-//   qnn_delta_step     one token per sequence, everything between the input product and the output product in one kernel
+// (One token per sequence: delta_step.cu.)
 //
 // Chunks (Yang et al., "Parallelizing Linear Transformers with the Delta Rule over Sequence Length").  With S the state before a
 // chunk, P_t the product of g_1 .. g_t and D_ti the product of g_(i+1) .. g_t,
@@ -23,7 +23,7 @@
 // qnn_delta_chunks forms T = (I + L)^-1 diag(beta), A, P and D_16,. by products of decays, never by their logarithms' differences.
 // Every decay product is at most 1.  The scan is then three small matrix products per chunk instead of 16 steps that wait for
 // one another.  The order of the sums depends on the sizes only; where a sequence's chunks start moves results by rounding.
-#include "common.cuh"
+#include "delta_rule.cuh"
 
 using namespace qnn;
 
@@ -31,11 +31,6 @@ namespace {
 
 constexpr int CK = 16;                       // rows of a chunk
 constexpr int RECORD = 2 * CK * CK + 2 * CK; // floats that qnn_delta_chunks leaves per (chunk, value head): T, A, P, D
-constexpr int MAX_DIM = 256;
-
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ float beta_of(float b) { return 1.f / (1.f + expf(-b)); }
-__device__ __forceinline__ float decay_of(float a, float rate, float bias) { return expf(-rate * softplus(a + bias)); }
 
 // chunk c of sequence b is record slot (row0 / 16 + b + c): the slots of different sequences never meet, and T / 16 + B of
 // them hold a step's chunks whatever its sequences' lengths
@@ -135,7 +130,7 @@ delta_chunks_kernel(const T* __restrict__ q, const T* __restrict__ k, long long 
 
 // ---- bfloat16 rows: the same on the tensor cores ---------------------------------------------------------------------
 // Keys and queries are bfloat16 numbers times a float32 factor per row, so a float32 matrix meets them on the tensor cores
-// without loss when it is cut into three bfloat16 numbers per element (hi + mid + lo holds 24 bits) and the factors are applied
+// without loss when it is cut into three bfloat16 numbers per element (8 bits of its 24 each) and the factors are applied
 // to the results: x = hi + mid + lo costs three products with one exact factor and six with another float32 matrix (the three
 // smallest of nine terms lie below float32's rounding).  Accumulation is float32.
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], unsigned addr) {
@@ -152,19 +147,25 @@ __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint3
         : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
         : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ uint32_t pack2(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&h);
+// d = a b without an accumulator to start from
+__device__ __forceinline__ void mma_first(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%10,%10,%10,%10};\n"
+        : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
 }
 __device__ __forceinline__ float low_of(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float high_of(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
 struct Split3 { uint32_t h[4], m[4], l[4]; };
+// The upper half of a float32 is a bfloat16 with its first 8 significant bits; what is left has 16, and once more 8: the three
+// parts add up to the number exactly (but for what lies below float32's smallest normal numbers).
+__device__ __forceinline__ float upper(float x) { return __uint_as_float(__float_as_uint(x) & 0xffff0000u); }
+__device__ __forceinline__ uint32_t uppers(float a, float b) { return __byte_perm(__float_as_uint(a), __float_as_uint(b), 0x7632); }
 __device__ __forceinline__ void split(float a, float b, uint32_t& h, uint32_t& m, uint32_t& l) {
-    h = pack2(a, b);
-    a -= low_of(h);
-    b -= high_of(h);
-    m = pack2(a, b);
-    l = pack2(a - low_of(m), b - high_of(m));
+    h = uppers(a, b);
+    a -= upper(a);
+    b -= upper(b);
+    m = uppers(a, b);
+    l = uppers(a - upper(a), b - upper(b));
 }
 // two accumulator tiles (16 x 8 each, side by side) as the A operand of a product over those 16 columns
 __device__ __forceinline__ void split_tiles(const float (&x)[4], const float (&y)[4], Split3& s) {
@@ -201,16 +202,17 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
     if (t0 >= n) return;                                      // (nothing below waits for another warp)
     const int nt = min(CK, n - t0);
     const int pieces = dpad / 8;
+    const unsigned kb = (unsigned)__cvta_generic_to_shared(mine), qb = kb + CK * pitch;
     for (int i = lane; i < CK * pieces; i += 32) {
         const int t = i / pieces, d = (i - t * pieces) * 8;
-        uint4 kv = make_uint4(0, 0, 0, 0), qv = kv;
         if (t < nt && d < dim) {
             const size_t at = (size_t)(row0 + t0 + t) * ld + (size_t)g * dim + d;
-            kv = *reinterpret_cast<const uint4*>(k + at);
-            qv = *reinterpret_cast<const uint4*>(q + at);
+            cp16(kb + t * pitch + d * 2, k + at);
+            cp16(qb + t * pitch + d * 2, q + at);
+        } else {
+            *reinterpret_cast<uint4*>(mine + t * pitch + d * 2) = make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(mine + (CK + t) * pitch + d * 2) = make_uint4(0, 0, 0, 0);
         }
-        *reinterpret_cast<uint4*>(mine + t * pitch + d * 2) = kv;
-        *reinterpret_cast<uint4*>(mine + (CK + t) * pitch + d * 2) = qv;
     }
     float iq = 0.f, ik = 0.f;                                 // of row j
     if (j < nt) {
@@ -218,8 +220,15 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
         iq = inv[row * ldi + g] * q_scale;
         ik = inv[row * ldi + G + g];
     }
+    const int per = H / G;
+    float zb = 0.f, za = 0.f;                                 // the first value head's logits, asked for with the rows
+    if (j < nt) {
+        const float* pr = pre + (size_t)(row0 + t0 + j) * ldp;
+        zb = pr[g * per];
+        za = pr[H + g * per];
+    }
+    asm volatile("cp.async.wait_all;\n" ::: "memory");
     __syncwarp();
-    const unsigned kb = (unsigned)__cvta_generic_to_shared(mine), qb = kb + CK * pitch;
     const int mi = lane >> 3, mr = lane & 7;                  // matrix and row that this lane addresses for ldmatrix
     float akk[2][4], aqk[2][4];
 #pragma unroll
@@ -246,7 +255,6 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
             qk[t * (CK + 1) + col] = aqk[i][e] * (qt * kj);
         }
     __syncwarp();
-    const int per = H / G;
     for (int s = 0; s < per; ++s) {
         const int h = g * per + s;
         unsigned char* out = rec + (record_of(row0, b, c) * H + h) * TC_RECORD;
@@ -255,18 +263,20 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
         float* oF = reinterpret_cast<float*>(out + TC_F);
         float be = 0.f, ga = 1.f;
         if (j < nt) {
-            const float* pr = pre + (size_t)(row0 + t0 + j) * ldp;
-            be = beta_of(pr[h]);
-            ga = decay_of(pr[H + h], rate[h], bias[h]);
+            be = beta_of(zb);
+            ga = decay_of(za, rate[h], bias[h]);
+            if (s + 1 < per) {
+                const float* pr = pre + (size_t)(row0 + t0 + j) * ldp;
+                zb = pr[h + 1];
+                za = pr[H + h + 1];
+            }
         }
         auto put = [&](bf16* m, int t, float v) {
-            const bf16 hi = __float2bfloat16_rn(v);
-            const float r = v - __bfloat162float(hi);
-            const bf16 mid = __float2bfloat16_rn(r);
+            const float r = v - upper(v), s = r - upper(r);
             const int at = (j >> 3) * (CK * 8) + t * 8 + (j & 7);
-            m[at] = hi;
-            m[CK * CK + at] = mid;
-            m[2 * CK * CK + at] = __float2bfloat16_rn(r - __bfloat162float(mid));
+            m[at] = __ushort_as_bfloat16((unsigned short)(__float_as_uint(v) >> 16));
+            m[CK * CK + at] = __ushort_as_bfloat16((unsigned short)(__float_as_uint(r) >> 16));
+            m[2 * CK * CK + at] = __ushort_as_bfloat16((unsigned short)(__float_as_uint(s) >> 16));
         };
         float d = 1.f, p = 1.f, mine_p = 1.f;
 #pragma unroll
@@ -304,8 +314,11 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
 // of the key channels each (KS times 16) as accumulator tiles, which serve as the A operand of the products with keys and queries
 // when they are split; their partial K S meet in shared memory (one barrier per chunk), and each of the four then forms X, U = T X
 // and its quarter of the update by itself, all in registers.  Q S is formed in the shadow of that; two more warps take alternate
-// chunks and turn it into the outputs a chunk later; the last warp fetches chunks ahead.
-constexpr int TC_WORKERS = 4, TC_READERS = 2, TC_THREADS = 32 * (TC_WORKERS + TC_READERS + 1), TC_STAGES = 6, TC_AHEAD = TC_STAGES - 2;
+// chunks and turn it into the outputs a chunk later; the last two fetch chunks ahead, keys and values the one, queries and what
+// qnn_delta_chunks left the other.
+constexpr int TC_WORKERS = 4, TC_READERS = 2, TC_LOADERS = 2, TC_THREADS = 32 * (TC_WORKERS + TC_READERS + TC_LOADERS), TC_STAGES = 6, TC_AHEAD = TC_STAGES - 2;
+
+template <bool V> struct Flag { static constexpr bool value = V; };
 
 template <int KS>
 struct TcStage {
@@ -317,7 +330,7 @@ struct TcStage {
 };
 
 template <int KS>
-__global__ void __launch_bounds__(TC_THREADS)
+__global__ void __launch_bounds__(TC_THREADS, KS <= 2 ? 2 : 1)
 delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, const bf16* __restrict__ v, long long ld,
                      const unsigned char* __restrict__ rec, const int* __restrict__ seq_row0, const int* __restrict__ seq_len,
                      const int* __restrict__ slots, float* __restrict__ state, long long slot_stride, float* __restrict__ out,
@@ -341,9 +354,12 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
     float4* red = reinterpret_cast<float4*>(smem + St::RED);
     auto red_at = [&](int parity, int which, int w, int tile) { return red + (((parity * 2 + which) * TC_WORKERS + w) * 2 + tile) * 32 + lane; };
     __syncthreads();                                          // the stages are zero: rows and columns that nothing fills stay so
-    if (warp == TC_WORKERS + TC_READERS) {
-        // ---- the loader.  Rows beyond the sequence keep what an earlier chunk left (or zeros): finite numbers whose factors are 0
+    if (warp >= TC_WORKERS + TC_READERS) {
+        // ---- a loader.  Rows beyond the sequence keep what an earlier chunk left (or zeros): finite numbers whose factors are 0
         const int pieces = dim / 8, vp = min(2, (vdim - c0) / 8);
+        const bool first_half = warp == TC_WORKERS + TC_READERS;
+        const bf16* rows = first_half ? k : q;
+        const int into = first_half ? St::K : St::Q;
         const int at_once = 32 / pieces, tl = lane / pieces, dl = lane - tl * pieces;        // rows side by side; this lane's
         auto load = [&](int c) {
             if (c < chunks) {
@@ -352,19 +368,17 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
                 const size_t first = (size_t)(row0 + c * CK);
                 if (tl < at_once) {
                     size_t at = (first + tl) * ld + (size_t)g * dim + dl * 8;
-                    unsigned to = st + tl * St::PITCH + dl * 16;
-                    for (int t = tl; t < nt; t += at_once, at += at_once * ld, to += at_once * St::PITCH) {
-                        cp16(to + St::K, k + at);
-                        cp16(to + St::Q, q + at);
-                    }
+                    unsigned to = st + into + tl * St::PITCH + dl * 16;
+                    for (int t = tl; t < nt; t += at_once, at += at_once * ld, to += at_once * St::PITCH) cp16(to, rows + at);
                 }
-                {
+                if (first_half) {
                     const int t = lane >> 1, p = lane & 1;
                     if (t < nt && p < vp)
                         cp16(st + St::V + t * St::VPITCH + p * 16, v + (first + t) * ld + (size_t)h * vdim + c0 + p * 8);
+                } else {
+                    const unsigned char* r = rec + (record_of(row0, b, c) * H + h) * TC_RECORD;
+                    for (int i = lane; i < TC_RECORD / 16; i += 32) cp16(st + St::R + i * 16, r + i * 16);
                 }
-                const unsigned char* r = rec + (record_of(row0, b, c) * H + h) * TC_RECORD;
-                for (int i = lane; i < TC_RECORD / 16; i += 32) cp16(st + St::R + i * 16, r + i * 16);
             }
             asm volatile("cp.async.commit_group;\n" ::: "memory");
         };
@@ -379,36 +393,47 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         __syncthreads();
         return;
     }
-    // X^T = V^T - (P K S)^T of chunk c from the workers' partial sums, split for a product over the chunk's rows
-    auto form_x = [&](int c, Split3& x) {
+    // X^T = V^T - (P K S)^T of chunk c from the workers' partial sums, split for a product over the chunk's rows: first the
+    // loads, then the rest, so that other work finds its place in between
+    struct Parts { float4 m[2][TC_WORKERS]; float2 pk[2]; uint32_t v[4]; };
+    auto fetch_x = [&](int c, Parts& p) {
         const unsigned st = base + (c % TC_STAGES) * St::BYTES;
         const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
-        uint32_t vr[4];
-        ldsm4t(vr, st + St::V + ((mi >> 1) * 8 + mr) * St::VPITCH + (mi & 1) * 16);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int w = 0; w < TC_WORKERS; ++w) p.m[i][w] = *red_at(c & 1, 0, w, i);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) p.pk[i] = *reinterpret_cast<const float2*>(f + i * 8 + t4 * 2);
+        ldsm4t(p.v, st + St::V + ((mi >> 1) * 8 + mr) * St::VPITCH + (mi & 1) * 16);
+    };
+    auto form_x = [&](const Parts& p, Split3& x) {
         float xs[2][4];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            float4 m = *red_at(c & 1, 0, 0, i);
+            float4 m = p.m[i][0];
 #pragma unroll
             for (int w = 1; w < TC_WORKERS; ++w) {
-                const float4 o = *red_at(c & 1, 0, w, i);
-                m.x += o.x; m.y += o.y; m.z += o.z; m.w += o.w;
+                m.x += p.m[i][w].x; m.y += p.m[i][w].y; m.z += p.m[i][w].z; m.w += p.m[i][w].w;
             }
-            const float2 pk = *reinterpret_cast<const float2*>(f + i * 8 + t4 * 2);
-            xs[i][0] = low_of(vr[2 * i]) - pk.x * m.x;
-            xs[i][1] = high_of(vr[2 * i]) - pk.y * m.y;
-            xs[i][2] = low_of(vr[2 * i + 1]) - pk.x * m.z;
-            xs[i][3] = high_of(vr[2 * i + 1]) - pk.y * m.w;
+            xs[i][0] = low_of(p.v[2 * i]) - p.pk[i].x * m.x;
+            xs[i][1] = high_of(p.v[2 * i]) - p.pk[i].y * m.y;
+            xs[i][2] = low_of(p.v[2 * i + 1]) - p.pk[i].x * m.z;
+            xs[i][3] = high_of(p.v[2 * i + 1]) - p.pk[i].y * m.w;
         }
         split_tiles(xs[0], xs[1], x);
     };
     // y += (x times the 16 x 16 matrix whose three parts are at `m`)^T, the small terms first
-    auto times = [&](const Split3& x, const uint32_t (&mh)[4], const uint32_t (&mm)[4], const uint32_t (&ml)[4], float (&y)[2][4]) {
-        float z[2][4] = {};
+    auto times = [&](const Split3& x, const uint32_t (&mh)[4], const uint32_t (&mm)[4], const uint32_t (&ml)[4], float (&y)[2][4],
+                     auto fresh) {                            // fresh: y starts from zero
+        float z[2][4];
 #pragma unroll
-        for (int i = 0; i < 2; ++i) mma(z[i], x.l, mh[2 * i], mh[2 * i + 1]);
+        for (int i = 0; i < 2; ++i) mma_first(z[i], x.l, mh[2 * i], mh[2 * i + 1]);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) mma(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
+        for (int i = 0; i < 2; ++i) {
+            if constexpr (decltype(fresh)::value) mma_first(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
+            else mma(y[i], x.m, mh[2 * i], mh[2 * i + 1]);
+        }
 #pragma unroll
         for (int i = 0; i < 2; ++i) mma(z[i], x.h, ml[2 * i], ml[2 * i + 1]);
 #pragma unroll
@@ -448,7 +473,7 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
                 o[i][2] = pq[i].x * m.z;
                 o[i][3] = pq[i].y * m.w;
             }
-            times(us, ah, am, al, o);
+            times(us, ah, am, al, o, Flag<false>());
             const int nt = min(CK, n - c * CK);
 #pragma unroll
             for (int i = 0; i < 2; ++i)
@@ -466,15 +491,15 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
                 continue;
             }
             Split3 x;
-            form_x(c, x);
+            {
+                Parts p;
+                fetch_x(c, p);
+                form_x(p, x);
+            }
             uint32_t th[4], tm[4], tl[4];
             load_matrix(c, TC_T, th, tm, tl);
             float u[2][4];
-#pragma unroll
-            for (int i = 0; i < 2; ++i)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) u[i][e] = 0.f;
-            times(x, th, tm, tl, u);
+            times(x, th, tm, tl, u, Flag<true>());
             split_tiles(u[0], u[1], us);
             load_matrix(c, TC_A, ah, am, al);                 // (the stage may be filled anew before the outputs are formed)
             const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
@@ -501,29 +526,32 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
         const unsigned st = base + (c % TC_STAGES) * St::BYTES;
         const float* f = reinterpret_cast<const float*>(smem + (c % TC_STAGES) * St::BYTES + St::R + TC_F);
         Split3 s[KS];
-        // S^T times the chunk's rows, over this warp's channels; one accumulator per part, so that no product waits for
-        // the one before it
+        // S^T times the chunk's rows, over this warp's channels; the small parts have an accumulator of their own, which also
+        // keeps products from waiting for one another
         auto product = [&](unsigned rows, float (&m)[2][4]) {
-            float lo[2][4] = {}, mid[2][4] = {};
-#pragma unroll
-            for (int i = 0; i < 2; ++i)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) m[i][e] = 0.f;
+            float low[2][4];
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
                 uint32_t r[4];
                 ldsm4(r, rows + ((mi >> 1) * 8 + mr) * St::PITCH + (d0 + ks * 16 + (mi & 1) * 8) * 2);
-                mma(lo[0], s[ks].l, r[0], r[1]);
-                mma(lo[1], s[ks].l, r[2], r[3]);
-                mma(mid[0], s[ks].m, r[0], r[1]);
-                mma(mid[1], s[ks].m, r[2], r[3]);
-                mma(m[0], s[ks].h, r[0], r[1]);
-                mma(m[1], s[ks].h, r[2], r[3]);
+                if (ks == 0) {
+                    mma_first(low[0], s[ks].l, r[0], r[1]);
+                    mma_first(low[1], s[ks].l, r[2], r[3]);
+                    mma_first(m[0], s[ks].h, r[0], r[1]);
+                    mma_first(m[1], s[ks].h, r[2], r[3]);
+                } else {
+                    mma(low[0], s[ks].l, r[0], r[1]);
+                    mma(low[1], s[ks].l, r[2], r[3]);
+                    mma(m[0], s[ks].h, r[0], r[1]);
+                    mma(m[1], s[ks].h, r[2], r[3]);
+                }
+                mma(low[0], s[ks].m, r[0], r[1]);
+                mma(low[1], s[ks].m, r[2], r[3]);
             }
 #pragma unroll
             for (int i = 0; i < 2; ++i)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) m[i][e] += mid[i][e] + lo[i][e];
+                for (int e = 0; e < 4; ++e) m[i][e] += low[i][e];
         };
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) split_tiles(S[2 * ks], S[2 * ks + 1], s[ks]);
@@ -536,16 +564,14 @@ delta_scan_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, con
             for (int i = 0; i < 2; ++i) *red_at(c & 1, 0, warp, i) = make_float4(m[i][0], m[i][1], m[i][2], m[i][3]);
         }
         __syncthreads();
+        Parts p;
+        fetch_x(c, p);
         float qs[2][4];
-        product(st + St::Q, qs);                              // the tensor cores work on this while X is formed
+        product(st + St::Q, qs);                              // the tensor cores work on this while the partial sums arrive
         Split3 x;
-        form_x(c, x);
+        form_x(p, x);
         float u[2][4];
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) u[i][e] = 0.f;
-        times(x, th, tm, tl, u);
+        times(x, th, tm, tl, u, Flag<true>());
         const float pc = f[3 * CK];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -955,326 +981,6 @@ int scan_as(const void* q, const void* k, const void* v, long long ld, const flo
     QNN_LAUNCH_CHECK();
 }
 
-// ---- one token per sequence -------------------------------------------------------------------------------------
-// A cluster of `splits` CTAs has one (sequence, value head); a CTA has `cw` of its value columns.  Everything is asked for
-// before the wait for the kernel in front but what that kernel writes: the state (the largest part), the ring of the
-// convolution's last inputs, filters, the gates' weights.  The CTAs of a cluster exchange their sums of squares for the
-// output norm through distributed shared memory.
-constexpr int STEP_THREADS = 256;
-
-struct StepArgs {
-    const void* p;              // rows of the input product: q | k | v | gate
-    long long ldp;
-    const void* x;              // [B, W]: the layer's normed input, for the gates' products
-    const void* w_ba;           // [2 H, W]
-    int W, w_dt;
-    const void* conv;           // [C, taps]
-    int c_dt, taps;
-    const float* rate;          // exp(A)
-    const float* bias;
-    const void* norm;           // [vdim]
-    int n_dt;
-    float eps, q_scale, unit_eps;
-    float* state;               // slot s: state + s * slot_stride: [taps][C]; from float s_off on [H][dim][vdim]
-    long long slot_stride, s_off;
-    const int* tok_pos;
-    const int* slots;
-    void* out;                  // [B, ldo]: H * vdim columns
-    long long ldo;
-    int B, H, G, dim, vdim, cw;
-};
-
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-__device__ __forceinline__ unsigned cluster_rank() {
-    unsigned r;
-    asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-    return r;
-}
-
-// VEC: the CTA's columns lie in fours on 16 bytes; RPT: state rows per thread
-template <typename T, int RPT, bool VEC>
-__global__ void __launch_bounds__(STEP_THREADS)
-delta_step_kernel(const StepArgs a, int splits) {
-    constexpr int V = VEC ? 4 : 1;
-    constexpr int CG = 16;                                    // threads side by side over columns: CG * V columns at most
-    constexpr int RG = STEP_THREADS / CG;                     // row groups
-    __shared__ float sk[MAX_DIM], sq[MAX_DIM], sv[CG * V], su[CG * V];
-    __shared__ float red[8][6];
-    __shared__ float part[2][8][CG * V];
-    __shared__ float squares[8];                              // by rank of the cluster
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int split = (int)(blockIdx.x % splits), h = (int)(blockIdx.x / splits), b = blockIdx.y;
-    const int g = h / (a.H / a.G), D = a.dim, VD = a.vdim;
-    const int c0 = split * a.cw, ncol = max(0, min(a.cw, VD - c0));
-    const int C = 2 * a.G * D + a.H * VD;
-    const int slot = a.slots[b], pos = a.tok_pos[b];
-    const int cg = tid % CG, rg = tid / CG;
-    if (splits > 1) cluster_arrive();                         // the other CTAs' shared memory is there (waited for below)
-    const bool live = slot >= 0;
-    float* base = a.state + (size_t)(live ? slot : 0) * a.slot_stride;
-    float* S0 = base + a.s_off + (size_t)h * D * VD + c0;
-    // Channels of the convolution that this CTA needs: q of its head, k of its head, its value columns, two or three per thread
-    // (dim <= 256).  The last three past inputs and their filter columns are asked for together, older ones one by one.
-    const int nch = 2 * D + ncol;
-    constexpr int PER = (2 * MAX_DIM + CG * V + STEP_THREADS - 1) / STEP_THREADS, NEAR = 3;
-    float past[PER], last[PER], near_x[PER][NEAR], near_w[PER][NEAR];
-    int chan[PER];
-    const int newest = pos % a.taps;                          // the ring's row of this token
-#pragma unroll
-    for (int e = 0; e < PER; ++e) {
-        const int i = tid + e * STEP_THREADS;
-        last[e] = 0.f;
-        chan[e] = -1;
-#pragma unroll
-        for (int j = 0; j < NEAR; ++j) near_x[e][j] = near_w[e][j] = 0.f;
-        if (i < nch) {
-            const int ch = i < D ? g * D + i : (i < 2 * D ? a.G * D + g * D + (i - D) : 2 * a.G * D + h * VD + c0 + (i - 2 * D));
-            const size_t f = (size_t)ch * a.taps + a.taps - 1;
-            chan[e] = ch;
-            last[e] = load_as_f(a.conv, a.c_dt, f);
-#pragma unroll
-            for (int j = 0; j < NEAR; ++j) {                  // j + 1 tokens ago
-                const int r = newest - 1 - j;
-                if (live && j + 1 < a.taps && pos - 1 - j >= 0) {
-                    near_w[e][j] = load_as_f(a.conv, a.c_dt, f - 1 - j);
-                    near_x[e][j] = base[(size_t)(r < 0 ? r + a.taps : r) * C + ch];
-                }
-            }
-        }
-    }
-    // the state: rows rg, rg + RG, ..; columns cg * V ..
-    float S[RPT][V];
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const int i = rg + r * RG;
-#pragma unroll
-        for (int c = 0; c < V; ++c) S[r][c] = 0.f;
-        if (live && i < D && cg * V < ncol) {
-            if (VEC) {
-                const float4 s4 = *reinterpret_cast<const float4*>(S0 + (size_t)i * VD + cg * 4);
-                S[r][0] = s4.x; S[r][1 % V] = s4.y; S[r][2 % V] = s4.z; S[r][3 % V] = s4.w;
-            } else {
-                S[r][0] = S0[(size_t)i * VD + cg];
-            }
-        }
-    }
-    const float rate = a.rate[h], bias = a.bias[h];
-    const float wn = tid < ncol ? load_as_f(a.norm, a.n_dt, c0 + tid) : 0.f;
-    // the gates' weights: the first two pieces of eight per thread stay as they come until the input is there
-    const size_t wb = (size_t)h * a.W, wa = (size_t)(a.H + h) * a.W;
-    const bool early = sizeof(T) == 2 && a.w_dt == QNN_DT_BF16 && a.W % 8 == 0;
-    constexpr int EARLY = 2;
-    Vec16<bf16> eb[EARLY], ea[EARLY];
-#pragma unroll
-    for (int u = 0; u < EARLY; ++u) {
-        const int i = (tid + u * STEP_THREADS) * 8;
-        eb[u].zero();
-        ea[u].zero();
-        if (early && i < a.W) {
-            eb[u].load((const bf16*)a.w_ba + wb + i);
-            ea[u].load((const bf16*)a.w_ba + wa + i);
-        }
-    }
-    pdl_wait();
-    const T* prow = (const T*)a.p + (size_t)b * a.ldp;
-    const T* xrow = (const T*)a.x + (size_t)b * a.W;
-    float raw[PER];
-#pragma unroll
-    for (int e = 0; e < PER; ++e) raw[e] = chan[e] >= 0 ? to_f(prow[chan[e]]) : 0.f;
-    const float z = tid < ncol ? to_f(prow[C + h * VD + c0 + tid]) : 0.f;
-    // the gates' products
-    float db = 0.f, da = 0.f;
-    if (early) {
-#pragma unroll
-        for (int u = 0; u < EARLY; ++u) {
-            const int i = (tid + u * STEP_THREADS) * 8;
-            if (i < a.W) {
-                float xf[8], f[8], e8[8];
-                load8_as_f(xrow, QNN_DT_BF16, i, xf);
-                eb[u].unpack(f);
-                ea[u].unpack(e8);
-#pragma unroll
-                for (int j = 0; j < 8; ++j) {
-                    db += xf[j] * f[j];
-                    da += xf[j] * e8[j];
-                }
-            }
-        }
-    }
-    if (a.W % 8 == 0) {
-        for (int i = (tid + (early ? EARLY * STEP_THREADS : 0)) * 8; i < a.W; i += STEP_THREADS * 8) {
-            float xf[8], f[8], e8[8];
-            load8_as_f(xrow, sizeof(T) == 2 ? QNN_DT_BF16 : QNN_DT_F32, i, xf);
-            load8_as_f(a.w_ba, a.w_dt, wb + i, f);
-            load8_as_f(a.w_ba, a.w_dt, wa + i, e8);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                db += xf[j] * f[j];
-                da += xf[j] * e8[j];
-            }
-        }
-    } else {
-        for (int i = tid; i < a.W; i += STEP_THREADS) {
-            const float xf = to_f(xrow[i]);
-            db += xf * load_as_f(a.w_ba, a.w_dt, wb + i);
-            da += xf * load_as_f(a.w_ba, a.w_dt, wa + i);
-        }
-    }
-    // the past inputs' part of the convolution, oldest first
-#pragma unroll
-    for (int e = 0; e < PER; ++e) {
-        past[e] = 0.f;
-        if (chan[e] >= 0 && live)
-            for (int j = min(a.taps - 1, pos); j > NEAR; --j) {
-                const int r = newest - j;
-                past[e] = fmaf(load_as_f(a.conv, a.c_dt, (size_t)chan[e] * a.taps + a.taps - 1 - j),
-                               base[(size_t)(r < 0 ? r + a.taps : r) * C + chan[e]], past[e]);
-            }
-#pragma unroll
-        for (int j = NEAR - 1; j >= 0; --j) past[e] = fmaf(near_w[e][j], near_x[e][j], past[e]);
-    }
-    // convolution, silu (rounded as a prompt's rows are stored), the ring's newest row
-    float ssq = 0.f, ssk = 0.f;
-#pragma unroll
-    for (int e = 0; e < PER; ++e) {
-        const int i = tid + e * STEP_THREADS;
-        if (chan[e] >= 0) {
-            const float y = to_f(from_f<T>(silu(fmaf(last[e], raw[e], past[e]))));
-            if (i < D) { sq[i] = y; ssq += y * y; }
-            else if (i < 2 * D) { sk[i - D] = y; ssk += y * y; }
-            else sv[i - 2 * D] = y;
-            // q and k belong to all heads of the group and all CTAs of a cluster: one of them keeps them
-            const bool keeper = i >= 2 * D || (split == 0 && h % (a.H / a.G) == 0);
-            if (live && keeper) base[(size_t)newest * C + chan[e]] = raw[e];
-        }
-    }
-    {
-        const float s0 = warp_sum(ssq), s1 = warp_sum(ssk), s2 = warp_sum(db), s3 = warp_sum(da);
-        if (lane == 0) { red[warp][0] = s0; red[warp][1] = s1; red[warp][2] = s2; red[warp][3] = s3; }
-    }
-    __syncthreads();
-    float tq = 0.f, tk = 0.f, tb = 0.f, ta = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) { tq += red[w][0]; tk += red[w][1]; tb += red[w][2]; ta += red[w][3]; }
-    const float fq = rsqrtf(tq + a.unit_eps) * a.q_scale, fk = rsqrtf(tk + a.unit_eps);
-    const float beta = beta_of(tb), gate = decay_of(ta, rate, bias);
-    // S^T k and S^T q: partial sums over a thread's rows, the two row groups of a warp by shuffle, the warps through shared memory
-    float mk[V], mq[V], kr[RPT], kq = 0.f;
-#pragma unroll
-    for (int c = 0; c < V; ++c) mk[c] = mq[c] = 0.f;
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const int i = rg + r * RG;
-        const float k1 = i < D ? sk[i] * fk : 0.f, q1 = i < D ? sq[i] * fq : 0.f;
-        kr[r] = k1;
-        if (cg == 0) kq += k1 * q1;
-#pragma unroll
-        for (int c = 0; c < V; ++c) {
-            mk[c] += k1 * S[r][c];
-            mq[c] += q1 * S[r][c];
-        }
-    }
-#pragma unroll
-    for (int c = 0; c < V; ++c) {
-        mk[c] += __shfl_xor_sync(0xffffffffu, mk[c], 16);
-        mq[c] += __shfl_xor_sync(0xffffffffu, mq[c], 16);
-        if (lane < CG) {
-            part[0][warp][cg * V + c] = mk[c];
-            part[1][warp][cg * V + c] = mq[c];
-        }
-    }
-    kq += __shfl_xor_sync(0xffffffffu, kq, 16);
-    if (lane == 0) red[warp][4] = kq;
-    __syncthreads();
-    float o = 0.f;
-    if (tid < CG * V) {
-        float s0 = 0.f, s1 = 0.f, s2 = 0.f;
-#pragma unroll
-        for (int w = 0; w < 8; ++w) { s0 += part[0][w][tid]; s1 += part[1][w][tid]; s2 += red[w][4]; }
-        const float u = tid < ncol ? beta * (sv[tid] - gate * s0) : 0.f;
-        su[tid] = u;
-        o = tid < ncol ? gate * s1 + s2 * u : 0.f;
-    }
-    float oo = o * o;                                         // threads of the first CG * V only: at most two warps
-    oo = warp_sum(oo);
-    if (lane == 0) red[warp][5] = oo;
-    __syncthreads();
-    float total = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) total += red[w][5];
-    if (splits > 1) {
-        cluster_wait();
-        if (tid < splits) {                                   // this CTA's sum to every rank
-            unsigned local = (unsigned)__cvta_generic_to_shared(&squares[cluster_rank()]), remote;
-            asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"((unsigned)tid));
-            asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(total) : "memory");
-        }
-        cluster_arrive();
-    }
-    // meanwhile the new state
-#pragma unroll
-    for (int r = 0; r < RPT; ++r) {
-        const int i = rg + r * RG;
-        if (live && i < D && cg * V < ncol) {
-            if (VEC) {
-                float4 s4;
-                s4.x = gate * S[r][0] + kr[r] * su[cg * V];
-                s4.y = gate * S[r][1 % V] + kr[r] * su[cg * V + 1 % V];
-                s4.z = gate * S[r][2 % V] + kr[r] * su[cg * V + 2 % V];
-                s4.w = gate * S[r][3 % V] + kr[r] * su[cg * V + 3 % V];
-                *reinterpret_cast<float4*>(S0 + (size_t)i * VD + cg * 4) = s4;
-            } else {
-                S0[(size_t)i * VD + cg] = gate * S[r][0] + kr[r] * su[cg];
-            }
-        }
-    }
-    if (splits > 1) {
-        cluster_wait();
-        total = 0.f;
-        for (int r = 0; r < splits; ++r) total += squares[r];
-    }
-    if (tid < ncol) {
-        const float y = o * rsqrtf(total / (float)VD + a.eps) * wn;
-        ((T*)a.out)[(size_t)b * a.ldo + (size_t)h * VD + c0 + tid] = from_f<T>(live ? y * silu(z) : 0.f);
-    }
-}
-
-template <typename T, int RPT, bool VEC>
-int step_as(const StepArgs& a, int splits, cudaStream_t st) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3((unsigned)(a.H * splits), (unsigned)a.B);
-    cfg.blockDim = dim3(STEP_THREADS);
-    cfg.stream = st;
-    cudaLaunchAttribute attr[2];
-    int n = 0;
-    if (splits > 1) {
-        attr[n].id = cudaLaunchAttributeClusterDimension;
-        attr[n].val.clusterDim.x = (unsigned)splits;
-        attr[n].val.clusterDim.y = 1;
-        attr[n].val.clusterDim.z = 1;
-        ++n;
-    }
-    if (pdl_enabled() && (long long)a.H * splits * a.B <= pdl_max_grid()) {
-        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-        attr[n].val.programmaticStreamSerializationAllowed = 1;
-        ++n;
-    }
-    cfg.attrs = attr;
-    cfg.numAttrs = n;
-    const cudaError_t rc = cudaLaunchKernelEx(&cfg, delta_step_kernel<T, RPT, VEC>, a, splits);
-    if (rc != cudaSuccess) return (int)rc;
-    QNN_LAUNCH_CHECK();
-}
-
-template <typename T, bool VEC>
-int step_rows(const StepArgs& a, int splits, cudaStream_t st) {
-    const int rpt = (a.dim + 15) / 16;
-    if (rpt <= 4) return step_as<T, 4, VEC>(a, splits, st);
-    if (rpt <= 8) return step_as<T, 8, VEC>(a, splits, st);
-    return step_as<T, 16, VEC>(a, splits, st);
-}
-
 }  // namespace
 
 // q, k: [rows, G * dim], v: [rows, H * vdim] of `dtype`, one row pitch `ld`; inv: [rows, ldi] with 1 / length of the G query heads,
@@ -1285,7 +991,7 @@ QNN_API int qnn_delta_chunks(const void* q, const void* k, long long ld, int dty
                              int ldp, const float* rate, const float* bias, float q_scale, const int* seq_row0, const int* seq_len,
                              void* rec, int B, int longest, int H, int G, int dim, int tensor_cores, cudaStream_t st) {
     if (B <= 0 || longest <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > MAX_DIM || B > 65535 || G > 65535 || ldi < 2 * G || ldp < 2 * H)
+    if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > DELTA_MAX_DIM || B > 65535 || G > 65535 || ldi < 2 * G || ldp < 2 * H)
         return QNN_ERR_ARGUMENT;
     if ((seq_row0 == nullptr) != (seq_len == nullptr)) return QNN_ERR_ARGUMENT;
     if (tensor_cores) {
@@ -1325,7 +1031,7 @@ QNN_API int qnn_delta_scan(const void* q, const void* k, const void* v, long lon
                            int tensor_cores,
                            cudaStream_t st) {
     if (B <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > MAX_DIM || vdim <= 0 || B > 65535 || H > 65535 || ldi < 2 * G ||
+    if (H <= 0 || G <= 0 || H % G || dim <= 0 || dim > DELTA_MAX_DIM || vdim <= 0 || B > 65535 || H > 65535 || ldi < 2 * G ||
         slot_stride < (long long)H * dim * vdim || (cpt != 1 && cpt != 2) || (seq_row0 == nullptr) != (seq_len == nullptr))
         return QNN_ERR_ARGUMENT;
     const size_t es = dtype == QNN_DT_BF16 ? 2 : 4;
@@ -1357,32 +1063,4 @@ QNN_API int qnn_delta_scan(const void* q, const void* k, const void* v, long lon
 #undef QNN_DS_ROWS
 #undef QNN_DS_COLS
 #undef QNN_DS
-}
-
-// p: [B, ldp] rows q | k | v | gate of the input product; x: [B, W] the product's input; w_ba: [2 H, W]; conv: [2 G dim + H vdim,
-// taps]; state: slot s at state + s * slot_stride: [taps][channels] the ring of last inputs (position p in row p mod taps), from
-// float s_off on [H][dim][vdim]; slots negative: a row of no sequence (its output is zero).  out: [B, ldo] of `dtype`.
-QNN_API int qnn_delta_step(const void* p, int dtype, long long ldp, const void* x, int W, const void* w_ba, int w_dt,
-                           const void* conv, int c_dt, int taps, const float* rate, const float* bias, const void* norm, int n_dt,
-                           float eps, float unit_eps, float q_scale, float* state, long long slot_stride, long long s_off, const int* tok_pos,
-                           const int* slots, void* out, long long ldo, int B, int H, int G, int dim, int vdim, cudaStream_t st) {
-    if (B <= 0) return 0;
-    const long long C = 2LL * G * dim + (long long)H * vdim;
-    if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || taps < 1 || W <= 0 || ldp < C + (long long)H * vdim ||
-        s_off < taps * C || slot_stride < s_off + (long long)H * dim * vdim || B > 65535 || ldo < (long long)H * vdim)
-        return QNN_ERR_ARGUMENT;
-    if (dim > MAX_DIM) return QNN_ERR_UNSUPPORTED;
-    if (W % 8 == 0 && (((uintptr_t)x | (uintptr_t)w_ba) & 15)) return QNN_ERR_ARGUMENT;
-    // columns of a CTA: up to 64 in fours, up to 16 one by one; at most eight CTAs share a head
-    const bool vec = vdim % 4 == 0 && s_off % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
-    const int most = vec ? 64 : 16;
-    int splits = 1;
-    while (splits < 8 && (long long)splits * most < vdim) splits *= 2;
-    int cw = (vdim + splits - 1) / splits;
-    if (vec) cw = (cw + 3) / 4 * 4;
-    if (cw > most) return QNN_ERR_UNSUPPORTED;
-    StepArgs a = {p, ldp, x, w_ba, W, w_dt, conv, c_dt, taps, rate, bias, norm, n_dt, eps, q_scale, unit_eps, state, slot_stride, s_off,
-                  tok_pos, slots, out, ldo, B, H, G, dim, vdim, cw};
-    if (dtype == QNN_DT_BF16) return vec ? step_rows<bf16, true>(a, splits, st) : step_rows<bf16, false>(a, splits, st);
-    return vec ? step_rows<float, true>(a, splits, st) : step_rows<float, false>(a, splits, st);
 }
