@@ -179,7 +179,8 @@ __device__ __forceinline__ void cp16(unsigned dst, const void* src) {
 }
 
 // What a chunk leaves for the scan, per value head: T and A in three bfloat16 matrices each ([3][2][16][8]: row t of the columns
-// j = 8 c .. 8 c + 7, c = 0, 1, so that the eight rows of an ldmatrix lie side by side), then per row P_t / |k_t|, P_t q_scale / |q_t|, D_16,t / |k_t|, and P_16: 3280 bytes.
+// j = 8 c .. 8 c + 7, c = 0, 1, so that the eight rows of an ldmatrix lie side by side), then per row P_t / |k_t|,
+// P_t q_scale / |q_t|, D_16,t / |k_t|, and P_16: 3280 bytes.
 constexpr int TC_T = 0, TC_A = 3 * CK * CK * 2, TC_F = 2 * TC_A, TC_RECORD = TC_F + (3 * CK + 4) * 4;
 
 // a warp per (chunk, query/key head)
@@ -316,7 +317,8 @@ delta_chunks_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, l
 // and its quarter of the update by itself, all in registers.  Q S is formed in the shadow of that; two more warps take alternate
 // chunks and turn it into the outputs a chunk later; the last two fetch chunks ahead, keys and values the one, queries and what
 // qnn_delta_chunks left the other.
-constexpr int TC_WORKERS = 4, TC_READERS = 2, TC_LOADERS = 2, TC_THREADS = 32 * (TC_WORKERS + TC_READERS + TC_LOADERS), TC_STAGES = 6, TC_AHEAD = TC_STAGES - 2;
+constexpr int TC_WORKERS = 4, TC_READERS = 2, TC_LOADERS = 2;
+constexpr int TC_THREADS = 32 * (TC_WORKERS + TC_READERS + TC_LOADERS), TC_STAGES = 6, TC_AHEAD = TC_STAGES - 2;
 
 template <bool V> struct Flag { static constexpr bool value = V; };
 
@@ -984,8 +986,8 @@ int scan_as(const void* q, const void* k, const void* v, long long ld, const flo
 }  // namespace
 
 // q, k: [rows, G * dim], v: [rows, H * vdim] of `dtype`, one row pitch `ld`; inv: [rows, ldi] with 1 / length of the G query heads,
-// then of the G key heads; seq_row0, seq_len: first row and row count of the B sequences (both null: row b alone); pre: [rows, ldp] with b of the H heads, then a of the H heads; rate, bias: [H] float32 (rate =
-// exp(A)); rec: at least (T / 16 + B) * H records of 3280 bytes (tensor_cores) or 544 floats.  longest: the most rows of a
+// then of the G key heads; seq_row0, seq_len: first row and row count of the B sequences (both null: row b alone); pre:
+// [rows, ldp] with b of the H heads, then a of the H heads; rate, bias: [H] float32 (rate = exp(A)); rec: at least (T / 16 + B) * H records of 3280 bytes (tensor_cores) or 544 floats.  longest: the most rows of a
 // sequence.  dim up to 256.  tensor_cores: bfloat16 rows, dim and vdim multiples of 8, everything on 16 bytes.
 QNN_API int qnn_delta_chunks(const void* q, const void* k, long long ld, int dtype, const float* inv, int ldi, const float* pre,
                              int ldp, const float* rate, const float* bias, float q_scale, const int* seq_row0, const int* seq_len,
